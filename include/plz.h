@@ -399,6 +399,94 @@ int32_t plz_add(const void* a, int64_t lda, const void* b, int64_t ldb, const vo
 int32_t plz_bwd_dw_hard_lora(const plz_weight_t* w, const void* x, int64_t ldx, const void* dY, int64_t lddy, int32_t M, float* dpalette,
                              const void* t, const void* dt, int32_t rank, float* dA, float* dB, void* stream);
 
+/* ---- Hybrid decoders: recurrent and attention mixers over a cache of per-sequence state ------------------------------------
+ * dtype: 0 = bf16, 1 = fp32: the type of activations and Linear weights. Accumulation, norms, scores, decays, states and the
+ * residual stream are fp32 in both. Rows are b * n + t: B sequences advance in lockstep by n tokens; pos is ONE int32 in device
+ * memory, the position of the first of the n tokens, so that a captured step can be replayed at later positions.
+ *
+ * plz_seq_linear: y = act(x W^T + bias), W [N, K] row-major, act 0 none / 1 square of relu; y_f32: write fp32 from bf16 operands.
+ *   Any shape; 16-byte aligned rows take the streaming (M <= 8) and tcgen05 (bf16) kernels.
+ * plz_seq_embed: x fp32 [rows, W] = table[ids] * scale, xb (may be NULL) the same in dtype; an id outside [0, vocab) gives zeros and
+ *   sets *bad (may be NULL).
+ * plz_seq_residual_norm: x += mult * y / sqrt(mean(y^2) + eps) * (w + w_offset); xb (may be NULL) = x in dtype. w fp32 [W].
+ * plz_seq_rows_norm: out[i] = x[idx[i]] / rms * (w + w_offset) in dtype (idx NULL: row i).
+ * plz_seq_norm_gate: out = o / rms(o over each group of L values) * w[c] * sigmoid(gate), o fp32 [rows, groups * L], w fp32 [L].
+ * plz_delta_prep: causal convolution + silu on the q, k, v slices of a projection, unit norm of q and k per head (q times q_scale),
+ *   logg = -exp(A_log) * softplus(a + dt_bias), beta = sigmoid(b slice); updates the convolution inputs `conv`
+ *   [B, n_taps - 1, 2 G dk + H dv] (dtype, oldest first).
+ * plz_delta_rule / plz_decay_attn: the recurrences, state fp32 [B, H, dk, dv] updated in place, o fp32 [B * n, H * dv].
+ * plz_attn_prep: RMS norm of the whole q and k projections, optional value mixing with the first mixing layer's values, and the
+ *   write of keys and values into the cache at *pos + t.
+ * plz_attn_bias: causal attention of the n new tokens against the cache (which already holds them), score * scale + bias by distance
+ *   (bias points at distance 0 of head 0; entry n_bias - 1 holds for everything farther; rows ldb apart, readable from 128 entries
+ *   before distance 0 to 256 entries past n_bias - 1), optional sink in the denominator. host_pos = *pos when the caller knows it, or
+ *   -1 (n == 1 only). ws: plz_attn_bias_ws_bytes bytes for n == 1, else unused. */
+int32_t plz_seq_linear(int32_t dtype, const void* x, int64_t ldx, int32_t M, int32_t K, const void* w, int64_t ldw, int32_t N, const void* bias,
+                       int32_t act, void* y, int64_t ldy, int32_t y_f32, void* stream);
+int32_t plz_seq_embed(int32_t dtype, const void* table, int64_t ldt, const int64_t* ids, int64_t rows, int32_t W, int64_t vocab, float scale,
+                      float* x, void* xb, int32_t* bad, void* stream);
+int32_t plz_seq_residual_norm(int32_t dtype, const void* y, int64_t ldy, const float* w, float w_offset, float mult, float eps, int64_t rows,
+                              int32_t W, float* x, void* xb, void* stream);
+int32_t plz_seq_rows_norm(int32_t dtype, const float* x, const int64_t* idx, const float* w, float w_offset, float eps, int64_t rows, int32_t W,
+                          void* out, void* stream);
+int32_t plz_seq_norm_gate(int32_t dtype, const float* o, const void* gate, int64_t ldg, const float* w, float eps, int64_t rows, int32_t groups,
+                          int32_t L, void* out, void* stream);
+
+typedef struct plz_delta_prep {
+    const void* proj; int64_t ldp; int32_t off_q, off_k, off_v, off_b;   /* projection rows (dtype) and column offsets of the slices */
+    const void* a; int64_t lda;                                          /* dtype [rows, H * dk]: decay pre-activation */
+    const float* taps; const float* A_log; const float* dt_bias;         /* [2 G dk + H dv, n_taps], [H], [H * dk] */
+    void* conv; int32_t n_taps;
+    int32_t B, n, H, G, dk, dv;
+    float q_scale;
+    float* q; float* k; float* v; float* logg; float* beta;              /* outputs, fp32 */
+} plz_delta_prep_t;
+int32_t plz_delta_prep(int32_t dtype, const plz_delta_prep_t* args, void* stream);
+
+typedef struct plz_delta_rule {
+    const float* q; const float* k; const float* v; const float* logg; const float* beta;   /* as written by plz_delta_prep */
+    float* state; float* o;
+    int32_t B, n, H, G, dk, dv;
+} plz_delta_rule_t;
+int32_t plz_delta_rule(const plz_delta_rule_t* args, void* stream);
+
+typedef struct plz_decay_attn {
+    const void* q; const void* k; const void* v; int64_t ld;   /* slices of one projection before silu, dtype, rows ld apart */
+    const float* decay;                                        /* [H] */
+    float* state; float* o;
+    int32_t B, n, H, dk, dv;
+} plz_decay_attn_t;
+int32_t plz_decay_attn(int32_t dtype, const plz_decay_attn_t* args, void* stream);
+
+typedef struct plz_attn_prep {
+    const void* proj; int64_t ldp; int32_t off_q, off_k, off_v;
+    const float* wq; const float* wk; const float* mix;        /* [qw], [kw], [1] or NULL */
+    void* v_first; int32_t v_first_write;                      /* [rows, vw]: written by the first mixing layer, read by the others */
+    void* q; void* kc; void* vc; int64_t k_batch, v_batch;     /* [rows, qw]; caches, elements between sequences */
+    const int32_t* pos;
+    int32_t B, n, qw, kw, vw, cap;
+    float eps;
+} plz_attn_prep_t;
+int32_t plz_attn_prep(int32_t dtype, const plz_attn_prep_t* args, void* stream);
+
+typedef struct plz_attn_bias {
+    const void* q; int64_t ldq;                                /* [B * n, H * dk] */
+    const void* k; const void* v; int64_t k_batch, v_batch;    /* caches [B, cap, G * dk], [B, cap, G * dv] */
+    void* o; int64_t ldo;                                      /* [B * n, H * dv] */
+    const float* bias; int64_t ldb; int32_t n_bias;
+    const int32_t* pos; int32_t host_pos, cap;
+    int32_t B, n, H, G, dk, dv, sink;
+    float scale;
+} plz_attn_bias_t;
+int64_t plz_attn_bias_ws_bytes(int32_t B, int32_t H, int32_t G, int32_t dv, int32_t cap);
+int32_t plz_attn_bias(int32_t dtype, const plz_attn_bias_t* args, void* ws, int64_t ws_bytes, void* stream);
+/* *pos += n, at the end of a step */
+int32_t plz_advance(int32_t* pos, int32_t n, void* stream);
+/* Next token of every row of fp32 logits [rows, V]: temperature 0: the largest (first of equals); else a draw from
+ * softmax(logits / temperature) over the top_k largest (top_k <= 0: all), noise from a counter hash of (seed, *pos, row, token). */
+int32_t plz_sample(const float* logits, int64_t ld, int32_t rows, int32_t V, float temperature, int32_t top_k, uint32_t seed, const int32_t* pos,
+                   int64_t* out, void* stream);
+
 #ifdef __cplusplus
 }
 #endif

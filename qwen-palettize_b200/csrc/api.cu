@@ -933,4 +933,132 @@ int32_t plz_bwd_dw_hard_lora(const plz_weight_t* w, const void* x, int64_t ldx, 
     return bwd_dw_common(EPI_HARD, w, x, ldx, dY, lddy, M, nullptr, nullptr, 1.0f, nullptr, dpalette, stream, t, dt, rank, dA, dB);
 }
 
+// ---- hybrid decoders ---------------------------------------------------------------------------------------
+static int check_dtype(int32_t dtype) {
+    if (dtype != 0 && dtype != 1) { set_last_error("dtype %d (0 = bf16, 1 = fp32)", dtype); return PLZ_ERR_UNSUPPORTED; }
+    return PLZ_OK;
+}
+static int check_rows(int64_t rows) {
+    if (rows < 0 || rows > 0x7FFFFFFF) { set_last_error("%lld rows", (long long)rows); return PLZ_ERR_BAD_SHAPE; }
+    return PLZ_OK;
+}
+
+int32_t plz_seq_linear(int32_t dtype, const void* x, int64_t ldx, int32_t M, int32_t K, const void* w, int64_t ldw, int32_t N, const void* bias,
+                       int32_t act, void* y, int64_t ldy, int32_t y_f32, void* stream) {
+    int rc = check_dtype(dtype);
+    if (rc) return rc;
+    if (M < 0 || ldx < K || ldw < K || ldy < N) { set_last_error("seq_linear: bad shape M=%d N=%d K=%d", M, N, K); return PLZ_ERR_BAD_SHAPE; }
+    return launch_seq_linear(dtype, x, ldx, M, K, w, ldw, N, bias, act, y, ldy, y_f32, (cudaStream_t)stream);
+}
+
+int32_t plz_seq_embed(int32_t dtype, const void* table, int64_t ldt, const int64_t* ids, int64_t rows, int32_t W, int64_t vocab, float scale,
+                      float* x, void* xb, int32_t* bad, void* stream) {
+    int rc = check_dtype(dtype);
+    if (rc || (rc = check_rows(rows))) return rc;
+    if (W <= 0 || vocab <= 0 || ldt < W) { set_last_error("seq_embed: bad shape"); return PLZ_ERR_BAD_SHAPE; }
+    if (rows && (!table || !ids || !x)) { set_last_error("null pointer"); return PLZ_ERR_NULL; }
+    return launch_seq_embed(dtype, table, ldt, (const long long*)ids, rows, W, vocab, scale, x, xb, bad, (cudaStream_t)stream);
+}
+
+int32_t plz_seq_residual_norm(int32_t dtype, const void* y, int64_t ldy, const float* w, float w_offset, float mult, float eps, int64_t rows,
+                              int32_t W, float* x, void* xb, void* stream) {
+    int rc = check_dtype(dtype);
+    if (rc || (rc = check_rows(rows))) return rc;
+    if (W <= 0 || ldy < W) { set_last_error("seq_residual_norm: bad shape"); return PLZ_ERR_BAD_SHAPE; }
+    if (rows && (!y || !w || !x)) { set_last_error("null pointer"); return PLZ_ERR_NULL; }
+    return launch_seq_residual_norm(dtype, y, ldy, w, w_offset, mult, eps, rows, W, x, xb, (cudaStream_t)stream);
+}
+
+int32_t plz_seq_rows_norm(int32_t dtype, const float* x, const int64_t* idx, const float* w, float w_offset, float eps, int64_t rows, int32_t W,
+                          void* out, void* stream) {
+    int rc = check_dtype(dtype);
+    if (rc || (rc = check_rows(rows))) return rc;
+    if (W <= 0) { set_last_error("seq_rows_norm: bad shape"); return PLZ_ERR_BAD_SHAPE; }
+    if (rows && (!x || !w || !out)) { set_last_error("null pointer"); return PLZ_ERR_NULL; }
+    return launch_seq_rows_norm(dtype, x, (const long long*)idx, w, w_offset, eps, rows, W, out, (cudaStream_t)stream);
+}
+
+int32_t plz_seq_norm_gate(int32_t dtype, const float* o, const void* gate, int64_t ldg, const float* w, float eps, int64_t rows, int32_t groups,
+                          int32_t L, void* out, void* stream) {
+    int rc = check_dtype(dtype);
+    if (rc || (rc = check_rows(rows))) return rc;
+    if (groups <= 0 || groups > 65535 || L <= 0 || ldg < (int64_t)groups * L) { set_last_error("seq_norm_gate: bad shape"); return PLZ_ERR_BAD_SHAPE; }
+    if (rows && (!o || !gate || !w || !out)) { set_last_error("null pointer"); return PLZ_ERR_NULL; }
+    return launch_seq_norm_gate(dtype, o, gate, ldg, w, eps, rows, groups, L, out, (cudaStream_t)stream);
+}
+
+int32_t plz_delta_prep(int32_t dtype, const plz_delta_prep_t* a, void* stream) {
+    int rc = check_dtype(dtype);
+    if (rc) return rc;
+    if (!a || !a->proj || !a->a || !a->taps || !a->A_log || !a->dt_bias || (!a->conv && a->n_taps > 1) || !a->q || !a->k || !a->v || !a->logg || !a->beta) {
+        set_last_error("null pointer"); return PLZ_ERR_NULL;
+    }
+    if (a->B < 0 || a->n < 0 || a->H <= 0 || a->G <= 0 || a->H % a->G || a->dk <= 0 || a->dv <= 0 || a->n_taps <= 0 || (rc = check_rows((int64_t)a->B * a->n))) {
+        set_last_error("delta_prep: bad shape H=%d G=%d dk=%d dv=%d taps=%d", a->H, a->G, a->dk, a->dv, a->n_taps); return PLZ_ERR_BAD_SHAPE;
+    }
+    return launch_delta_prep(dtype, *a, (cudaStream_t)stream);
+}
+
+int32_t plz_delta_rule(const plz_delta_rule_t* a, void* stream) {
+    if (!a || !a->q || !a->k || !a->v || !a->logg || !a->beta || !a->state || !a->o) { set_last_error("null pointer"); return PLZ_ERR_NULL; }
+    if (a->B < 0 || a->n < 0 || a->H <= 0 || a->G <= 0 || a->H % a->G || a->dk <= 0 || a->dv <= 0 || a->H > 65535 || a->B > 65535) {
+        set_last_error("delta_rule: bad shape H=%d G=%d dk=%d dv=%d", a->H, a->G, a->dk, a->dv); return PLZ_ERR_BAD_SHAPE;
+    }
+    return launch_recurrent_delta(*a, (cudaStream_t)stream);
+}
+
+int32_t plz_decay_attn(int32_t dtype, const plz_decay_attn_t* a, void* stream) {
+    int rc = check_dtype(dtype);
+    if (rc) return rc;
+    if (!a || !a->q || !a->k || !a->v || !a->decay || !a->state || !a->o) { set_last_error("null pointer"); return PLZ_ERR_NULL; }
+    if (a->B < 0 || a->n < 0 || a->H <= 0 || a->dk <= 0 || a->dv <= 0 || a->H > 65535 || a->B > 65535) {
+        set_last_error("decay_attn: bad shape H=%d dk=%d dv=%d", a->H, a->dk, a->dv); return PLZ_ERR_BAD_SHAPE;
+    }
+    return launch_recurrent_decay(dtype, *a, (cudaStream_t)stream);
+}
+
+int32_t plz_attn_prep(int32_t dtype, const plz_attn_prep_t* a, void* stream) {
+    int rc = check_dtype(dtype);
+    if (rc) return rc;
+    if (!a || !a->proj || !a->wq || !a->wk || !a->q || !a->kc || !a->vc || !a->pos || ((a->mix || a->v_first_write) && !a->v_first)) {
+        set_last_error("null pointer"); return PLZ_ERR_NULL;
+    }
+    if (a->B < 0 || a->n < 0 || a->qw <= 0 || a->kw <= 0 || a->vw <= 0 || (rc = check_rows((int64_t)a->B * a->n))) { set_last_error("attn_prep: bad shape"); return PLZ_ERR_BAD_SHAPE; }
+    return launch_attn_prep(dtype, *a, (cudaStream_t)stream);
+}
+
+int64_t plz_attn_bias_ws_bytes(int32_t B, int32_t H, int32_t G, int32_t dv, int32_t cap) {
+    if (B <= 0 || H <= 0 || G <= 0 || H % G || dv <= 0 || cap <= 0) return 0;
+    return attn_bias_decode_ws_bytes(B, H, G, dv, cap);
+}
+
+int32_t plz_attn_bias(int32_t dtype, const plz_attn_bias_t* a, void* ws, int64_t ws_bytes, void* stream) {
+    int rc = check_dtype(dtype);
+    if (rc) return rc;
+    if (!a || !a->q || !a->k || !a->v || !a->o || !a->pos) { set_last_error("null pointer"); return PLZ_ERR_NULL; }
+    if (a->B < 0 || a->n < 0 || a->H <= 0 || a->G <= 0 || a->H % a->G || a->dk <= 0 || a->dv <= 0 || a->H > 65535 || a->B > 65535 || (a->bias && a->n_bias <= 0) ||
+        (a->n > 1 && a->host_pos < 0) || a->host_pos + (int64_t)a->n > a->cap) {
+        set_last_error("attn_bias: bad shape H=%d G=%d dk=%d dv=%d n=%d pos=%d cap=%d", a->H, a->G, a->dk, a->dv, a->n, a->host_pos, a->cap); return PLZ_ERR_BAD_SHAPE;
+    }
+    if (a->B == 0 || a->n == 0) return PLZ_OK;
+    cudaStream_t s = (cudaStream_t)stream;
+    const int per16 = dtype == 0 ? 8 : 4;
+    const bool vec = a->dk % 8 == 0 && a->dv % 8 == 0 && a->ldq % per16 == 0 && a->k_batch % per16 == 0 && a->v_batch % per16 == 0 &&
+                     !((uintptr_t)a->q & 15) && !((uintptr_t)a->k & 15) && !((uintptr_t)a->v & 15);
+    if (a->n == 1 && vec && a->dk <= 256 && a->dv <= 256) return launch_attn_bias_decode(dtype, *a, a->cap, ws, ws ? ws_bytes : 0, s);
+    return launch_attn_bias_simt(dtype, *a, s);
+}
+
+int32_t plz_advance(int32_t* pos, int32_t n, void* stream) {
+    if (!pos) { set_last_error("null pointer"); return PLZ_ERR_NULL; }
+    return launch_advance(pos, n, (cudaStream_t)stream);
+}
+
+int32_t plz_sample(const float* logits, int64_t ld, int32_t rows, int32_t V, float temperature, int32_t top_k, uint32_t seed, const int32_t* pos,
+                   int64_t* out, void* stream) {
+    if (rows < 0 || V <= 0 || ld < V || !(temperature >= 0.f)) { set_last_error("sample: bad arguments"); return PLZ_ERR_BAD_SHAPE; }
+    if (rows && (!logits || !pos || !out)) { set_last_error("null pointer"); return PLZ_ERR_NULL; }
+    return launch_sample(logits, ld, rows, V, temperature, top_k, seed, pos, (long long*)out, (cudaStream_t)stream);
+}
+
 }  // extern "C"

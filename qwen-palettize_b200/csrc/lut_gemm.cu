@@ -48,7 +48,8 @@ struct LutGemmParams {
     __nv_bfloat16* gate_out; __nv_bfloat16* up_out; long long ld_gu;  // FUSE == 1: optional copies of the two pre-activations
     const __nv_bfloat16* col_scale;  // [K]: norm weight g[k], multiplied into the decoded weights (may be null)
     const float* row_scale;          // [M]: 1 / rms(x[m, :]), applied to the accumulator rows (may be null)
-    const __nv_bfloat16* bias;       // FUSE == 2: [J], added in fp32 before the bf16 store (may be null)
+    const __nv_bfloat16* bias;       // FUSE >= 2: [J], added in fp32 before the bf16 store (may be null)
+    int relu2;                       // FUSE == 3: 1 = square of relu after the bias
     StatusWord* status;
     unsigned long long* prof;  // optional [gridDim][8] cycle counters of the MMA thread (diagnostics)
 };
@@ -102,7 +103,7 @@ lut_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
 
     const int warp = threadIdx.x >> 5;
     const int lane = threadIdx.x & 31;
-    const int nkb = p.R / kBK;
+    const int nkb = (p.R + kBK - 1) / kBK;  // dense B: columns past R read as zero
     const int nkb_total = nkb + p.n_extra;
     const int n_tiles = p.n_items;
 
@@ -476,19 +477,26 @@ lut_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
                             __syncwarp();
                             if (lane == 0) mbar_arrive(tmem_empty);
                         }
-                        if (FUSE == 2 && p.bias != nullptr) {
+                        if ((FUSE == 2 && p.bias != nullptr) || FUSE == 3) {
                             // bias in fp32 before the rounding (scripts/fused_lut_kernel.cu:512-514); columns past J are
                             // clipped by the TMA store, so only the loads need the bound
                             const int jc = j0 + col + c * 32;
 #pragma unroll
                             for (int g = 0; g < 4; ++g) {
                                 uint4 bb = make_uint4(0u, 0u, 0u, 0u);
-                                if (jc + g * 8 < p.J) bb = __ldg(reinterpret_cast<const uint4*>(p.bias + jc + g * 8));
+                                if ((FUSE == 2 || p.bias != nullptr) && jc + g * 8 < p.J) bb = __ldg(reinterpret_cast<const uint4*>(p.bias + jc + g * 8));
                                 const uint32_t bw[4] = {bb.x, bb.y, bb.z, bb.w};
 #pragma unroll
                                 for (int i = 0; i < 4; ++i) {
                                     v[g * 8 + 2 * i] = __float_as_uint(__uint_as_float(v[g * 8 + 2 * i]) * scale + __uint_as_float(bw[i] << 16));
                                     v[g * 8 + 2 * i + 1] = __float_as_uint(__uint_as_float(v[g * 8 + 2 * i + 1]) * scale + __uint_as_float(bw[i] & 0xFFFF0000u));
+                                    if (FUSE == 3 && p.relu2) {
+#pragma unroll
+                                        for (int q = 0; q < 2; ++q) {
+                                            const float r = fmaxf(__uint_as_float(v[g * 8 + 2 * i + q]), 0.f);
+                                            v[g * 8 + 2 * i + q] = __float_as_uint(r * r);
+                                        }
+                                    }
                                 }
                             }
 #pragma unroll
@@ -573,7 +581,7 @@ static int launch_t(const LutGemmArgs& a, cudaStream_t stream) {
     p.packed2 = (const uint8_t*)a.packed2; p.palette2 = (const __nv_bfloat16*)a.palette2;
     p.gate_out = (__nv_bfloat16*)a.gate_out; p.up_out = (__nv_bfloat16*)a.up_out; p.ld_gu = a.ld_gu;
     p.col_scale = (const __nv_bfloat16*)a.col_scale; p.row_scale = a.row_scale;
-    p.bias = (const __nv_bfloat16*)a.bias;
+    p.bias = (const __nv_bfloat16*)a.bias; p.relu2 = a.act == 1;
     p.status = device_status_ptr();
     p.prof = (unsigned long long*)a.prof;
     auto kern = lut_gemm_kernel<MT, BMODE, NARROW, FUSE>;
@@ -602,7 +610,8 @@ static int launch_t(const LutGemmArgs& a, cudaStream_t stream) {
 
 int launch_lut_gemm(const LutGemmArgs& a, cudaStream_t stream) {
     if (a.M <= 0 || a.J <= 0 || a.R <= 0) { set_last_error("lut_gemm: empty problem"); return PLZ_ERR_BAD_SHAPE; }
-    if (a.R % kBK) { set_last_error("lut_gemm: reduction length %d is not a multiple of 64", a.R); return PLZ_ERR_BAD_SHAPE; }
+    const bool dense_k = a.bmode == B_TMA_K && a.r2 == 0;   // operands by TMA, reduction length padded with zeros by the copy
+    if (a.R % (dense_k ? 8 : kBK)) { set_last_error("lut_gemm: reduction length %d is not a multiple of %d", a.R, dense_k ? 8 : kBK); return PLZ_ERR_BAD_SHAPE; }
     if (a.J % 8) { set_last_error("lut_gemm: output width %d is not a multiple of 8", a.J); return PLZ_ERR_BAD_SHAPE; }
     if (a.r2 < 0 || a.r2 > 64 || (a.r2 % 8)) { set_last_error("lut_gemm: extra rank %d must be a multiple of 8 in [0, 64]", a.r2); return PLZ_ERR_BAD_SHAPE; }
     if (((uintptr_t)a.out & 15) || ((a.ld_out * 2) & 15)) { set_last_error("lut_gemm: output must be 16-byte aligned"); return PLZ_ERR_BAD_ALIGN; }
@@ -628,6 +637,10 @@ int launch_lut_gemm(const LutGemmArgs& a, cudaStream_t stream) {
             return big ? launch_t<2, B_DECODE_K, false>(a, stream) : launch_t<1, B_DECODE_K, false>(a, stream);
         case B_DECODE_MN: return big ? launch_t<2, B_DECODE_MN, false>(a, stream) : launch_t<1, B_DECODE_MN, false>(a, stream);
         case B_TMA_K:
+            if (a.fuse == 3) {   // bias and / or activation in the epilogue
+                if (narrow) return launch_t<1, B_TMA_K, true, 3>(a, stream);
+                return big ? launch_t<2, B_TMA_K, false, 3>(a, stream) : launch_t<1, B_TMA_K, false, 3>(a, stream);
+            }
             if (narrow) return launch_t<1, B_TMA_K, true>(a, stream);
             return big ? launch_t<2, B_TMA_K, false>(a, stream) : launch_t<1, B_TMA_K, false>(a, stream);
         case B_TMA_MN:

@@ -7,16 +7,7 @@
 
 #include "plz_sm100.cuh"
 
-// error codes returned through the C ABI (include/plz.h documents them)
-#define PLZ_OK 0
-#define PLZ_ERR_BAD_SHAPE 1
-#define PLZ_ERR_BAD_ALIGN 2
-#define PLZ_ERR_UNSUPPORTED 3
-#define PLZ_ERR_CUDA 4
-#define PLZ_ERR_WORKSPACE 5
-#define PLZ_ERR_DEVICE_WAIT 6
-#define PLZ_ERR_NULL 7
-#define PLZ_ERR_TOO_LARGE 8
+#include "../../include/plz.h"   // error codes
 
 namespace plz {
 

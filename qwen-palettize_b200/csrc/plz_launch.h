@@ -1,5 +1,6 @@
 // Argument structures and prototypes of the kernel launchers (one per .cu file).
 #pragma once
+#include "../../include/plz.h"
 #include "plz_host.h"
 
 namespace plz {
@@ -22,7 +23,8 @@ struct LutGemmArgs {
     // col_scale bf16 [K] and row_scale fp32 [M] are the RMSNorm factors (either may be null)
     int fuse; const void* packed2; const void* palette2; const void* col_scale; const float* row_scale;
     void* gate_out; void* up_out; long long ld_gu;  // fuse == 1: optional bf16 copies of the two pre-activations
-    const void* bias;  // fuse == 2: optional bf16 [J], added in fp32 before the bf16 store
+    const void* bias;  // fuse == 2 or 3: optional bf16 [J], added in fp32 before the bf16 store
+    int act;           // fuse == 3 (dense B, no LoRA block): 1 = square of relu after the bias
     int sm_limit;  // > 0: use at most this many CTAs (tests of the multi-tile schedule)
     void* prof;  // optional device buffer of cycle counters, 8 x uint64 per CTA (diagnostics)
 };
@@ -160,6 +162,34 @@ int launch_qknorm_rope(int backward, const void* x, long long ldx, const void* w
 int launch_swiglu_fwd(const void* gate, long long ldg, const void* up, long long ldu, int M, int N, void* act, long long lda, cudaStream_t stream);
 int launch_add(const void* a, long long lda, const void* b, long long ldb, const void* c, long long ldc, int M, int N, void* out, long long ldo,
                cudaStream_t stream);
+
+// ---- seq_linear.cu / seq_ops.cu / seq_recurrent.cu / attention_bias.cu: hybrid decoders ------------------------
+// dtype: 0 = bf16, 1 = fp32 (activations and weights; accumulation and the marked fp32 tensors are fp32 in both)
+int launch_seq_linear(int dtype, const void* x, long long ldx, int M, int K, const void* w, long long ldw, int N, const void* bias, int act,
+                      void* y, long long ldy, int y_f32, cudaStream_t stream);
+int launch_seq_embed(int dtype, const void* table, long long ldt, const long long* ids, long long rows, int W, long long vocab, float scale,
+                     float* x, void* xb, int* bad, cudaStream_t stream);
+int launch_seq_residual_norm(int dtype, const void* y, long long ldy, const float* w, float w_offset, float mult, float eps, long long rows, int W,
+                             float* x, void* xb, cudaStream_t stream);
+int launch_seq_rows_norm(int dtype, const float* x, const long long* idx, const float* w, float w_offset, float eps, long long rows, int W, void* out,
+                         cudaStream_t stream);
+int launch_seq_norm_gate(int dtype, const float* o, const void* gate, long long ldg, const float* w, float eps, long long rows, int groups, int L,
+                         void* out, cudaStream_t stream);
+using DeltaPrepArgs = plz_delta_prep_t;
+int launch_delta_prep(int dtype, const DeltaPrepArgs& a, cudaStream_t stream);
+using DeltaRuleArgs = plz_delta_rule_t;
+int launch_recurrent_delta(const DeltaRuleArgs& a, cudaStream_t stream);
+using DecayAttnArgs = plz_decay_attn_t;
+int launch_recurrent_decay(int dtype, const DecayAttnArgs& a, cudaStream_t stream);
+using AttnPrepArgs = plz_attn_prep_t;
+int launch_attn_prep(int dtype, const AttnPrepArgs& a, cudaStream_t stream);
+using AttnBiasArgs = plz_attn_bias_t;
+long long attn_bias_decode_ws_bytes(int B, int H, int G, int dv, int cap);
+int launch_attn_bias_decode(int dtype, const AttnBiasArgs& a, int cap, void* ws, long long ws_bytes, cudaStream_t stream);
+int launch_attn_bias_simt(int dtype, const AttnBiasArgs& a, cudaStream_t stream);
+int launch_advance(int* pos, int n, cudaStream_t stream);
+int launch_sample(const float* logits, long long ld, int rows, int V, float temperature, int top_k, uint32_t seed, const int* pos, long long* out,
+                  cudaStream_t stream);
 
 // ---- train_ops.cu ------------------------------------------------------------------------------
 struct AdamParams {

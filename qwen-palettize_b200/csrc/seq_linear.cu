@@ -1,0 +1,203 @@
+// Dense Linear y = act(x W^T + b) for the hybrid decoders, weights bf16 or fp32 [N, K] row-major.
+//
+//   linear_rows_kernel   a handful of rows (token decode): bound by streaming W once. KS warps of a block share the reduction of
+//                        two output rows, chosen so that the launch has enough loads in flight whatever N is; the first
+//                        weights are requested before the wait on the previous kernel of the stream.
+//   linear_tile_kernel   any shape and both types on the CUDA cores, fp32 products and sums: the 32-bit mode, and bf16 shapes
+//                        that the tensor-core path's 16-byte rows exclude.
+//   launch_seq_linear    picks one of them or the tcgen05 GEMM (lut_gemm.cu, dense B, bias and activation in its epilogue).
+#include "seq_math.cuh"
+
+namespace plz {
+namespace {
+
+struct LinParams {
+    const void* x; long long ldx;
+    const void* w; long long ldw;
+    const void* bias;
+    void* y; long long ldy;
+    int M, N, K, act;
+};
+
+template <typename T> struct Raw8;
+template <> struct Raw8<__nv_bfloat16> {
+    uint4 r;
+    __device__ __forceinline__ void load(const __nv_bfloat16* p) { r = __ldg(reinterpret_cast<const uint4*>(p)); }
+    __device__ __forceinline__ void zero() { r = make_uint4(0u, 0u, 0u, 0u); }
+    __device__ __forceinline__ void unpack(float (&f)[8]) const {
+        const uint32_t w[4] = {r.x, r.y, r.z, r.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i) { f[2 * i] = __uint_as_float(w[i] << 16); f[2 * i + 1] = __uint_as_float(w[i] & 0xFFFF0000u); }
+    }
+};
+template <> struct Raw8<float> {
+    float4 a, b;
+    __device__ __forceinline__ void load(const float* p) { a = __ldg(reinterpret_cast<const float4*>(p)); b = __ldg(reinterpret_cast<const float4*>(p + 4)); }
+    __device__ __forceinline__ void zero() { a = make_float4(0.f, 0.f, 0.f, 0.f); b = a; }
+    __device__ __forceinline__ void unpack(float (&f)[8]) const {
+        f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+    }
+};
+
+constexpr int kRowsBatch = 4;   // 8-element chunks of a weight row in flight per lane and row
+
+// K % 8 == 0 and 16-byte aligned rows. Block = 8 warps = 8 / KS pairs of output rows.
+template <typename T, typename TO, int MR>
+__global__ void __launch_bounds__(256)
+linear_rows_kernel(const LinParams p, int ks) {
+    __shared__ float part[8][2][MR];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int pairs = 8 / ks, pair = warp / ks, kw = warp % ks;
+    const int n0 = ((int)blockIdx.x * pairs + pair) * 2;
+    const int chunks = p.K >> 3, step = 32 * ks;
+    const bool has0 = n0 < p.N, has1 = n0 + 1 < p.N;
+    const T* w0 = (const T*)p.w + (long long)n0 * p.ldw;
+    const T* w1 = w0 + p.ldw;
+    Raw8<T> a[kRowsBatch], b[kRowsBatch];
+    auto fetch = [&](int c) {
+#pragma unroll
+        for (int i = 0; i < kRowsBatch; ++i) {
+            const int cc = c + i * step;
+            if (has0 && cc < chunks) a[i].load(w0 + cc * 8); else a[i].zero();
+            if (has1 && cc < chunks) b[i].load(w1 + cc * 8); else b[i].zero();
+        }
+    };
+    int c = kw * 32 + lane;
+    fetch(c);                          // weights do not depend on the previous kernel
+    pdl_launch_dependents();
+    pdl_wait();
+    float s0[MR], s1[MR];
+#pragma unroll
+    for (int m = 0; m < MR; ++m) { s0[m] = 0.f; s1[m] = 0.f; }
+    while (c < chunks) {
+#pragma unroll
+        for (int i = 0; i < kRowsBatch; ++i) {
+            const int cc = c + i * step;
+            if (cc < chunks) {
+                float f0[8], f1[8];
+                a[i].unpack(f0); b[i].unpack(f1);
+#pragma unroll
+                for (int m = 0; m < MR; ++m) {
+                    if (m < p.M) {
+                        float xv[8];
+                        load8((const T*)p.x + (long long)m * p.ldx + cc * 8, xv);
+#pragma unroll
+                        for (int e = 0; e < 8; ++e) { s0[m] = fmaf(f0[e], xv[e], s0[m]); s1[m] = fmaf(f1[e], xv[e], s1[m]); }
+                    }
+                }
+            }
+        }
+        c += kRowsBatch * step;
+        if (c < chunks) fetch(c);
+    }
+#pragma unroll
+    for (int m = 0; m < MR; ++m) {
+        const float t0 = warp_sum(s0[m]), t1 = warp_sum(s1[m]);
+        if (lane == 0) { part[warp][0][m] = t0; part[warp][1][m] = t1; }
+    }
+    __syncthreads();
+    if (kw == 0 && lane < 2 * MR) {
+        const int r = lane / MR, m = lane % MR;
+        if (m < p.M && n0 + r < p.N) {
+            float v = 0.f;
+            for (int i = 0; i < ks; ++i) v += part[warp + i][r][m];
+            if (p.bias) v += to_f(((const T*)p.bias)[n0 + r]);
+            ((TO*)p.y)[(long long)m * p.ldy + n0 + r] = from_f<TO>(activate(v, p.act));
+        }
+    }
+}
+
+template <typename T, typename TO>
+__global__ void __launch_bounds__(256)
+linear_tile_kernel(const LinParams p) {
+    __shared__ float sx[16][64 + 4], sw[16][64 + 4];
+    const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
+    const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
+    pdl_launch_dependents();
+    pdl_wait();
+    float acc[4][4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+    for (int k0 = 0; k0 < p.K; k0 += 16) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int e = tid + i * 256, r = e >> 4, kk = e & 15, k = k0 + kk;
+            sx[kk][r] = (m0 + r < p.M && k < p.K) ? to_f(((const T*)p.x)[(long long)(m0 + r) * p.ldx + k]) : 0.f;
+            sw[kk][r] = (n0 + r < p.N && k < p.K) ? to_f(((const T*)p.w)[(long long)(n0 + r) * p.ldw + k]) : 0.f;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int kk = 0; kk < 16; ++kk) {
+            float a[4], b[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) { a[i] = sx[kk][ty * 4 + i]; b[i] = sw[kk][tx * 4 + i]; }
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int m = m0 + ty * 4 + i;
+        if (m >= p.M) continue;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const int n = n0 + tx * 4 + j;
+            if (n >= p.N) continue;
+            float v = acc[i][j];
+            if (p.bias) v += to_f(((const T*)p.bias)[n]);
+            ((TO*)p.y)[(long long)m * p.ldy + n] = from_f<TO>(activate(v, p.act));
+        }
+    }
+}
+
+template <typename T, typename TO>
+int launch_rows(const LinParams& p, cudaStream_t stream) {
+    const int groups = (p.N + 1) / 2, chunks = p.K >> 3;
+    int ks = 1;   // more warps per row pair until the launch has about 24 warps per SM or a warp has less than one batch of loads
+    while (ks < 8 && (long long)groups * ks < 24ll * seq_sm_count() && chunks > 32 * ks) ks *= 2;
+    const dim3 grid((groups + 8 / ks - 1) / (8 / ks));
+    if (p.M == 1) PLZ_LAUNCH_CHAIN((linear_rows_kernel<T, TO, 1>), grid, dim3(256), 0, stream, p, ks);
+    else if (p.M <= 4) PLZ_LAUNCH_CHAIN((linear_rows_kernel<T, TO, 4>), grid, dim3(256), 0, stream, p, ks);
+    else PLZ_LAUNCH_CHAIN((linear_rows_kernel<T, TO, 8>), grid, dim3(256), 0, stream, p, ks);
+    return PLZ_OK;
+}
+template <typename T, typename TO>
+int launch_tile(const LinParams& p, cudaStream_t stream) {
+    const long long my = (p.M + 63) / 64;
+    if (my > 65535) { set_last_error("linear: too many rows"); return PLZ_ERR_TOO_LARGE; }
+    PLZ_LAUNCH_CHAIN((linear_tile_kernel<T, TO>), dim3((p.N + 63) / 64, (unsigned)my), dim3(256), 0, stream, p);
+    return PLZ_OK;
+}
+
+}  // namespace
+
+int launch_seq_linear(int dtype, const void* x, long long ldx, int M, int K, const void* w, long long ldw, int N, const void* bias, int act,
+                      void* y, long long ldy, int y_f32, cudaStream_t stream) {
+    if (M <= 0) return PLZ_OK;
+    if (N <= 0 || K <= 0 || act < 0 || act > 1) { set_last_error("linear: bad shape M=%d N=%d K=%d act=%d", M, N, K, act); return PLZ_ERR_BAD_SHAPE; }
+    if (!x || !w || !y) { set_last_error("linear: null pointer"); return PLZ_ERR_NULL; }
+    const LinParams p = {x, ldx, w, ldw, bias, y, ldy, M, N, K, act};
+    const int per16 = dtype == 0 ? 8 : 4;
+    const bool vec = K % 8 == 0 && ldx % per16 == 0 && ldw % per16 == 0 && !((uintptr_t)x & 15) && !((uintptr_t)w & 15);
+    if (M <= 8 && vec) {
+        if (dtype == 1) return launch_rows<float, float>(p, stream);
+        return y_f32 ? launch_rows<__nv_bfloat16, float>(p, stream) : launch_rows<__nv_bfloat16, __nv_bfloat16>(p, stream);
+    }
+    if (dtype == 0 && !y_f32 && vec && N % 8 == 0 && ldy % 8 == 0 && !((uintptr_t)y & 15) && !((uintptr_t)bias & 15)) {
+        LutGemmArgs g = {};
+        g.bmode = B_TMA_K; g.M = M; g.J = N; g.R = K;
+        g.A = x; g.lda = ldx; g.Bdense = w; g.ldb = ldw;
+        g.bias = bias; g.act = act; g.fuse = (bias || act) ? 3 : 0;
+        g.out = y; g.ld_out = ldy; g.alpha = 1.0f;
+        return launch_lut_gemm(g, stream);
+    }
+    if (dtype == 1) return launch_tile<float, float>(p, stream);
+    return y_f32 ? launch_tile<__nv_bfloat16, float>(p, stream) : launch_tile<__nv_bfloat16, __nv_bfloat16>(p, stream);
+}
+
+}  // namespace plz

@@ -1,0 +1,425 @@
+// Row-wise steps of the hybrid decoders around their Linears, recurrences and attention: embedding with a scale, the norm on a
+// sublayer's output fused with the fp32 residual update, the norm + gate that closes a recurrent mixer, the short causal
+// convolution with its activation, unit norm and decay, the query / key norm that feeds the cache, and token sampling.
+//
+// Rows are b * n + t: B sequences advance in lockstep by n tokens each; *pos (device memory, so that a captured step can be
+// replayed at later positions) is the position of the first of them. The residual stream, statistics, decays and gates are fp32.
+#include "seq_math.cuh"
+
+namespace plz {
+namespace {
+
+// x[r, :] = table[ids[r], :] * scale (fp32), xb the same in T (bf16 models: the operand of the first Linear)
+template <typename T>
+__global__ void __launch_bounds__(256)
+embed_scale_kernel(const T* __restrict__ table, long long ldt, const long long* __restrict__ ids, int W, long long vocab, float scale,
+                   float* __restrict__ x, T* __restrict__ xb, int* __restrict__ bad) {
+    const long long r = blockIdx.x;
+    pdl_launch_dependents();
+    pdl_wait();
+    const long long id = ids[r];
+    const bool ok = id >= 0 && id < vocab;
+    if (!ok && bad && threadIdx.x == 0) *bad = 1;
+    for (int c = threadIdx.x; c < W; c += 256) {
+        const float v = ok ? to_f(table[id * ldt + c]) * scale : 0.f;
+        x[r * W + c] = v;
+        if (xb) xb[r * W + c] = from_f<T>(v);
+    }
+}
+
+// x += mult * y / rms(y) * (w + w_offset); xb = T(x)
+template <typename T>
+__global__ void __launch_bounds__(256)
+residual_norm_kernel(const T* __restrict__ y, long long ldy, const float* __restrict__ w, float w_offset, float mult, float eps, int W,
+                     float* __restrict__ x, T* __restrict__ xb) {
+    __shared__ float part[8];
+    const long long r = blockIdx.x;
+    pdl_launch_dependents();
+    pdl_wait();
+    const T* yr = y + r * ldy;
+    float s = 0.f;
+    for (int c = threadIdx.x; c < W; c += 256) { const float v = to_f(yr[c]); s = fmaf(v, v, s); }
+    s = block_sum<8>(s, part);
+    const float rs = 1.0f / sqrtf(s / (float)W + eps);
+    for (int c = threadIdx.x; c < W; c += 256) {
+        const float v = x[r * W + c] + mult * (to_f(yr[c]) * rs * (w[c] + w_offset));
+        x[r * W + c] = v;
+        if (xb) xb[r * W + c] = from_f<T>(v);
+    }
+}
+// the same for W % 4 == 0 and 16-byte aligned rows, four columns per access, y kept in registers (W <= 4096)
+template <typename T> struct Quad { T v[4]; };
+template <typename T>
+__global__ void __launch_bounds__(256)
+residual_norm4_kernel(const T* __restrict__ y, long long ldy, const float* __restrict__ w, float w_offset, float mult, float eps, int W,
+                      float* __restrict__ x, T* __restrict__ xb) {
+    __shared__ float part[8];
+    const long long r = blockIdx.x;
+    const int n4 = W >> 2;
+    pdl_launch_dependents();
+    pdl_wait();
+    const T* yr = y + r * ldy;
+    float f[4][4];
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int c = threadIdx.x + i * 256;
+        if (c < n4) {
+            if (sizeof(T) == 2) {
+                const uint2 q = *reinterpret_cast<const uint2*>(yr + c * 4);
+                f[i][0] = __uint_as_float(q.x << 16); f[i][1] = __uint_as_float(q.x & 0xFFFF0000u);
+                f[i][2] = __uint_as_float(q.y << 16); f[i][3] = __uint_as_float(q.y & 0xFFFF0000u);
+            } else {
+                const float4 q = *reinterpret_cast<const float4*>(yr + c * 4);
+                f[i][0] = q.x; f[i][1] = q.y; f[i][2] = q.z; f[i][3] = q.w;
+            }
+#pragma unroll
+            for (int e = 0; e < 4; ++e) s = fmaf(f[i][e], f[i][e], s);
+        }
+    }
+    s = block_sum<8>(s, part);
+    const float rs = 1.0f / sqrtf(s / (float)W + eps);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int c = threadIdx.x + i * 256;
+        if (c < n4) {
+            float4 a = *reinterpret_cast<const float4*>(x + r * W + c * 4);
+            const float4 g = __ldg(reinterpret_cast<const float4*>(w + c * 4));
+            a.x += mult * (f[i][0] * rs * (g.x + w_offset)); a.y += mult * (f[i][1] * rs * (g.y + w_offset));
+            a.z += mult * (f[i][2] * rs * (g.z + w_offset)); a.w += mult * (f[i][3] * rs * (g.w + w_offset));
+            *reinterpret_cast<float4*>(x + r * W + c * 4) = a;
+            if (xb) {
+                if (sizeof(T) == 2) *reinterpret_cast<uint2*>(xb + r * W + c * 4) = make_uint2(pack_bf16x2(a.x, a.y), pack_bf16x2(a.z, a.w));
+                else *reinterpret_cast<float4*>(xb + r * W + c * 4) = a;
+            }
+        }
+    }
+}
+
+// out[i, :] = x[idx[i], :] / rms * (w + w_offset) in T (idx null: row i)
+template <typename T>
+__global__ void __launch_bounds__(256)
+rows_norm_kernel(const float* __restrict__ x, const long long* __restrict__ idx, const float* __restrict__ w, float w_offset, float eps, int W,
+                 T* __restrict__ out) {
+    __shared__ float part[8];
+    pdl_launch_dependents();
+    pdl_wait();
+    const long long i = blockIdx.x, r = idx ? idx[i] : i;
+    float s = 0.f;
+    for (int c = threadIdx.x; c < W; c += 256) { const float v = x[r * W + c]; s = fmaf(v, v, s); }
+    s = block_sum<8>(s, part);
+    const float rs = 1.0f / sqrtf(s / (float)W + eps);
+    for (int c = threadIdx.x; c < W; c += 256) out[i * W + c] = from_f<T>(x[r * W + c] * rs * (w[c] + w_offset));
+}
+
+// out[r, g * L + c] = o / rms(o over the L values of the group) * w[c] * sigmoid(gate); a block per (row, several groups), a warp
+// per group when L is small, the whole block otherwise
+template <typename T, bool BLOCK>
+__global__ void __launch_bounds__(256)
+norm_gate_kernel(const float* __restrict__ o, const T* __restrict__ gate, long long ldg, const float* __restrict__ w, float eps, int groups, int L,
+                 T* __restrict__ out) {
+    __shared__ float part[8];
+    const long long r = blockIdx.x;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int g = BLOCK ? (int)blockIdx.y : (int)blockIdx.y * 8 + warp;
+    const int t = BLOCK ? (int)threadIdx.x : lane, team = BLOCK ? 256 : 32;
+    pdl_launch_dependents();
+    pdl_wait();
+    if (!BLOCK && g >= groups) return;
+    const long long W = (long long)groups * L;
+    const float* og = o + r * W + (long long)g * L;
+    const T* gg = gate + r * ldg + (long long)g * L;
+    float s = 0.f;
+    for (int c = t; c < L; c += team) s = fmaf(og[c], og[c], s);
+    s = BLOCK ? block_sum<8>(s, part) : warp_sum(s);
+    const float rs = 1.0f / sqrtf(s / (float)L + eps);
+    T* dst = out + r * W + (long long)g * L;
+    for (int c = t; c < L; c += team) dst[c] = from_f<T>(og[c] * rs * w[c] * sigmoid_f(to_f(gg[c])));
+}
+
+// ---- gated delta rule: everything between the projections and the recurrence ------------------------------------------
+struct DeltaPrep {
+    const void* proj; long long ldp; int off_q, off_k, off_v, off_b;   // raw projections of this step
+    const void* a; long long lda;                                      // decay pre-activation [rows, H * dk]
+    const float* taps;                                                 // [channels, n_taps], channels = q | k | v
+    const float* A_log; const float* dt_bias;                          // [H], [H * dk]
+    void* conv; int n_taps;                                            // [B, n_taps - 1, channels] inputs before this step, oldest first
+    int B, n, H, G, dk, dv;
+    float q_scale;
+    float* q; float* k; float* v; float* logg; float* beta;            // [rows, G * dk] x 2, [rows, H * dv], [rows, H * dk], [rows, H]
+    int update;                                                        // n == 1: shift this token into `conv`
+};
+
+// One warp per item of a row: G query heads, G key heads, H value heads, H decay heads (lane 0 of the last also does beta).
+template <typename T>
+__global__ void __launch_bounds__(256)
+delta_prep_kernel(const DeltaPrep p) {
+    const long long r = blockIdx.x;
+    const int lane = threadIdx.x & 31, item = (int)blockIdx.y * 8 + (threadIdx.x >> 5);
+    const int t = (int)(r % p.n);
+    const long long b = r / p.n;
+    pdl_launch_dependents();
+    pdl_wait();
+    if (item >= 2 * p.G + 2 * p.H) return;
+    if (item >= 2 * p.G + p.H) {
+        const int h = item - 2 * p.G - p.H;
+        const float rate = expf(p.A_log[h]);
+        const T* ar = (const T*)p.a + r * p.lda + (long long)h * p.dk;
+        float* gr = p.logg + (r * p.H + h) * p.dk;
+        for (int c = lane; c < p.dk; c += 32) gr[c] = -rate * softplus_f(to_f(ar[c]) + p.dt_bias[h * p.dk + c]);
+        if (lane == 0) p.beta[r * p.H + h] = sigmoid_f(to_f(((const T*)p.proj)[r * p.ldp + p.off_b + h]));
+        return;
+    }
+    const int kind = item < p.G ? 0 : (item < 2 * p.G ? 1 : 2);
+    const int head = kind == 0 ? item : (kind == 1 ? item - p.G : item - 2 * p.G);
+    const int L = kind == 2 ? p.dv : p.dk;
+    const int off = (kind == 0 ? p.off_q : (kind == 1 ? p.off_k : p.off_v)) + head * L;       // column of the projection
+    const int ch0 = (kind == 0 ? 0 : (kind == 1 ? p.G * p.dk : 2 * p.G * p.dk)) + head * L;   // convolution channel
+    const int C = 2 * p.G * p.dk + p.H * p.dv, keep = p.n_taps - 1;
+    T* cs = (T*)p.conv + b * (long long)keep * C;
+    float* dst = kind == 0 ? p.q + (r * p.G + head) * p.dk : (kind == 1 ? p.k + (r * p.G + head) * p.dk : p.v + (r * p.H + head) * p.dv);
+    float ss = 0.f;
+    for (int c = lane; c < L; c += 32) {
+        const float* w = p.taps + (long long)(ch0 + c) * p.n_taps;
+        const T cur = ((const T*)p.proj)[r * p.ldp + off + c];
+        float s = 0.f;
+        for (int j = 0; j < keep; ++j) {             // tap j looks back keep - j tokens
+            const int tt = t - (keep - j);
+            const T in = tt >= 0 ? ((const T*)p.proj)[(r - (keep - j)) * p.ldp + off + c] : cs[(long long)(tt + keep) * C + ch0 + c];
+            s = fmaf(w[j], to_f(in), s);
+        }
+        s = fmaf(w[keep], to_f(cur), s);
+        if (p.update && keep > 0) {
+            for (int j = 0; j + 1 < keep; ++j) cs[(long long)j * C + ch0 + c] = cs[(long long)(j + 1) * C + ch0 + c];
+            cs[(long long)(keep - 1) * C + ch0 + c] = cur;
+        }
+        s = silu_f(s);
+        dst[c] = s;
+        ss = fmaf(s, s, ss);
+    }
+    if (kind == 2) return;
+    ss = warp_sum(ss);
+    const float f = (kind == 0 ? p.q_scale : 1.0f) / sqrtf(ss + 1e-6f);
+    for (int c = lane; c < L; c += 32) dst[c] *= f;      // this lane's own elements
+}
+
+// the last n_taps - 1 inputs after a portion of n tokens (n >= 1)
+template <typename T>
+__global__ void __launch_bounds__(256)
+conv_state_kernel(const T* __restrict__ proj, long long ldp, int off_q, int off_k, int off_v, int qk, int C, int keep, int n, T* __restrict__ conv) {
+    const long long b = blockIdx.y;
+    const int ch = (int)blockIdx.x * 256 + threadIdx.x;
+    pdl_launch_dependents();
+    pdl_wait();
+    if (ch >= C) return;
+    const int col = ch < qk ? off_q + ch : (ch < 2 * qk ? off_k + ch - qk : off_v + ch - 2 * qk);
+    T* cs = conv + b * (long long)keep * C + ch;
+    for (int j = 0; j < keep; ++j) {             // ascending: a slot is read (as j + n) before it is overwritten
+        const int t = n - keep + j;
+        cs[(long long)j * C] = t >= 0 ? proj[(b * n + t) * ldp + col] : cs[(long long)(j + n) * C];
+    }
+}
+
+// ---- attention: norm over the whole query / key projection, value mixing, cache write ----------------------------------
+struct AttnPrep {
+    const void* proj; long long ldp; int off_q, off_k, off_v;
+    const float* wq; const float* wk;              // [H * dk], [G * dk]
+    const float* mix;                              // [1] or null; v <- (1 - mix) v + mix v_first
+    void* v_first; int v_first_write;              // [rows, G * dv]
+    void* q;                                       // [rows, H * dk]
+    void* kc; void* vc; long long k_batch, v_batch;   // caches [B, T, G * dk], [B, T, G * dv]; elements per sequence
+    const int* pos;
+    int n, qw, kw, vw, cap;
+    float eps;
+};
+template <typename T>
+__global__ void __launch_bounds__(256)
+attn_prep_kernel(const AttnPrep p) {
+    __shared__ float part[8];
+    const long long r = blockIdx.x, b = r / p.n;
+    pdl_launch_dependents();
+    pdl_wait();
+    const int at = *p.pos + (int)(r % p.n);
+    if (at >= p.cap) return;                       // the host checks the capacity; never write past it
+    const T* row = (const T*)p.proj + r * p.ldp;
+    float sq = 0.f, sk = 0.f;
+    for (int c = threadIdx.x; c < p.qw; c += 256) { const float v = to_f(row[p.off_q + c]); sq = fmaf(v, v, sq); }
+    for (int c = threadIdx.x; c < p.kw; c += 256) { const float v = to_f(row[p.off_k + c]); sk = fmaf(v, v, sk); }
+    sq = block_sum<8>(sq, part);
+    sk = block_sum<8>(sk, part);
+    const float rq = 1.0f / sqrtf(sq / (float)p.qw + p.eps), rk = 1.0f / sqrtf(sk / (float)p.kw + p.eps);
+    T* qo = (T*)p.q + r * p.qw;
+    T* ko = (T*)p.kc + b * p.k_batch + (long long)at * p.kw;
+    T* vo = (T*)p.vc + b * p.v_batch + (long long)at * p.vw;
+    for (int c = threadIdx.x; c < p.qw; c += 256) qo[c] = from_f<T>(to_f(row[p.off_q + c]) * rq * p.wq[c]);
+    for (int c = threadIdx.x; c < p.kw; c += 256) ko[c] = from_f<T>(to_f(row[p.off_k + c]) * rk * p.wk[c]);
+    const float lam = p.mix ? *p.mix : 0.f;
+    T* vf = (T*)p.v_first + (p.v_first ? r * p.vw : 0);
+    for (int c = threadIdx.x; c < p.vw; c += 256) {
+        T v = row[p.off_v + c];
+        if (p.v_first_write) vf[c] = v;
+        if (p.mix) v = from_f<T>((1.0f - lam) * to_f(v) + lam * to_f(vf[c]));
+        vo[c] = v;
+    }
+}
+
+__global__ void advance_kernel(int* pos, int n) {
+    pdl_wait();
+    *pos += n;
+}
+
+// ---- sampling: one block per row ------------------------------------------------------------------------------------------
+// temperature == 0: index of the largest logit, the first of equals. Else the largest of logit / temperature + Gumbel noise
+// among the top_k logits (top_k <= 0: all), the noise from a counter hash of (seed, *pos, row, index).
+__device__ __forceinline__ uint32_t mix32(uint32_t h) {
+    h ^= h >> 16; h *= 0x85EBCA6Bu; h ^= h >> 13; h *= 0xC2B2AE35u; h ^= h >> 16;
+    return h;
+}
+__global__ void __launch_bounds__(256)
+sample_kernel(const float* __restrict__ logits, long long ld, int V, float temperature, int top_k, uint32_t seed, const int* __restrict__ pos,
+              long long* __restrict__ out) {
+    __shared__ float sv[8];
+    __shared__ int si[8];
+    __shared__ int cnt;
+    const int row = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    pdl_launch_dependents();
+    pdl_wait();
+    const float* lr = logits + (long long)row * ld;
+    uint32_t floor_key = 0;              // smallest admitted key
+    auto key_of = [](float v) { const uint32_t u = __float_as_uint(v); return (u & 0x80000000u) ? ~u : (u | 0x80000000u); };
+    if (temperature > 0.f && top_k > 0 && top_k < V) {
+        // largest key that at least top_k logits reach, bit by bit
+        for (int bit = 31; bit >= 0; --bit) {
+            const uint32_t trial = floor_key | (1u << bit);
+            if (threadIdx.x == 0) cnt = 0;
+            __syncthreads();
+            int c = 0;
+            for (int i = threadIdx.x; i < V; i += 256) c += key_of(lr[i]) >= trial;
+            c = __reduce_add_sync(0xFFFFFFFFu, c);
+            if (lane == 0) atomicAdd(&cnt, c);
+            __syncthreads();
+            if (cnt >= top_k) floor_key = trial;
+            __syncthreads();
+        }
+    }
+    const uint32_t base = mix32(seed ^ mix32((uint32_t)*pos * 0x9E3779B1u + (uint32_t)row));
+    float best = -INFINITY;
+    int bi = V;
+    for (int i = threadIdx.x; i < V; i += 256) {
+        float v = lr[i];
+        if (temperature > 0.f) {
+            if (key_of(v) < floor_key) continue;
+            const float u = ((float)(mix32(base ^ mix32((uint32_t)i + 0x7F4A7C15u)) >> 8) + 0.5f) * (1.0f / 16777216.0f);
+            v = v / temperature - logf(-logf(u));
+        }
+        if (v > best || bi == V) { best = v; bi = i; }
+    }
+    for (int o = 16; o > 0; o >>= 1) {
+        const float ov = __shfl_xor_sync(0xFFFFFFFFu, best, o);
+        const int oi = __shfl_xor_sync(0xFFFFFFFFu, bi, o);
+        if (oi < V && (bi == V || ov > best || (ov == best && oi < bi))) { best = ov; bi = oi; }
+    }
+    if (lane == 0) { sv[warp] = best; si[warp] = bi; }
+    __syncthreads();
+    if (threadIdx.x == 0) {
+        for (int w = 1; w < 8; ++w)
+            if (si[w] < V && (bi == V || sv[w] > best || (sv[w] == best && si[w] < bi))) { best = sv[w]; bi = si[w]; }
+        out[row] = bi < V ? bi : 0;
+    }
+}
+
+typedef __nv_bfloat16 bf;
+
+}  // namespace
+
+int launch_seq_embed(int dtype, const void* table, long long ldt, const long long* ids, long long rows, int W, long long vocab, float scale,
+                     float* x, void* xb, int* bad, cudaStream_t stream) {
+    if (rows <= 0) return PLZ_OK;
+    if (dtype == 1) PLZ_LAUNCH_CHAIN(embed_scale_kernel<float>, dim3((unsigned)rows), dim3(256), 0, stream, (const float*)table, ldt, ids, W, vocab, scale, x, (float*)xb, bad);
+    else PLZ_LAUNCH_CHAIN(embed_scale_kernel<bf>, dim3((unsigned)rows), dim3(256), 0, stream, (const bf*)table, ldt, ids, W, vocab, scale, x, (bf*)xb, bad);
+    return PLZ_OK;
+}
+
+template <typename T>
+static int residual_norm_t(const T* y, long long ldy, const float* w, float off, float mult, float eps, long long rows, int W, float* x, T* xb, cudaStream_t s) {
+    const bool vec = W % 4 == 0 && W <= 4096 && ldy % 4 == 0 && !((uintptr_t)y & 15) && !((uintptr_t)x & 15) && !((uintptr_t)w & 15) && !((uintptr_t)xb & 15);
+    if (vec) PLZ_LAUNCH_CHAIN(residual_norm4_kernel<T>, dim3((unsigned)rows), dim3(256), 0, s, y, ldy, w, off, mult, eps, W, x, xb);
+    else PLZ_LAUNCH_CHAIN(residual_norm_kernel<T>, dim3((unsigned)rows), dim3(256), 0, s, y, ldy, w, off, mult, eps, W, x, xb);
+    return PLZ_OK;
+}
+int launch_seq_residual_norm(int dtype, const void* y, long long ldy, const float* w, float w_offset, float mult, float eps, long long rows, int W,
+                             float* x, void* xb, cudaStream_t stream) {
+    if (rows <= 0) return PLZ_OK;
+    if (dtype == 1) return residual_norm_t<float>((const float*)y, ldy, w, w_offset, mult, eps, rows, W, x, (float*)xb, stream);
+    return residual_norm_t<bf>((const bf*)y, ldy, w, w_offset, mult, eps, rows, W, x, (bf*)xb, stream);
+}
+
+int launch_seq_rows_norm(int dtype, const float* x, const long long* idx, const float* w, float w_offset, float eps, long long rows, int W, void* out,
+                         cudaStream_t stream) {
+    if (rows <= 0) return PLZ_OK;
+    if (dtype == 1) PLZ_LAUNCH_CHAIN(rows_norm_kernel<float>, dim3((unsigned)rows), dim3(256), 0, stream, x, idx, w, w_offset, eps, W, (float*)out);
+    else PLZ_LAUNCH_CHAIN(rows_norm_kernel<bf>, dim3((unsigned)rows), dim3(256), 0, stream, x, idx, w, w_offset, eps, W, (bf*)out);
+    return PLZ_OK;
+}
+
+int launch_seq_norm_gate(int dtype, const float* o, const void* gate, long long ldg, const float* w, float eps, long long rows, int groups, int L,
+                         void* out, cudaStream_t stream) {
+    if (rows <= 0) return PLZ_OK;
+    const bool block = L > 256;
+    const dim3 grid((unsigned)rows, block ? groups : (groups + 7) / 8);
+    if (dtype == 1) {
+        if (block) PLZ_LAUNCH_CHAIN((norm_gate_kernel<float, true>), grid, dim3(256), 0, stream, o, (const float*)gate, ldg, w, eps, groups, L, (float*)out);
+        else PLZ_LAUNCH_CHAIN((norm_gate_kernel<float, false>), grid, dim3(256), 0, stream, o, (const float*)gate, ldg, w, eps, groups, L, (float*)out);
+    } else {
+        if (block) PLZ_LAUNCH_CHAIN((norm_gate_kernel<bf, true>), grid, dim3(256), 0, stream, o, (const bf*)gate, ldg, w, eps, groups, L, (bf*)out);
+        else PLZ_LAUNCH_CHAIN((norm_gate_kernel<bf, false>), grid, dim3(256), 0, stream, o, (const bf*)gate, ldg, w, eps, groups, L, (bf*)out);
+    }
+    return PLZ_OK;
+}
+
+int launch_delta_prep(int dtype, const DeltaPrepArgs& a, cudaStream_t stream) {
+    const long long rows = (long long)a.B * a.n;
+    if (rows <= 0) return PLZ_OK;
+    DeltaPrep p;
+    p.proj = a.proj; p.ldp = a.ldp; p.off_q = a.off_q; p.off_k = a.off_k; p.off_v = a.off_v; p.off_b = a.off_b; p.a = a.a; p.lda = a.lda;
+    p.taps = a.taps; p.A_log = a.A_log; p.dt_bias = a.dt_bias; p.conv = a.conv; p.n_taps = a.n_taps;
+    p.B = a.B; p.n = a.n; p.H = a.H; p.G = a.G; p.dk = a.dk; p.dv = a.dv; p.q_scale = a.q_scale;
+    p.q = a.q; p.k = a.k; p.v = a.v; p.logg = a.logg; p.beta = a.beta;
+    p.update = a.n == 1;
+    const dim3 grid((unsigned)rows, (2 * a.G + 2 * a.H + 7) / 8);
+    if (dtype == 1) PLZ_LAUNCH_CHAIN(delta_prep_kernel<float>, grid, dim3(256), 0, stream, p);
+    else PLZ_LAUNCH_CHAIN(delta_prep_kernel<bf>, grid, dim3(256), 0, stream, p);
+    if (a.n > 1 && a.n_taps > 1) {
+        const int qk = a.G * a.dk, C = 2 * qk + a.H * a.dv;
+        const dim3 g2((C + 255) / 256, a.B);
+        if (dtype == 1) PLZ_LAUNCH_CHAIN(conv_state_kernel<float>, g2, dim3(256), 0, stream, (const float*)a.proj, a.ldp, a.off_q, a.off_k, a.off_v, qk, C, a.n_taps - 1, a.n, (float*)a.conv);
+        else PLZ_LAUNCH_CHAIN(conv_state_kernel<bf>, g2, dim3(256), 0, stream, (const bf*)a.proj, a.ldp, a.off_q, a.off_k, a.off_v, qk, C, a.n_taps - 1, a.n, (bf*)a.conv);
+    }
+    return PLZ_OK;
+}
+
+int launch_attn_prep(int dtype, const AttnPrepArgs& a, cudaStream_t stream) {
+    const long long rows = (long long)a.B * a.n;
+    if (rows <= 0) return PLZ_OK;
+    AttnPrep p;
+    p.proj = a.proj; p.ldp = a.ldp; p.off_q = a.off_q; p.off_k = a.off_k; p.off_v = a.off_v; p.wq = a.wq; p.wk = a.wk; p.mix = a.mix;
+    p.v_first = a.v_first; p.v_first_write = a.v_first_write; p.q = a.q; p.kc = a.kc; p.vc = a.vc; p.k_batch = a.k_batch; p.v_batch = a.v_batch;
+    p.pos = a.pos; p.n = a.n; p.qw = a.qw; p.kw = a.kw; p.vw = a.vw; p.cap = a.cap; p.eps = a.eps;
+    if (dtype == 1) PLZ_LAUNCH_CHAIN(attn_prep_kernel<float>, dim3((unsigned)rows), dim3(256), 0, stream, p);
+    else PLZ_LAUNCH_CHAIN(attn_prep_kernel<bf>, dim3((unsigned)rows), dim3(256), 0, stream, p);
+    return PLZ_OK;
+}
+
+int launch_advance(int* pos, int n, cudaStream_t stream) {
+    PLZ_LAUNCH_CHAIN(advance_kernel, dim3(1), dim3(1), 0, stream, pos, n);
+    return PLZ_OK;
+}
+
+int launch_sample(const float* logits, long long ld, int rows, int V, float temperature, int top_k, uint32_t seed, const int* pos, long long* out,
+                  cudaStream_t stream) {
+    if (rows <= 0) return PLZ_OK;
+    PLZ_LAUNCH_CHAIN(sample_kernel, dim3(rows), dim3(256), 0, stream, logits, ld, V, temperature, top_k, seed, pos, out);
+    return PLZ_OK;
+}
+
+}  // namespace plz

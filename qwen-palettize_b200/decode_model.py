@@ -41,6 +41,14 @@ class KVCache:
     v: torch.Tensor
     length: int = 0      # positions filled
 
+    @property
+    def capacity(self) -> int:
+        return self.k.shape[2]
+
+    def reset(self):
+        """Start over: positions at and beyond the length are never read, so nothing needs clearing."""
+        self.length = 0
+
 
 class PalettizedQwen:
     def __init__(self, cfg: ModelConfig, layers, embed: torch.Tensor, final_norm: torch.Tensor, max_positions: int = 4096):
@@ -69,6 +77,58 @@ class PalettizedQwen:
         embed = (torch.randn(cfg.vocab, cfg.hidden, generator=g, device=device) * 0.02).to(torch.bfloat16)
         fin = (1.0 + 0.1 * torch.randn(cfg.hidden, generator=g, device=device)).to(torch.bfloat16)
         return cls(cfg, layers, embed, fin, max_positions)
+
+    # ---- registry and serving --------------------------------------------------------------------------------------
+    DTYPES = (torch.bfloat16,)
+
+    @property
+    def vocab(self) -> int:
+        return self.cfg.vocab
+
+    @classmethod
+    def from_config(cls, config: dict, tensors, dtype=torch.bfloat16, device="cuda"):
+        """config: the fields of ModelConfig plus 'max_positions'; tensors: 'l<i>.<linear>.packed' / '.palette', the four norms of a layer,
+        'embed' and 'final_norm' (state_dict)."""
+        assert dtype == torch.bfloat16
+        known = {k: v for k, v in config.items() if k in ModelConfig.__dataclass_fields__}
+        cfg = ModelConfig(**known)
+        layers = []
+        for i in range(cfg.n_layers):
+            L = {n: ops.PackedWeight(tensors[f"l{i}.{n}.packed"].to(device), tensors[f"l{i}.{n}.palette"].to(device), N, K, 1, 256)
+                 for n, (N, K) in cfg.shapes().items()}
+            L.update({n: tensors[f"l{i}.{n}"].to(device) for n in ("input_ln", "post_ln", "q_norm", "k_norm")})
+            layers.append(L)
+        return cls(cfg, layers, tensors["embed"].to(device), tensors["final_norm"].to(device), config.get("max_positions", 4096))
+
+    def state_dict(self) -> dict:
+        out = {"embed": self.embed, "final_norm": self.final_norm}
+        for i, L in enumerate(self.layers):
+            for n in LINEARS:
+                out[f"l{i}.{n}.packed"], out[f"l{i}.{n}.palette"] = L[n].packed, L[n].palette
+            out.update({f"l{i}.{n}": L[n] for n in ("input_ln", "post_ln", "q_norm", "k_norm")})
+        return out
+
+    def forward(self, ids: torch.Tensor, cache: KVCache, want=None):
+        """Run ids int64 [B, n] from the state in `cache`; want: rows (b * n + t) whose logits are returned, fp32 [len(want), vocab].
+        A fresh sequence takes its leading multiple of 128 tokens through prefill, the rest goes token by token."""
+        dev = self.embed.device
+        ids = ids.to(dev)
+        B, n = ids.shape
+        if cache.length + n > cache.capacity:
+            raise ValueError(f"{cache.length} + {n} tokens exceed the capacity {cache.capacity} of the state")
+        want = list(want) if want is not None else []
+        rows, head = {}, 0
+        if cache.length == 0 and n >= 128:
+            head = n // 128 * 128
+            h, _ = self.prefill(ids[:, :head].contiguous(), cache, want_logits=False)
+            at = [w for w in want if w % n < head]
+            if at:
+                lg = self.logits(h.view(B, head, -1)[[w // n for w in at], [w % n for w in at]].contiguous()).float()
+                rows.update({w: lg[i] for i, w in enumerate(at)})
+        for t in range(head, n):
+            lg = self.decode_step(ids[:, t].contiguous(), cache)
+            rows.update({b * n + t: lg[b].float() for b in range(B) if b * n + t in want})
+        return torch.stack([rows[w] for w in want]) if want else None
 
     def weight_bytes(self) -> int:
         """Bytes of packed indices and palettes of all layers (what a decode step must read, the embedding table aside)."""

@@ -1,0 +1,196 @@
+"""Token mixers and feed-forwards of the hybrid decoders. Each mixer is built from its configuration entry and the stored tensors of one
+layer, declares the per-sequence state it keeps, and runs a portion of n tokens for B sequences from that state. The kernels are
+sequence-length agnostic, so one code path serves whole prompts, portions of prompts and single tokens.
+
+    MIXERS['lightning']       decayed linear attention, RMS norm over all heads, sigmoid gate
+    MIXERS['channel_delta']   gated delta rule with one decay per head and key channel, short convolutions on q, k, v
+    MIXERS['attention']       softmax attention with a learned bias by distance, a sink, whole-projection q / k norm and value mixing
+    MLPS['dense']             W_down relu(W_up x)^2
+"""
+from __future__ import annotations
+
+import math
+from dataclasses import dataclass
+
+import torch
+
+import seq_ops as S
+
+
+@dataclass
+class StepContext:
+    """What the mixers of one step share."""
+    B: int
+    n: int
+    pos: torch.Tensor              # int32 [1], position of the first token (device)
+    host_pos: int                  # the same on the host; -1 in a step that is captured for replay
+    eps: float
+    v_first: torch.Tensor | None = None    # values of the first mixing layer, [B * n, width]
+
+
+@dataclass
+class StateSpec:
+    """A tensor a layer keeps per sequence: shape without the leading batch; 'T_max' stands for the cache capacity. Tensors that must
+    start at zero are cleared when a sequence starts."""
+    shape: tuple
+    fp32: bool = False
+    zero: bool = False
+
+
+class Loader:
+    """Tensors of one layer by short name, moved to the device in the requested type."""
+
+    def __init__(self, tensors, prefix: str, dtype: torch.dtype, device):
+        self.t, self.prefix, self.dtype, self.device = tensors, prefix, dtype, device
+
+    def has(self, name: str) -> bool:
+        return self.prefix + name in self.t
+
+    def raw(self, name: str, shape=None) -> torch.Tensor:
+        t = self.t[self.prefix + name]
+        if shape is not None and tuple(t.shape) != tuple(shape):
+            raise ValueError(f"tensor {self.prefix + name}: shape {tuple(t.shape)}, expected {tuple(shape)}")
+        return t
+
+    def mat(self, name: str, shape=None) -> torch.Tensor:
+        return self.raw(name, shape).to(self.device, self.dtype).contiguous()
+
+    def f32(self, name: str, shape=None) -> torch.Tensor:
+        return self.raw(name, shape).to(self.device, torch.float32).contiguous()
+
+    def stack(self, names, shapes, biases: bool = False):
+        """The named matrices one under the other, each starting at a multiple of eight rows (zero rows between), so that one Linear
+        serves all of them and every slice of its output starts on 16 bytes. Returns (weight, bias or None, first row of each)."""
+        K = shapes[0][1]
+        offs, at = [], 0
+        for _, (N, _) in zip(names, shapes):
+            offs.append(at)
+            at += (N + 7) // 8 * 8
+        w = torch.zeros(at, K, dtype=self.dtype, device=self.device)
+        b = torch.zeros(at, dtype=self.dtype, device=self.device) if biases else None
+        for name, shape, o in zip(names, shapes, offs):
+            w[o:o + shape[0]] = self.mat(name, shape)
+            if biases:
+                b[o:o + shape[0]] = self.mat(name + ".b", (shape[0],))
+        return w, b, offs
+
+
+class Lightning:
+    """Per head S <- decay S + k v^T, o = S^T q, with q, k, v = silu of their projections."""
+
+    def __init__(self, mc: dict, L: Loader, width: int):
+        self.H, self.dk, self.dv = mc["heads"], mc["dim"], mc["vdim"]
+        if len(mc["decay"]) != self.H:
+            raise ValueError(f"{len(mc['decay'])} decays for {self.H} heads")
+        qk, v = self.H * self.dk, self.H * self.dv
+        self.w_in, _, self.off = L.stack(("q", "k", "v", "g"), ((qk, width), (qk, width), (v, width), (v, width)))
+        self.w_out, self.norm = L.mat("o", (width, v)), L.f32("norm", (v,))
+        self.decay = torch.tensor(mc["decay"], dtype=torch.float32, device=L.device)
+
+    def state_spec(self):
+        return {"S": StateSpec((self.H, self.dk, self.dv), fp32=True, zero=True)}
+
+    def forward(self, x: torch.Tensor, st: dict, ctx: StepContext) -> torch.Tensor:
+        qk, v, (oq, ok, ov, og) = self.H * self.dk, self.H * self.dv, self.off
+        p = S.linear(x, self.w_in)
+        o = S.decay_attention(p[:, oq:oq + qk], p[:, ok:ok + qk], p[:, ov:ov + v], self.decay, st["S"], ctx.B, ctx.n, self.H, self.dk, self.dv)
+        return S.linear(S.norm_gate(o, p[:, og:og + v], self.norm, ctx.eps, 1), self.w_out)
+
+
+class ChannelDelta:
+    """Gated delta rule; the decay is a vector over the key channels of every head."""
+
+    def __init__(self, mc: dict, L: Loader, width: int):
+        self.H, self.G, self.dk, self.dv = mc["heads"], mc["kv_heads"], mc["dim"], mc["vdim"]
+        self.taps = mc["conv"]
+        if self.H % self.G:
+            raise ValueError(f"{self.H} heads over {self.G} key heads")
+        qk, v = self.G * self.dk, self.H * self.dv
+        ra, rg = L.raw("a1").shape[0], L.raw("g1").shape[0]
+        self.w_in, _, self.off = L.stack(("q", "k", "v", "b", "a1", "g1"), ((qk, width), (qk, width), (v, width), (self.H, width), (ra, width), (rg, width)))
+        self.ra, self.rg = ra, rg
+        self.w_a2, self.w_g2 = L.mat("a2", (self.H * self.dk, ra)), L.mat("g2", (v, rg))
+        self.conv = torch.cat([L.f32(n + ".conv", (c, self.taps)) for n, c in (("q", qk), ("k", qk), ("v", v))]).contiguous()
+        self.A_log, self.dt_bias = L.f32("A_log", (self.H,)), L.f32("dt_bias", (self.H * self.dk,))
+        self.norm, self.w_out = L.f32("norm", (self.dv,)), L.mat("o", (width, v))
+
+    def state_spec(self):
+        spec = {"S": StateSpec((self.H, self.dk, self.dv), fp32=True, zero=True)}
+        if self.taps > 1:
+            spec["conv"] = StateSpec((self.taps - 1, self.conv.shape[0]), zero=True)
+        return spec
+
+    def forward(self, x: torch.Tensor, st: dict, ctx: StepContext) -> torch.Tensor:
+        oq, ok, ov, ob, oa, og = self.off
+        p = S.linear(x, self.w_in)
+        a = S.linear(p[:, oa:oa + self.ra], self.w_a2)
+        gate = S.linear(p[:, og:og + self.rg], self.w_g2)
+        q, k, v, logg, beta = S.delta_prep(p, (oq, ok, ov, ob), a, self.conv, self.A_log, self.dt_bias, st.get("conv"), ctx.B, ctx.n, self.H, self.G,
+                                           self.dk, self.dv, self.dk ** -0.5)
+        o = S.delta_rule(q, k, v, logg, beta, st["S"], ctx.B, ctx.n, self.H, self.G, self.dk, self.dv)
+        return S.linear(S.norm_gate(o, gate, self.norm, ctx.eps, self.H), self.w_out)
+
+
+def distance_bucket(n: int, buckets: int, bias_max: int) -> int:
+    """Bucket of distance n: the first half of the buckets one distance each, the rest spaced evenly in the logarithm up to bias_max."""
+    half = buckets // 2
+    if n < half:
+        return n
+    if half < 1 or bias_max <= half:
+        return buckets - 1
+    at = math.log(n / half) / math.log(bias_max / half) * (buckets - half)
+    return min(buckets - 1, half + math.floor(at + 1e-9))     # a distance on a bucket's border belongs to the bucket it opens
+
+
+def distance_table(rel: torch.Tensor, bias_max: int) -> torch.Tensor:
+    """rel [buckets, H] -> fp32 [H, D]: the bias of distances 0 .. D - 1, the last entry holding for all beyond."""
+    B = rel.shape[0]
+    row = [distance_bucket(0, B, bias_max)]
+    while row[-1] < B - 1:
+        row.append(distance_bucket(len(row), B, bias_max))
+    return rel.float()[torch.tensor(row, device=rel.device)].T.contiguous()
+
+
+class BiasAttention:
+    """Softmax attention with positions only in a learned bias by distance."""
+
+    def __init__(self, mc: dict, L: Loader, width: int):
+        self.H, self.G, self.dk, self.dv, self.scale = mc["heads"], mc["kv_heads"], mc["dim"], mc["vdim"], mc["scale"]
+        if self.H % self.G:
+            raise ValueError(f"{self.H} heads over {self.G} key / value heads")
+        q, k, v = self.H * self.dk, self.G * self.dk, self.G * self.dv
+        self.w_in, self.b_in, self.off = L.stack(("q", "k", "v"), ((q, width), (k, width), (v, width)), biases=True)
+        self.wq, self.wk = L.f32("q.norm", (q,)), L.f32("k.norm", (k,))
+        self.bias = S.bias_rows(distance_table(L.f32("rel"), mc["bias_max"]))
+        if self.bias.shape[0] != self.H:
+            raise ValueError(f"{L.prefix}rel holds {self.bias.shape[0]} heads, expected {self.H}")
+        self.v_mix = bool(mc.get("v_mix", False))
+        self.mix = L.f32("vmix").reshape(1) if self.v_mix and L.has("vmix") else None
+        self.w_out = L.mat("o", (width, self.H * self.dv))
+
+    def state_spec(self):
+        return {"k": StateSpec(("T_max", self.G * self.dk)), "v": StateSpec(("T_max", self.G * self.dv))}
+
+    def forward(self, x: torch.Tensor, st: dict, ctx: StepContext) -> torch.Tensor:
+        p = S.linear(x, self.w_in, self.b_in)
+        first = self.v_mix and ctx.v_first is None
+        if first:
+            ctx.v_first = torch.empty(ctx.B * ctx.n, self.G * self.dv, dtype=p.dtype, device=p.device)
+        elif self.v_mix and (self.mix is None or ctx.v_first.shape[1] != self.G * self.dv):
+            raise ValueError("value mixing needs the weight 'vmix' and the value width of the first mixing layer")
+        q = S.attn_prep(p, self.off, self.wq, self.wk, self.mix if self.v_mix and not first else None, ctx.v_first if self.v_mix else None, first,
+                        st["k"], st["v"], ctx.pos, ctx.B, ctx.n, ctx.eps)
+        o = S.attention_bias(q, st["k"], st["v"], self.bias, ctx.pos, ctx.host_pos, ctx.B, ctx.n, self.H, self.G, self.dk, self.dv, self.scale, True)
+        return S.linear(o, self.w_out)
+
+
+class DenseMlp:
+    def __init__(self, fc: dict, L: Loader, width: int):
+        self.up, self.down = L.mat("up", (fc["ff"], width)), L.mat("down", (width, fc["ff"]))
+
+    def forward(self, x: torch.Tensor) -> torch.Tensor:
+        return S.linear(S.linear(x, self.up, act=S.ACT_RELU2), self.down)
+
+
+MIXERS = {"lightning": Lightning, "channel_delta": ChannelDelta, "attention": BiasAttention}
+MLPS = {"dense": DenseMlp}

@@ -41,6 +41,39 @@ class Noise(C.Structure):
                 ("s_k", C.c_int64), ("s_p", C.c_int64)]
 
 
+class DeltaPrep(C.Structure):
+    _fields_ = [("proj", C.c_void_p), ("ldp", C.c_int64), ("off_q", C.c_int32), ("off_k", C.c_int32), ("off_v", C.c_int32), ("off_b", C.c_int32),
+                ("a", C.c_void_p), ("lda", C.c_int64), ("taps", C.c_void_p), ("A_log", C.c_void_p), ("dt_bias", C.c_void_p),
+                ("conv", C.c_void_p), ("n_taps", C.c_int32), ("B", C.c_int32), ("n", C.c_int32), ("H", C.c_int32), ("G", C.c_int32),
+                ("dk", C.c_int32), ("dv", C.c_int32), ("q_scale", C.c_float),
+                ("q", C.c_void_p), ("k", C.c_void_p), ("v", C.c_void_p), ("logg", C.c_void_p), ("beta", C.c_void_p)]
+
+
+class DeltaRule(C.Structure):
+    _fields_ = [("q", C.c_void_p), ("k", C.c_void_p), ("v", C.c_void_p), ("logg", C.c_void_p), ("beta", C.c_void_p), ("state", C.c_void_p),
+                ("o", C.c_void_p), ("B", C.c_int32), ("n", C.c_int32), ("H", C.c_int32), ("G", C.c_int32), ("dk", C.c_int32), ("dv", C.c_int32)]
+
+
+class DecayAttn(C.Structure):
+    _fields_ = [("q", C.c_void_p), ("k", C.c_void_p), ("v", C.c_void_p), ("ld", C.c_int64), ("decay", C.c_void_p), ("state", C.c_void_p),
+                ("o", C.c_void_p), ("B", C.c_int32), ("n", C.c_int32), ("H", C.c_int32), ("dk", C.c_int32), ("dv", C.c_int32)]
+
+
+class AttnPrep(C.Structure):
+    _fields_ = [("proj", C.c_void_p), ("ldp", C.c_int64), ("off_q", C.c_int32), ("off_k", C.c_int32), ("off_v", C.c_int32),
+                ("wq", C.c_void_p), ("wk", C.c_void_p), ("mix", C.c_void_p), ("v_first", C.c_void_p), ("v_first_write", C.c_int32),
+                ("q", C.c_void_p), ("kc", C.c_void_p), ("vc", C.c_void_p), ("k_batch", C.c_int64), ("v_batch", C.c_int64),
+                ("pos", C.c_void_p), ("B", C.c_int32), ("n", C.c_int32), ("qw", C.c_int32), ("kw", C.c_int32), ("vw", C.c_int32),
+                ("cap", C.c_int32), ("eps", C.c_float)]
+
+
+class AttnBias(C.Structure):
+    _fields_ = [("q", C.c_void_p), ("ldq", C.c_int64), ("k", C.c_void_p), ("v", C.c_void_p), ("k_batch", C.c_int64), ("v_batch", C.c_int64),
+                ("o", C.c_void_p), ("ldo", C.c_int64), ("bias", C.c_void_p), ("ldb", C.c_int64), ("n_bias", C.c_int32),
+                ("pos", C.c_void_p), ("host_pos", C.c_int32), ("cap", C.c_int32), ("B", C.c_int32), ("n", C.c_int32), ("H", C.c_int32),
+                ("G", C.c_int32), ("dk", C.c_int32), ("dv", C.c_int32), ("sink", C.c_int32), ("scale", C.c_float)]
+
+
 _I32, _I64, _P, _F = C.c_int32, C.c_int64, C.c_void_p, C.c_float
 _WP, _LP, _GP, _NP = C.POINTER(Weight), C.POINTER(Lora), C.POINTER(Logits), C.POINTER(Noise)
 
@@ -104,9 +137,23 @@ SIGNATURES = {
     "plz_swiglu_fwd": [_P, _I64, _P, _I64, _I32, _I32, _P, _I64, _P],
     "plz_add": [_P, _I64, _P, _I64, _P, _I64, _I32, _I32, _P, _I64, _P],
     "plz_bwd_dw_hard_lora": [_WP, _P, _I64, _P, _I64, _I32, _P, _P, _P, _I32, _P, _P, _P],
+    "plz_seq_linear": [_I32, _P, _I64, _I32, _I32, _P, _I64, _I32, _P, _I32, _P, _I64, _I32, _P],
+    "plz_seq_embed": [_I32, _P, _I64, _P, _I64, _I32, _I64, _F, _P, _P, _P, _P],
+    "plz_seq_residual_norm": [_I32, _P, _I64, _P, _F, _F, _F, _I64, _I32, _P, _P, _P],
+    "plz_seq_rows_norm": [_I32, _P, _P, _P, _F, _F, _I64, _I32, _P, _P],
+    "plz_seq_norm_gate": [_I32, _P, _P, _I64, _P, _F, _I64, _I32, _I32, _P, _P],
+    "plz_delta_prep": [_I32, C.POINTER(DeltaPrep), _P],
+    "plz_delta_rule": [C.POINTER(DeltaRule), _P],
+    "plz_decay_attn": [_I32, C.POINTER(DecayAttn), _P],
+    "plz_attn_prep": [_I32, C.POINTER(AttnPrep), _P],
+    "plz_attn_bias_ws_bytes": [_I32, _I32, _I32, _I32, _I32],
+    "plz_attn_bias": [_I32, C.POINTER(AttnBias), _P, _I64, _P],
+    "plz_advance": [_P, _I32, _P],
+    "plz_sample": [_P, _I64, _I32, _I32, _F, _I32, C.c_uint32, _P, _P, _P],
     "plz_distill_loss": [_P, _I64, _P, _I64, _I32, _I32, _F, _F, _F, _P, _P, _P, _I64, _I32, _P],
 }
-_RESTYPES = {"plz_last_error": C.c_char_p, "plz_launch_count": C.c_uint64, "plz_attn_decode_ws_bytes": C.c_int64}
+_RESTYPES = {"plz_last_error": C.c_char_p, "plz_launch_count": C.c_uint64, "plz_attn_decode_ws_bytes": C.c_int64,
+             "plz_attn_bias_ws_bytes": C.c_int64}
 
 
 def lib():

@@ -1,0 +1,147 @@
+"""Functional wrappers over the hybrid-decoder entry points of include/plz.h (recurrent and attention mixers, fp32 residual stream,
+sampling). Tensors are torch CUDA tensors in the model's type T (bf16, or fp32 in the 32-bit mode) unless noted; rows are b * n + t for
+B sequences that advance in lockstep by n tokens."""
+from __future__ import annotations
+
+import ctypes as C
+
+import torch
+
+import plz_native as P
+
+ACT_NONE, ACT_RELU2 = 0, 1
+BIAS_FRONT, BIAS_BACK = 128, 256      # readable entries before distance 0 / after the last one of a bias row (tile-wide reads)
+
+
+def code(dtype: torch.dtype) -> int:
+    return {torch.bfloat16: 0, torch.float32: 1}[dtype]
+
+
+def _ptr(t):
+    return None if t is None else t.data_ptr()
+
+
+def linear(x: torch.Tensor, w: torch.Tensor, bias=None, act: int = ACT_NONE, out_f32: bool = False) -> torch.Tensor:
+    """act(x W^T + bias); x [M, K] rows of any pitch, w [N, K] (its rows may be pitched)."""
+    P._need_cuda(x, w)
+    M, K = x.shape
+    N = w.shape[0]
+    assert w.shape[1] == K and x.stride(1) == 1 and w.stride(1) == 1 and x.dtype == w.dtype
+    y = torch.empty(M, N, dtype=torch.float32 if out_f32 else x.dtype, device=x.device)
+    f32 = out_f32 and x.dtype != torch.float32
+    P.check(P.lib().plz_seq_linear(code(x.dtype), x.data_ptr(), x.stride(0), M, K, w.data_ptr(), w.stride(0), N, _ptr(bias), act, y.data_ptr(),
+                                   y.stride(0), int(f32), P.stream_ptr()), "plz_seq_linear")
+    return y
+
+
+def embed(table: torch.Tensor, ids: torch.Tensor, scale: float):
+    """(x fp32 [rows, W], the same in T: x itself in the 32-bit mode)."""
+    P._need_cuda(table, ids)
+    rows, W = ids.numel(), table.shape[1]
+    assert ids.dtype == torch.int64 and ids.is_contiguous()
+    x = torch.empty(rows, W, dtype=torch.float32, device=table.device)
+    xb = x if table.dtype == torch.float32 else torch.empty(rows, W, dtype=table.dtype, device=table.device)
+    P.check(P.lib().plz_seq_embed(code(table.dtype), table.data_ptr(), table.stride(0), ids.data_ptr(), rows, W, table.shape[0], float(scale),
+                                  x.data_ptr(), None if xb is x else xb.data_ptr(), None, P.stream_ptr()), "plz_seq_embed")
+    return x, xb
+
+
+def residual_norm(y: torch.Tensor, w: torch.Tensor, w_offset: float, mult: float, eps: float, x: torch.Tensor, xb: torch.Tensor):
+    """x += mult * rms_norm(y) * (w + w_offset) in place; xb follows (nothing to do when it is x)."""
+    P.check(P.lib().plz_seq_residual_norm(code(y.dtype), y.data_ptr(), y.stride(0), w.data_ptr(), float(w_offset), float(mult), float(eps),
+                                          y.shape[0], y.shape[1], x.data_ptr(), None if xb is x else xb.data_ptr(), P.stream_ptr()),
+            "plz_seq_residual_norm")
+
+
+def rows_norm(x: torch.Tensor, idx, w: torch.Tensor, w_offset: float, eps: float, dtype: torch.dtype) -> torch.Tensor:
+    rows = x.shape[0] if idx is None else idx.numel()
+    out = torch.empty(rows, x.shape[1], dtype=dtype, device=x.device)
+    P.check(P.lib().plz_seq_rows_norm(code(dtype), x.data_ptr(), _ptr(idx), w.data_ptr(), float(w_offset), float(eps), rows, x.shape[1],
+                                      out.data_ptr(), P.stream_ptr()), "plz_seq_rows_norm")
+    return out
+
+
+def norm_gate(o: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, eps: float, groups: int) -> torch.Tensor:
+    """o fp32 [rows, groups * L]; gate a T view [rows, groups * L]; w fp32 [L]."""
+    rows, W = o.shape
+    out = torch.empty(rows, W, dtype=gate.dtype, device=o.device)
+    P.check(P.lib().plz_seq_norm_gate(code(gate.dtype), o.data_ptr(), gate.data_ptr(), gate.stride(0), w.data_ptr(), float(eps), rows, groups,
+                                      W // groups, out.data_ptr(), P.stream_ptr()), "plz_seq_norm_gate")
+    return out
+
+
+def delta_prep(proj: torch.Tensor, offs, a: torch.Tensor, taps: torch.Tensor, A_log: torch.Tensor, dt_bias: torch.Tensor, conv, B: int, n: int,
+               H: int, G: int, dk: int, dv: int, q_scale: float):
+    """(q, k, v, log decay, beta), all fp32; offs = columns of (q, k, v, beta) in proj; conv (inputs kept for the convolution) is updated."""
+    dev, rows = proj.device, B * n
+    f = lambda w: torch.empty(rows, w, dtype=torch.float32, device=dev)
+    q, k, v, lg, beta = f(G * dk), f(G * dk), f(H * dv), f(H * dk), f(H)
+    d = P.DeltaPrep(proj.data_ptr(), proj.stride(0), *offs, a.data_ptr(), a.stride(0), taps.data_ptr(), A_log.data_ptr(), dt_bias.data_ptr(),
+                    _ptr(conv), taps.shape[1], B, n, H, G, dk, dv, float(q_scale), q.data_ptr(), k.data_ptr(), v.data_ptr(), lg.data_ptr(), beta.data_ptr())
+    P.check(P.lib().plz_delta_prep(code(proj.dtype), C.byref(d), P.stream_ptr()), "plz_delta_prep")
+    return q, k, v, lg, beta
+
+
+def delta_rule(q, k, v, logg, beta, state: torch.Tensor, B: int, n: int, H: int, G: int, dk: int, dv: int) -> torch.Tensor:
+    """o fp32 [B * n, H * dv]; state fp32 [B, H, dk, dv] in place."""
+    o = torch.empty(B * n, H * dv, dtype=torch.float32, device=state.device)
+    d = P.DeltaRule(q.data_ptr(), k.data_ptr(), v.data_ptr(), logg.data_ptr(), beta.data_ptr(), state.data_ptr(), o.data_ptr(), B, n, H, G, dk, dv)
+    P.check(P.lib().plz_delta_rule(C.byref(d), P.stream_ptr()), "plz_delta_rule")
+    return o
+
+
+def decay_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, B: int, n: int, H: int, dk: int,
+                    dv: int) -> torch.Tensor:
+    """q, k, v: slices (before silu) of one projection; o fp32 [B * n, H * dv]; state fp32 [B, H, dk, dv] in place."""
+    assert q.stride(0) == k.stride(0) == v.stride(0)
+    o = torch.empty(B * n, H * dv, dtype=torch.float32, device=state.device)
+    d = P.DecayAttn(q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), decay.data_ptr(), state.data_ptr(), o.data_ptr(), B, n, H, dk, dv)
+    P.check(P.lib().plz_decay_attn(code(q.dtype), C.byref(d), P.stream_ptr()), "plz_decay_attn")
+    return o
+
+
+def attn_prep(proj: torch.Tensor, offs, wq: torch.Tensor, wk: torch.Tensor, mix, v_first, v_first_write: bool, kc: torch.Tensor, vc: torch.Tensor,
+              pos: torch.Tensor, B: int, n: int, eps: float) -> torch.Tensor:
+    """Normalised queries [B * n, qw]; keys and (mixed) values go into the caches kc [B, cap, kw], vc [B, cap, vw] at pos."""
+    qw, kw, vw = wq.numel(), kc.shape[2], vc.shape[2]
+    q = torch.empty(B * n, qw, dtype=proj.dtype, device=proj.device)
+    d = P.AttnPrep(proj.data_ptr(), proj.stride(0), *offs, wq.data_ptr(), wk.data_ptr(), _ptr(mix), _ptr(v_first), int(v_first_write), q.data_ptr(),
+                   kc.data_ptr(), vc.data_ptr(), kc.stride(0), vc.stride(0), pos.data_ptr(), B, n, qw, kw, vw, kc.shape[1], float(eps))
+    P.check(P.lib().plz_attn_prep(code(proj.dtype), C.byref(d), P.stream_ptr()), "plz_attn_prep")
+    return q
+
+
+def bias_rows(by_distance: torch.Tensor) -> torch.Tensor:
+    """[H, D] biases of distances 0 .. D - 1 (the last one for all beyond) -> padded rows; pass the result to attention_bias."""
+    H, D = by_distance.shape
+    out = torch.zeros(H, BIAS_FRONT + D + BIAS_BACK, dtype=torch.float32, device=by_distance.device)
+    out[:, BIAS_FRONT:BIAS_FRONT + D] = by_distance
+    out[:, BIAS_FRONT + D:] = by_distance[:, -1:]
+    return out
+
+
+def attention_bias(q: torch.Tensor, kc: torch.Tensor, vc: torch.Tensor, bias, pos: torch.Tensor, host_pos: int, B: int, n: int, H: int, G: int,
+                   dk: int, dv: int, scale: float, sink: bool) -> torch.Tensor:
+    """Causal attention of n new tokens per sequence (their keys and values already in the caches). bias: bias_rows(...) or None.
+    host_pos: the value of pos, or -1 (one token only) when the launch is to be replayed at other positions."""
+    o = torch.empty(B * n, H * dv, dtype=q.dtype, device=q.device)
+    bp, ldb, nb = (None, 0, 0) if bias is None else (bias.data_ptr() + 4 * BIAS_FRONT, bias.stride(0), bias.shape[1] - BIAS_FRONT - BIAS_BACK)
+    d = P.AttnBias(q.data_ptr(), q.stride(0), kc.data_ptr(), vc.data_ptr(), kc.stride(0), vc.stride(0), o.data_ptr(), o.stride(0), bp, ldb, nb,
+                   pos.data_ptr(), host_pos, kc.shape[1], B, n, H, G, dk, dv, int(sink), float(scale))
+    need = P.lib().plz_attn_bias_ws_bytes(B, H, G, dv, kc.shape[1]) if n == 1 else 0
+    ws = torch.empty(need, dtype=torch.uint8, device=q.device) if need else None
+    P.check(P.lib().plz_attn_bias(code(q.dtype), C.byref(d), _ptr(ws), need, P.stream_ptr()), "plz_attn_bias")
+    return o
+
+
+def advance(pos: torch.Tensor, n: int):
+    P.check(P.lib().plz_advance(pos.data_ptr(), n, P.stream_ptr()), "plz_advance")
+
+
+def sample(logits: torch.Tensor, pos: torch.Tensor, temperature: float = 0.0, top_k: int = 0, seed: int = 0) -> torch.Tensor:
+    """Next token int64 [rows] of fp32 logits [rows, V]; temperature 0 is greedy."""
+    assert logits.dtype == torch.float32 and logits.stride(1) == 1
+    out = torch.empty(logits.shape[0], dtype=torch.int64, device=logits.device)
+    P.check(P.lib().plz_sample(logits.data_ptr(), logits.stride(0), logits.shape[0], logits.shape[1], float(temperature), int(top_k),
+                               seed & 0xFFFFFFFF, pos.data_ptr(), out.data_ptr(), P.stream_ptr()), "plz_sample")
+    return out
