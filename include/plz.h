@@ -418,7 +418,7 @@ int32_t plz_bwd_dw_hard_lora(const plz_weight_t* w, const void* x, int64_t ldx, 
  * plz_attn_prep: RMS norm of the whole q and k projections, optional value mixing with the first mixing layer's values, and the
  *   write of keys and values into the cache at *pos + t.
  * plz_attn_bias: causal attention of the n new tokens against the cache (which already holds them), score * scale + bias by distance
- *   (bias points at distance 0 of head 0; entry n_bias - 1 holds for everything farther; rows ldb apart, readable from 128 entries
+ *   (bias points at distance 0 of head 0; entry n_bias - 1 holds for everything farther; rows ldb apart, readable from 256 entries
  *   before distance 0 to 256 entries past n_bias - 1), optional sink in the denominator. host_pos = *pos when the caller knows it, or
  *   -1 (n == 1 only). ws: plz_attn_bias_ws_bytes bytes for n == 1, else unused. */
 int32_t plz_seq_linear(int32_t dtype, const void* x, int64_t ldx, int32_t M, int32_t K, const void* w, int64_t ldw, int32_t N, const void* bias,
@@ -474,6 +474,7 @@ typedef struct plz_attn_bias {
     const void* k; const void* v; int64_t k_batch, v_batch;    /* caches [B, cap, G * dk], [B, cap, G * dv] */
     void* o; int64_t ldo;                                      /* [B * n, H * dv] */
     const float* bias; int64_t ldb; int32_t n_bias;
+    const float* bias_top;                                     /* [H], at least the largest bias of the head; NULL: CUDA-core kernel */
     const int32_t* pos; int32_t host_pos, cap;
     int32_t B, n, H, G, dk, dv, sink;
     float scale;

@@ -82,6 +82,25 @@ int make_tmap_bf16(CUtensorMap* map, const void* base, uint64_t rows, uint64_t c
     return PLZ_OK;
 }
 
+int make_tmap_bf16_heads(CUtensorMap* map, const void* base, uint64_t dim, uint64_t heads, uint64_t tokens, uint64_t batch, uint64_t tok_pitch,
+                         uint64_t batch_pitch, uint32_t box_tokens) {
+    EncodeTiledFn enc = get_encode_fn();
+    static thread_local int bound_dev = -1;
+    int dev = -1;
+    if (cudaGetDevice(&dev) == cudaSuccess && dev != bound_dev) { cudaSetDevice(dev); bound_dev = dev; }   // see make_tmap_bf16
+    if (!enc) { set_last_error("cuTensorMapEncodeTiled is not available from the driver"); return PLZ_ERR_CUDA; }
+    if (!base) { set_last_error("null tensor pointer"); return PLZ_ERR_NULL; }
+    if (((uintptr_t)base & 15) || dim % 8 || tok_pitch % 8 || batch_pitch % 8) { set_last_error("bf16 head tensor: base and pitches must be multiples of 16 bytes"); return PLZ_ERR_BAD_ALIGN; }
+    cuuint64_t dims[4] = {dim, heads, tokens, batch};
+    cuuint64_t strides[3] = {dim * 2, tok_pitch * 2, batch_pitch * 2};
+    cuuint32_t box[4] = {64, 1, box_tokens, 1};
+    cuuint32_t estr[4] = {1, 1, 1, 1};
+    CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                     CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    if (r != CUDA_SUCCESS) { set_last_error("cuTensorMapEncodeTiled failed with CUresult %d (dim %llu heads %llu tokens %llu)", (int)r, (unsigned long long)dim, (unsigned long long)heads, (unsigned long long)tokens); return PLZ_ERR_CUDA; }
+    return PLZ_OK;
+}
+
 static int check_weight(const plz_weight_t* w, bool need_packed) {
     if (!w) { set_last_error("null weight descriptor"); return PLZ_ERR_NULL; }
     if (w->N <= 0 || w->K <= 0) { set_last_error("weight is empty (N=%d, K=%d)", w->N, w->K); return PLZ_ERR_BAD_SHAPE; }
@@ -1046,6 +1065,8 @@ int32_t plz_attn_bias(int32_t dtype, const plz_attn_bias_t* a, void* ws, int64_t
     const bool vec = a->dk % 8 == 0 && a->dv % 8 == 0 && a->ldq % per16 == 0 && a->k_batch % per16 == 0 && a->v_batch % per16 == 0 &&
                      !((uintptr_t)a->q & 15) && !((uintptr_t)a->k & 15) && !((uintptr_t)a->v & 15);
     if (a->n == 1 && vec && a->dk <= 256 && a->dv <= 256) return launch_attn_bias_decode(dtype, *a, a->cap, ws, ws ? ws_bytes : 0, s);
+    if (dtype == 0 && vec && a->n > 1 && a->dk <= 128 && a->dv <= 128 && a->scale > 0.f && (!a->bias || a->bias_top) && a->ldo % 8 == 0 && !((uintptr_t)a->o & 15))
+        return launch_attn_bias_tc(*a, s);
     return launch_attn_bias_simt(dtype, *a, s);
 }
 

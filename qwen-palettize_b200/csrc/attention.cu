@@ -16,16 +16,13 @@
 //                  S, dP -> P, dS to shared memory -> dV += P^T dO, dK += dS^T Q  (P^T / dS^T are the same bytes read
 //                  through an MN-major operand descriptor)
 // D[row] = sum_d dO O is a small pre-pass. Every barrier wait is bounded (status word, as in the GEMM kernels).
-#include "plz_launch.h"
+#include "attention_tiles.cuh"
 
 namespace plz {
 namespace {
 
-constexpr int kT = 128;                         // tokens per tile
 constexpr int kD = 128;                         // head dimension
-constexpr uint32_t kBlk = kT * 64 * 2;          // one 64-column block of a 128-row bf16 tile: 16 KB
 constexpr uint32_t kTile = 2 * kBlk;            // a 128 x 128 bf16 tile: 32 KB
-constexpr float kLog2e = 1.4426950408889634f;
 
 struct AttnParams {
     int B, S, Hq, Hkv;
@@ -35,18 +32,6 @@ struct AttnParams {
     StatusWord* status;
 };
 
-__device__ __forceinline__ void tmem_st_32x32(uint32_t taddr, const uint32_t (&r)[32]) {
-    asm volatile(
-        "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], "
-        "{%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16, "
-        "%17, %18, %19, %20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31, %32};\n\t"
-        "tcgen05.wait::st.sync.aligned;"
-        ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]),
-          "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]), "r"(r[16]), "r"(r[17]), "r"(r[18]), "r"(r[19]),
-          "r"(r[20]), "r"(r[21]), "r"(r[22]), "r"(r[23]), "r"(r[24]), "r"(r[25]), "r"(r[26]), "r"(r[27]), "r"(r[28]), "r"(r[29]),
-          "r"(r[30]), "r"(r[31])
-        : "memory");
-}
 __device__ __forceinline__ void bar_sync_128() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
 
 // eight MMAs of one 128 x 128 x 128 product. A / B tiles are 128-row bf16 tiles of two 64-column blocks.
@@ -66,10 +51,6 @@ __device__ __forceinline__ void mma_128(uint32_t d_tmem, uint32_t sA, bool a_mn,
     }
 }
 
-// 16-byte chunk c (8 bf16) of row r of a two-block K-major tile, 128-byte swizzle
-__device__ __forceinline__ uint8_t* tile_chunk(uint8_t* tile, int r, int c16) {
-    return tile + (c16 >> 3) * kBlk + r * 128 + (((c16 & 7) ^ (r & 7)) << 4);
-}
 __device__ __forceinline__ void load_tile(uint32_t dst, const CUtensorMap* map, uint32_t bar, int col0, int row0) {
     tma_load_2d(dst, map, bar, col0, row0);
     tma_load_2d(dst + kBlk, map, bar, col0 + 64, row0);

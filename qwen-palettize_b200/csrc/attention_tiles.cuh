@@ -1,0 +1,42 @@
+// Tile geometry and TMEM / shared-memory helpers shared by the tensor-core attention kernels: 128-token tiles, bf16 operands in
+// 128-byte-swizzled shared memory as 64-column blocks of 16 KB.
+#pragma once
+#include "plz_launch.h"
+
+namespace plz {
+
+constexpr int kT = 128;                         // tokens per tile
+constexpr uint32_t kBlk = kT * 64 * 2;          // one 64-column block of a 128-row bf16 tile: 16 KB
+constexpr float kLog2e = 1.4426950408889634f;
+
+__device__ __forceinline__ void tmem_st_32x32(uint32_t taddr, const uint32_t (&r)[32]) {
+    asm volatile(
+        "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], "
+        "{%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16, "
+        "%17, %18, %19, %20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31, %32};\n\t"
+        "tcgen05.wait::st.sync.aligned;"
+        ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]),
+          "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]), "r"(r[16]), "r"(r[17]), "r"(r[18]), "r"(r[19]),
+          "r"(r[20]), "r"(r[21]), "r"(r[22]), "r"(r[23]), "r"(r[24]), "r"(r[25]), "r"(r[26]), "r"(r[27]), "r"(r[28]), "r"(r[29]),
+          "r"(r[30]), "r"(r[31])
+        : "memory");
+}
+
+// 16-byte chunk c (8 bf16) of row r of a two-block K-major tile, 128-byte swizzle
+__device__ __forceinline__ uint8_t* tile_chunk(uint8_t* tile, int r, int c16) {
+    return tile + (c16 >> 3) * kBlk + r * 128 + (((c16 & 7) ^ (r & 7)) << 4);
+}
+
+// 4-D box load / store (coordinates innermost first)
+__device__ __forceinline__ void tma_load_4d(uint32_t dst_smem, const CUtensorMap* map, uint32_t bar, int32_t x, int32_t y, int32_t z, int32_t w) {
+    asm volatile("cp.async.bulk.tensor.4d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5, %6}], [%2];"
+                 ::"r"(dst_smem), "l"(reinterpret_cast<uint64_t>(map)), "r"(bar), "r"(x), "r"(y), "r"(z), "r"(w)
+                 : "memory");
+}
+__device__ __forceinline__ void tma_store_4d(const CUtensorMap* map, uint32_t src_smem, int32_t x, int32_t y, int32_t z, int32_t w) {
+    asm volatile("cp.async.bulk.tensor.4d.global.shared::cta.bulk_group [%0, {%2, %3, %4, %5}], [%1];"
+                 ::"l"(reinterpret_cast<uint64_t>(map)), "r"(src_smem), "r"(x), "r"(y), "r"(z), "r"(w)
+                 : "memory");
+}
+
+}  // namespace plz

@@ -25,6 +25,11 @@ EncodeTiledFn get_encode_fn();
 int make_tmap_bf16(CUtensorMap* map, const void* base, uint64_t rows, uint64_t cols, uint64_t ld,
                    uint32_t box_cols, uint32_t box_rows);
 
+// bf16 [batch, tokens, heads, dim] with the given pitches (elements): boxes of 64 dim columns x 1 head x box_tokens, 128-byte swizzle,
+// out-of-range elements read as zero and are not written. dim may be any multiple of 8.
+int make_tmap_bf16_heads(CUtensorMap* map, const void* base, uint64_t dim, uint64_t heads, uint64_t tokens, uint64_t batch, uint64_t tok_pitch,
+                         uint64_t batch_pitch, uint32_t box_tokens);
+
 #define PLZ_CUDA_CHECK(expr)                                                            \
     do {                                                                                \
         cudaError_t _e = (expr);                                                        \

@@ -186,6 +186,7 @@ int launch_attn_prep(int dtype, const AttnPrepArgs& a, cudaStream_t stream);
 using AttnBiasArgs = plz_attn_bias_t;
 long long attn_bias_decode_ws_bytes(int B, int H, int G, int dv, int cap);
 int launch_attn_bias_decode(int dtype, const AttnBiasArgs& a, int cap, void* ws, long long ws_bytes, cudaStream_t stream);
+int launch_attn_bias_tc(const AttnBiasArgs& a, cudaStream_t stream);   // attention_bias_tc.cu
 int launch_attn_bias_simt(int dtype, const AttnBiasArgs& a, cudaStream_t stream);
 int launch_advance(int* pos, int n, cudaStream_t stream);
 int launch_sample(const float* logits, long long ld, int rows, int V, float temperature, int top_k, uint32_t seed, const int* pos, long long* out,

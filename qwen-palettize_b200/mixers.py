@@ -161,9 +161,9 @@ class BiasAttention:
         q, k, v = self.H * self.dk, self.G * self.dk, self.G * self.dv
         self.w_in, self.b_in, self.off = L.stack(("q", "k", "v"), ((q, width), (k, width), (v, width)), biases=True)
         self.wq, self.wk = L.f32("q.norm", (q,)), L.f32("k.norm", (k,))
-        self.bias = S.bias_rows(distance_table(L.f32("rel"), mc["bias_max"]))
-        if self.bias.shape[0] != self.H:
-            raise ValueError(f"{L.prefix}rel holds {self.bias.shape[0]} heads, expected {self.H}")
+        self.bias = S.DistanceBias.from_distances(distance_table(L.f32("rel"), mc["bias_max"]))
+        if self.bias.top.numel() != self.H:
+            raise ValueError(f"{L.prefix}rel holds {self.bias.top.numel()} heads, expected {self.H}")
         self.v_mix = bool(mc.get("v_mix", False))
         self.mix = L.f32("vmix").reshape(1) if self.v_mix and L.has("vmix") else None
         self.w_out = L.mat("o", (width, self.H * self.dv))

@@ -69,7 +69,7 @@ class AttnPrep(C.Structure):
 
 class AttnBias(C.Structure):
     _fields_ = [("q", C.c_void_p), ("ldq", C.c_int64), ("k", C.c_void_p), ("v", C.c_void_p), ("k_batch", C.c_int64), ("v_batch", C.c_int64),
-                ("o", C.c_void_p), ("ldo", C.c_int64), ("bias", C.c_void_p), ("ldb", C.c_int64), ("n_bias", C.c_int32),
+                ("o", C.c_void_p), ("ldo", C.c_int64), ("bias", C.c_void_p), ("ldb", C.c_int64), ("n_bias", C.c_int32), ("bias_top", C.c_void_p),
                 ("pos", C.c_void_p), ("host_pos", C.c_int32), ("cap", C.c_int32), ("B", C.c_int32), ("n", C.c_int32), ("H", C.c_int32),
                 ("G", C.c_int32), ("dk", C.c_int32), ("dv", C.c_int32), ("sink", C.c_int32), ("scale", C.c_float)]
 

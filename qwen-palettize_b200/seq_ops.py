@@ -4,13 +4,14 @@ B sequences that advance in lockstep by n tokens."""
 from __future__ import annotations
 
 import ctypes as C
+from dataclasses import dataclass
 
 import torch
 
 import plz_native as P
 
 ACT_NONE, ACT_RELU2 = 0, 1
-BIAS_FRONT, BIAS_BACK = 128, 256      # readable entries before distance 0 / after the last one of a bias row (tile-wide reads)
+BIAS_FRONT, BIAS_BACK = 256, 256      # readable entries before distance 0 / after the last one of a bias row (tile-wide reads)
 
 
 def code(dtype: torch.dtype) -> int:
@@ -111,22 +112,30 @@ def attn_prep(proj: torch.Tensor, offs, wq: torch.Tensor, wk: torch.Tensor, mix,
     return q
 
 
-def bias_rows(by_distance: torch.Tensor) -> torch.Tensor:
-    """[H, D] biases of distances 0 .. D - 1 (the last one for all beyond) -> padded rows; pass the result to attention_bias."""
-    H, D = by_distance.shape
-    out = torch.zeros(H, BIAS_FRONT + D + BIAS_BACK, dtype=torch.float32, device=by_distance.device)
-    out[:, BIAS_FRONT:BIAS_FRONT + D] = by_distance
-    out[:, BIAS_FRONT + D:] = by_distance[:, -1:]
-    return out
+@dataclass
+class DistanceBias:
+    """Bias by distance of every head, as the attention kernels read it."""
+    rows: torch.Tensor      # fp32 [H, BIAS_FRONT + D + BIAS_BACK]: zeros, distances 0 .. D - 1, the last one repeated
+    top: torch.Tensor       # fp32 [H], the largest of each head
+    D: int
+
+    @classmethod
+    def from_distances(cls, by_distance: torch.Tensor) -> "DistanceBias":
+        """by_distance [H, D]: the biases of distances 0 .. D - 1; the last one holds for all beyond."""
+        H, D = by_distance.shape
+        rows = torch.zeros(H, BIAS_FRONT + D + BIAS_BACK, dtype=torch.float32, device=by_distance.device)
+        rows[:, BIAS_FRONT:BIAS_FRONT + D] = by_distance
+        rows[:, BIAS_FRONT + D:] = by_distance[:, -1:]
+        return cls(rows, by_distance.float().max(1).values.contiguous(), D)
 
 
-def attention_bias(q: torch.Tensor, kc: torch.Tensor, vc: torch.Tensor, bias, pos: torch.Tensor, host_pos: int, B: int, n: int, H: int, G: int,
-                   dk: int, dv: int, scale: float, sink: bool) -> torch.Tensor:
-    """Causal attention of n new tokens per sequence (their keys and values already in the caches). bias: bias_rows(...) or None.
+def attention_bias(q: torch.Tensor, kc: torch.Tensor, vc: torch.Tensor, bias: DistanceBias | None, pos: torch.Tensor, host_pos: int, B: int, n: int,
+                   H: int, G: int, dk: int, dv: int, scale: float, sink: bool) -> torch.Tensor:
+    """Causal attention of n new tokens per sequence (their keys and values already in the caches).
     host_pos: the value of pos, or -1 (one token only) when the launch is to be replayed at other positions."""
     o = torch.empty(B * n, H * dv, dtype=q.dtype, device=q.device)
-    bp, ldb, nb = (None, 0, 0) if bias is None else (bias.data_ptr() + 4 * BIAS_FRONT, bias.stride(0), bias.shape[1] - BIAS_FRONT - BIAS_BACK)
-    d = P.AttnBias(q.data_ptr(), q.stride(0), kc.data_ptr(), vc.data_ptr(), kc.stride(0), vc.stride(0), o.data_ptr(), o.stride(0), bp, ldb, nb,
+    bp, ldb, nb, top = (None, 0, 0, None) if bias is None else (bias.rows.data_ptr() + 4 * BIAS_FRONT, bias.rows.stride(0), bias.D, bias.top.data_ptr())
+    d = P.AttnBias(q.data_ptr(), q.stride(0), kc.data_ptr(), vc.data_ptr(), kc.stride(0), vc.stride(0), o.data_ptr(), o.stride(0), bp, ldb, nb, top,
                    pos.data_ptr(), host_pos, kc.shape[1], B, n, H, G, dk, dv, int(sink), float(scale))
     need = P.lib().plz_attn_bias_ws_bytes(B, H, G, dv, kc.shape[1]) if n == 1 else 0
     ws = torch.empty(need, dtype=torch.uint8, device=q.device) if need else None
