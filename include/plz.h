@@ -448,7 +448,10 @@ typedef struct plz_delta_rule {
     float* state; float* o;
     int32_t B, n, H, G, dk, dv;
 } plz_delta_rule_t;
-int32_t plz_delta_rule(const plz_delta_rule_t* args, void* stream);
+/* ws (both recurrences): NULL: token by token; else the chunked form (dk <= 128; 64-token chunks on the tensor cores, operands as
+ * hi + lo bf16 pairs), plz_chunk_ws_bytes bytes, 16-byte aligned. */
+int64_t plz_chunk_ws_bytes(int32_t B, int32_t n, int32_t H, int32_t dk, int32_t dv);
+int32_t plz_delta_rule(const plz_delta_rule_t* args, void* ws, int64_t ws_bytes, void* stream);
 
 typedef struct plz_decay_attn {
     const void* q; const void* k; const void* v; int64_t ld;   /* slices of one projection before silu, dtype, rows ld apart */
@@ -456,7 +459,7 @@ typedef struct plz_decay_attn {
     float* state; float* o;
     int32_t B, n, H, dk, dv;
 } plz_decay_attn_t;
-int32_t plz_decay_attn(int32_t dtype, const plz_decay_attn_t* args, void* stream);
+int32_t plz_decay_attn(int32_t dtype, const plz_decay_attn_t* args, void* ws, int64_t ws_bytes, void* stream);
 
 typedef struct plz_attn_prep {
     const void* proj; int64_t ldp; int32_t off_q, off_k, off_v;

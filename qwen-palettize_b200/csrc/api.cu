@@ -1018,20 +1018,30 @@ int32_t plz_delta_prep(int32_t dtype, const plz_delta_prep_t* a, void* stream) {
     return launch_delta_prep(dtype, *a, (cudaStream_t)stream);
 }
 
-int32_t plz_delta_rule(const plz_delta_rule_t* a, void* stream) {
+int64_t plz_chunk_ws_bytes(int32_t B, int32_t n, int32_t H, int32_t dk, int32_t dv) {
+    if (B <= 0 || n <= 0 || H <= 0 || dk <= 0 || dv <= 0) return 0;
+    return chunk_ws_bytes(B, n, H, dk, dv);
+}
+
+int32_t plz_delta_rule(const plz_delta_rule_t* a, void* ws, int64_t ws_bytes, void* stream) {
     if (!a || !a->q || !a->k || !a->v || !a->logg || !a->beta || !a->state || !a->o) { set_last_error("null pointer"); return PLZ_ERR_NULL; }
     if (a->B < 0 || a->n < 0 || a->H <= 0 || a->G <= 0 || a->H % a->G || a->dk <= 0 || a->dv <= 0 || a->H > 65535 || a->B > 65535) {
         set_last_error("delta_rule: bad shape H=%d G=%d dk=%d dv=%d", a->H, a->G, a->dk, a->dv); return PLZ_ERR_BAD_SHAPE;
     }
+    if (ws && a->B > 0 && a->n > 0) return launch_chunk_delta(*a, ws, ws_bytes, (cudaStream_t)stream);
     return launch_recurrent_delta(*a, (cudaStream_t)stream);
 }
 
-int32_t plz_decay_attn(int32_t dtype, const plz_decay_attn_t* a, void* stream) {
+int32_t plz_decay_attn(int32_t dtype, const plz_decay_attn_t* a, void* ws, int64_t ws_bytes, void* stream) {
     int rc = check_dtype(dtype);
     if (rc) return rc;
     if (!a || !a->q || !a->k || !a->v || !a->decay || !a->state || !a->o) { set_last_error("null pointer"); return PLZ_ERR_NULL; }
     if (a->B < 0 || a->n < 0 || a->H <= 0 || a->dk <= 0 || a->dv <= 0 || a->H > 65535 || a->B > 65535) {
         set_last_error("decay_attn: bad shape H=%d dk=%d dv=%d", a->H, a->dk, a->dv); return PLZ_ERR_BAD_SHAPE;
+    }
+    if (ws && a->B > 0 && a->n > 0) {
+        if (dtype != 0) { set_last_error("decay_attn: the chunked form takes bf16 projections"); return PLZ_ERR_UNSUPPORTED; }
+        return launch_chunk_decay(*a, ws, ws_bytes, (cudaStream_t)stream);
     }
     return launch_recurrent_decay(dtype, *a, (cudaStream_t)stream);
 }

@@ -180,6 +180,10 @@ int launch_delta_prep(int dtype, const DeltaPrepArgs& a, cudaStream_t stream);
 using DeltaRuleArgs = plz_delta_rule_t;
 int launch_recurrent_delta(const DeltaRuleArgs& a, cudaStream_t stream);
 using DecayAttnArgs = plz_decay_attn_t;
+// seq_chunk.cu: the same recurrences in chunks of 64 tokens
+long long chunk_ws_bytes(int B, int n, int H, int dk, int dv);
+int launch_chunk_decay(const DecayAttnArgs& a, void* ws, long long ws_bytes, cudaStream_t stream);
+int launch_chunk_delta(const DeltaRuleArgs& a, void* ws, long long ws_bytes, cudaStream_t stream);
 int launch_recurrent_decay(int dtype, const DecayAttnArgs& a, cudaStream_t stream);
 using AttnPrepArgs = plz_attn_prep_t;
 int launch_attn_prep(int dtype, const AttnPrepArgs& a, cudaStream_t stream);

@@ -1,0 +1,642 @@
+// Chunked form of the two linear recurrences (prompts of bf16 models), 64 tokens per chunk. With b_i the cumulative log decay inside a
+// chunk (per key channel; inclusive), S0 the state at its start, and all of it exact algebra on the token-by-token rule:
+//
+//   u_i = beta_i (v_i - S0^T (k_i e^{b_i}) - sum_{j<i} A'_ij u_j),      A'_ij = sum_c k_i k_j e^{b_i - b_j}
+//   =>  U = T beta V - (T beta Kbar) S0 = U0 - W S0,                    T = (I + tril(beta A', -1))^{-1},  Kbar_i = k_i e^{b_i}
+//   o_i = S0^T (q_i e^{b_i}) + sum_{j<=i} M_ij u_j,                     M_ij = sum_c q_i k_j e^{b_i - b_j}
+//   S1  = diag(e^{b_C}) S0 + sum_j (k_j e^{b_C - b_j}) u_j^T
+//
+// (decayed linear attention: u = v, no W, scalar decay). Two launches per segment of chunks:
+//   delta_chunk_kernel / decay_chunk_kernel   one CTA per (chunk, head, sequence), all in parallel: -W, U0, Q~, K~, M, e^{b_C}
+//   chunk_scan_kernel                         one CTA per (64 value columns, head, sequence) walks the chunks in order.
+//
+// Exponents of decays are never positive: products e^{b_i - b_j} = e^{b_i - r} e^{r - b_j} use a reference r between the two tokens (the
+// token before the 16- or 8-row block of i), and pairs inside one 8-row block are evaluated directly. So a decay of any strength
+// underflows to zero and nothing overflows.
+//
+// The recurrence is fp32: every operand of a product is split into two bf16 terms (hi + lo) and the product takes the three terms
+// hi hi + hi lo + lo hi, i.e. about 16 bits of mantissa, with fp32 accumulation and an fp32 state. The products are 16 x 8 x 16
+// mma.sync on register fragments: the blocks here are 8 to 16 rows, the state of the scan has to leave the accumulator and come back as
+// an operand at every chunk, and with the state held TRANSPOSED (value rows x key columns) the accumulator layout IS the operand layout,
+// so a chunk costs no trip of state or U through shared or tensor memory.
+#include "seq_math.cuh"
+
+namespace plz {
+namespace {
+
+constexpr int kC = 64;                     // tokens per chunk
+constexpr float kL2e = 1.4426950408889634f;
+
+__device__ __forceinline__ float ex2a(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
+
+// (x, y) -> bf16 pairs hi, lo with x ~ hi.x + lo.x
+__device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
+    hi = pack_bf16x2(x, y);
+    lo = pack_bf16x2(x - __uint_as_float(hi << 16), y - __uint_as_float(hi & 0xFFFF0000u));
+}
+__device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+struct AFrag { uint32_t h[4], l[4]; };
+__device__ __forceinline__ void mma_split(float (&d)[4], const AFrag& a, uint32_t bh0, uint32_t bh1, uint32_t bl0, uint32_t bl1) {
+    mma16816(d, a.h, bh0, bh1);
+    mma16816(d, a.h, bl0, bl1);
+    mma16816(d, a.l, bh0, bh1);
+}
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void cp16(uint32_t dst, const void* src) { asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory"); }
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+// Workspace of one (sequence, head, chunk): bf16 planes (hi, lo) of -W, Q~, K~ [64][DK] and M [64][64], then fp32 U0 [64][DVP], e^{b_C} [DK]
+template <int DK>
+struct Ws {
+    static constexpr int PLANE = kC * DK;                      // bf16 elements
+    static constexpr int W = 0, Q = 2 * PLANE, M = 4 * PLANE, K = M + 2 * kC * kC, U_BYTES = (K + 2 * PLANE) * 2;
+    static __host__ __device__ long long bytes(int dvp) { return (long long)U_BYTES + (long long)kC * dvp * 4 + DK * 4; }
+};
+__device__ __forceinline__ void put_split(__nv_bfloat16* plane, int stride, int at, float x, float y) {
+    uint32_t h, l;
+    split2(x, y, h, l);
+    *reinterpret_cast<uint32_t*>(plane + at) = h;
+    *reinterpret_cast<uint32_t*>(plane + stride + at) = l;
+}
+
+struct ChunkParams {
+    // delta: fp32 q, k [rows, G * dk], v [rows, H * dv], logg [rows, H * dk], beta [rows, H]; decay: bf16 slices, pitch ld
+    const void* q; const void* k; const void* v; long long ld;
+    const float* logg; const float* beta; const float* decay;
+    float* state; float* o;
+    uint8_t* ws; long long ws_stride;
+    int n, t_begin, chunks;      // tokens per sequence; first token and number of chunks of this segment
+    int H, G, dk, dv, dvp;
+};
+
+// ---------------------------------------------------------------------------------------------------------------------
+// gated delta rule, per chunk
+// ---------------------------------------------------------------------------------------------------------------------
+template <int DK>
+struct DeltaSmem {
+    static constexpr int PK = DK + 4, PT = kC + 4;
+    float k[kC][PK], b[kC][PK];      // keys; cumulative log2 decay
+    float a[kC][PT], t[kC][PT];      // beta A' (strictly lower); T
+    float tmp[4][16][20];
+    float beta[kC];
+};
+
+template <int DK>
+__global__ void __launch_bounds__(128)
+delta_chunk_kernel(const ChunkParams p) {
+    extern __shared__ uint8_t sm_raw[];
+    DeltaSmem<DK>& s = *reinterpret_cast<DeltaSmem<DK>*>(sm_raw);
+    constexpr int KS = DK / 16;
+    const int tid = threadIdx.x, w = tid >> 5, lane = tid & 31, r4 = lane >> 2, c2 = (lane & 3) * 2;
+    const int ch = blockIdx.x, h = blockIdx.y, b = blockIdx.z, hk = h / (p.H / p.G);
+    const int t0 = p.t_begin + ch * kC, L = min(kC, p.n - t0);
+    const long long row0 = (long long)b * p.n + t0;
+    uint8_t* ws = p.ws + (((long long)b * p.H + h) * p.chunks + ch) * p.ws_stride;
+    __nv_bfloat16* wb = reinterpret_cast<__nv_bfloat16*>(ws);
+    float* U0 = reinterpret_cast<float*>(ws + Ws<DK>::U_BYTES);
+    const float* qg = (const float*)p.q + (row0 * p.G + hk) * p.dk;        // row pitch G * dk
+    const long long ldq = (long long)p.G * p.dk;
+
+    for (int e = tid; e < kC * DK; e += 128) {
+        const int t = e / DK, c = e % DK;
+        const bool in = t < L && c < p.dk;
+        s.k[t][c] = in ? ((const float*)p.k)[((row0 + t) * p.G + hk) * p.dk + c] : 0.f;
+        s.b[t][c] = in ? p.logg[((row0 + t) * p.H + h) * p.dk + c] * kL2e : 0.f;
+    }
+    if (tid < kC) s.beta[tid] = tid < L ? p.beta[(row0 + tid) * p.H + h] : 0.f;
+    __syncthreads();
+    if (tid < DK) {
+        float run = 0.f;
+        for (int t = 0; t < kC; ++t) { run += s.b[t][tid]; s.b[t][tid] = run; }
+    }
+    __syncthreads();
+
+    // ---- A' and M: warp w takes rows 16 w .. 16 w + 15 -----------------------------------------------------------------
+    auto q_at = [&](int t, int c) { return (t < L && c < p.dk) ? __ldg(qg + t * ldq + c) : 0.f; };
+    const int i0 = 16 * w + r4, i1 = i0 + 8;
+    // blocks left of the diagonal blocks of this warp (reference: token 16 w - 1), then rows 8..15 against columns 0..7 (reference 16 w + 7)
+    for (int part = 0; part < 2; ++part) {
+        if (part == 0 && w == 0) continue;
+        const int ref = part == 0 ? 16 * w - 1 : 16 * w + 7;
+        const int nt0 = part == 0 ? 0 : 2 * w, ntn = part == 0 ? 2 * w : 1;
+        float kk[6][4], qk[6][4];
+#pragma unroll
+        for (int i = 0; i < 6; ++i)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) { kk[i][e] = 0.f; qk[i][e] = 0.f; }
+#pragma unroll 1
+        for (int ks = 0; ks < KS; ++ks) {
+            AFrag ak, aq;
+            float rr[4];
+#pragma unroll
+            for (int x = 0; x < 4; ++x) rr[x] = s.b[ref][ks * 16 + c2 + (x & 1) + (x >> 1) * 8];
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {          // k columns c2, c2 + 1 and + 8
+                const int c = ks * 16 + c2 + half * 8;
+                float e00 = 0.f, e01 = 0.f;
+                if (part == 0) { e00 = ex2a(s.b[i0][c] - rr[half * 2]); e01 = ex2a(s.b[i0][c + 1] - rr[half * 2 + 1]); }
+                const float e10 = ex2a(s.b[i1][c] - rr[half * 2]), e11 = ex2a(s.b[i1][c + 1] - rr[half * 2 + 1]);
+                split2(s.k[i0][c] * e00, s.k[i0][c + 1] * e01, ak.h[half * 2], ak.l[half * 2]);
+                split2(s.k[i1][c] * e10, s.k[i1][c + 1] * e11, ak.h[half * 2 + 1], ak.l[half * 2 + 1]);
+                split2(q_at(i0, c) * e00, q_at(i0, c + 1) * e01, aq.h[half * 2], aq.l[half * 2]);
+                split2(q_at(i1, c) * e10, q_at(i1, c + 1) * e11, aq.h[half * 2 + 1], aq.l[half * 2 + 1]);
+            }
+#pragma unroll
+            for (int i = 0; i < 6; ++i) {
+                if (i < ntn) {
+                    const int j = (nt0 + i) * 8 + r4, c = ks * 16 + c2;
+                    uint32_t bh0, bl0, bh1, bl1;
+                    split2(s.k[j][c] * ex2a(rr[0] - s.b[j][c]), s.k[j][c + 1] * ex2a(rr[1] - s.b[j][c + 1]), bh0, bl0);
+                    split2(s.k[j][c + 8] * ex2a(rr[2] - s.b[j][c + 8]), s.k[j][c + 9] * ex2a(rr[3] - s.b[j][c + 9]), bh1, bl1);
+                    mma_split(kk[i], ak, bh0, bh1, bl0, bl1);
+                    mma_split(qk[i], aq, bh0, bh1, bl0, bl1);
+                }
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < 6; ++i) {
+            if (i < ntn) {
+                const int j = (nt0 + i) * 8 + c2;
+                if (part == 0) {
+                    s.a[i0][j] = kk[i][0] * s.beta[i0]; s.a[i0][j + 1] = kk[i][1] * s.beta[i0];
+                    put_split(wb + Ws<DK>::M, kC * kC, i0 * kC + j, qk[i][0], qk[i][1]);
+                }
+                s.a[i1][j] = kk[i][2] * s.beta[i1]; s.a[i1][j + 1] = kk[i][3] * s.beta[i1];
+                put_split(wb + Ws<DK>::M, kC * kC, i1 * kC + j, qk[i][2], qk[i][3]);
+            }
+        }
+    }
+    // pairs inside the two 8-row diagonal blocks: lane = (row, one of four channel slices), all exponents explicit
+    for (int blk = 0; blk < 2; ++blk) {
+        const int base = 16 * w + 8 * blk, row = base + (lane & 7), quarter = lane >> 3;
+        float ak[8], aq[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) { ak[j] = 0.f; aq[j] = 0.f; }
+#pragma unroll 1
+        for (int c4 = quarter; c4 < DK / 4; c4 += 4) {
+            const int c = c4 * 4;
+            const float4 bi = *reinterpret_cast<const float4*>(&s.b[row][c]), ki = *reinterpret_cast<const float4*>(&s.k[row][c]);
+            const float q0 = q_at(row, c), q1 = q_at(row, c + 1), q2 = q_at(row, c + 2), q3 = q_at(row, c + 3);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                const float4 bj = *reinterpret_cast<const float4*>(&s.b[base + j][c]), kj = *reinterpret_cast<const float4*>(&s.k[base + j][c]);
+                // j > row: discarded below (the exponent would be positive; clamp it so that nothing overflows)
+                const float e0 = ex2a(fminf(bi.x - bj.x, 0.f)) * kj.x, e1 = ex2a(fminf(bi.y - bj.y, 0.f)) * kj.y;
+                const float e2 = ex2a(fminf(bi.z - bj.z, 0.f)) * kj.z, e3 = ex2a(fminf(bi.w - bj.w, 0.f)) * kj.w;
+                ak[j] += ki.x * e0 + ki.y * e1 + ki.z * e2 + ki.w * e3;
+                aq[j] += q0 * e0 + q1 * e1 + q2 * e2 + q3 * e3;
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            ak[j] += __shfl_xor_sync(0xFFFFFFFFu, ak[j], 8); ak[j] += __shfl_xor_sync(0xFFFFFFFFu, ak[j], 16);
+            aq[j] += __shfl_xor_sync(0xFFFFFFFFu, aq[j], 8); aq[j] += __shfl_xor_sync(0xFFFFFFFFu, aq[j], 16);
+        }
+        const int ri = lane & 7;
+        if (quarter == 0) {
+#pragma unroll
+            for (int j = 0; j < 8; ++j) s.a[row][base + j] = j < ri ? ak[j] * s.beta[row] : 0.f;
+        } else if (quarter == 1) {
+#pragma unroll
+            for (int j = 0; j < 8; j += 2)
+                put_split(wb + Ws<DK>::M, kC * kC, row * kC + base + j, j <= ri ? aq[j] : 0.f, j + 1 <= ri ? aq[j + 1] : 0.f);
+        } else if (quarter == 2 && blk == 0) {
+            // rows 0..7 against columns 8..15 of the 16-row block lie above the diagonal
+#pragma unroll
+            for (int j = 0; j < 8; j += 2) put_split(wb + Ws<DK>::M, kC * kC, row * kC + base + 8 + j, 0.f, 0.f);
+        }
+    }
+    __syncthreads();
+
+    // ---- T = (I + a)^{-1}: 16-row diagonal blocks by substitution, then block diagonals outwards -------------------------
+    if (lane < 16) {
+        float x[16];
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+            float v = i == lane ? 1.f : 0.f;
+#pragma unroll
+            for (int j = 0; j < i; ++j) v = fmaf(-s.a[16 * w + i][16 * w + j], x[j], v);
+            x[i] = v;
+        }
+#pragma unroll
+        for (int i = 0; i < 16; ++i) s.t[16 * w + i][16 * w + lane] = x[i];
+    }
+    __syncthreads();
+    for (int d = 1; d < 4; ++d) {
+        if (w + d < 4) {
+            const int J = w, I = w + d, col = lane & 15, rh = (lane >> 4) * 8;
+            float acc[8];
+#pragma unroll
+            for (int i = 0; i < 8; ++i) acc[i] = 0.f;
+            for (int K = J; K < I; ++K)
+#pragma unroll 4
+                for (int kk = 0; kk < 16; ++kk) {
+                    const float tv = s.t[16 * K + kk][16 * J + col];
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) acc[i] = fmaf(s.a[16 * I + rh + i][16 * K + kk], tv, acc[i]);
+                }
+#pragma unroll
+            for (int i = 0; i < 8; ++i) s.tmp[w][rh + i][col] = acc[i];
+            __syncwarp();
+#pragma unroll
+            for (int i = 0; i < 8; ++i) acc[i] = 0.f;
+#pragma unroll 4
+            for (int kk = 0; kk < 16; ++kk) {
+                const float pv = s.tmp[w][kk][col];
+#pragma unroll
+                for (int i = 0; i < 8; ++i) acc[i] = fmaf(s.t[16 * I + rh + i][16 * I + kk], pv, acc[i]);
+            }
+#pragma unroll
+            for (int i = 0; i < 8; ++i) s.t[16 * I + rh + i][16 * J + col] = -acc[i];
+        }
+        __syncthreads();
+    }
+
+    // ---- -W = -(T beta) Kbar and U0 = (T beta) V; a warp takes every fourth 8-column tile ---------------------------------
+    AFrag at[10];     // (m, ks) with ks <= m
+#pragma unroll
+    for (int m = 0; m < 4; ++m)
+#pragma unroll
+        for (int ks = 0; ks <= m; ++ks) {
+            AFrag& f = at[m * (m + 1) / 2 + ks];
+#pragma unroll
+            for (int x = 0; x < 4; ++x) {
+                const int i = 16 * m + r4 + (x & 1) * 8, j = 16 * ks + c2 + (x >> 1) * 8;
+                split2(s.t[i][j] * s.beta[j], s.t[i][j + 1] * s.beta[j + 1], f.h[x], f.l[x]);
+            }
+        }
+    const int nt_w = DK / 8, nt_all = nt_w + p.dvp / 8;
+#pragma unroll 1
+    for (int nt = w; nt < nt_all; nt += 4) {
+        const bool is_w = nt < nt_w;
+        const int c = (is_w ? nt : nt - nt_w) * 8 + r4;
+        float acc[4][4];
+#pragma unroll
+        for (int m = 0; m < 4; ++m)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) acc[m][e] = 0.f;
+#pragma unroll
+        for (int ks = 0; ks < 4; ++ks) {
+            float f[4];
+#pragma unroll
+            for (int x = 0; x < 4; ++x) {
+                const int j = 16 * ks + c2 + (x & 1) + (x >> 1) * 8;
+                if (is_w) f[x] = -s.k[j][c] * ex2a(s.b[j][c]);
+                else f[x] = (j < L && c < p.dv) ? __ldg((const float*)p.v + ((row0 + j) * p.H + h) * (long long)p.dv + c) : 0.f;
+            }
+            uint32_t bh0, bl0, bh1, bl1;
+            split2(f[0], f[1], bh0, bl0);
+            split2(f[2], f[3], bh1, bl1);
+#pragma unroll
+            for (int m = 0; m < 4; ++m)
+                if (ks <= m) mma_split(acc[m], at[m * (m + 1) / 2 + ks], bh0, bh1, bl0, bl1);
+        }
+        const int cc = (is_w ? nt : nt - nt_w) * 8 + c2;
+#pragma unroll
+        for (int m = 0; m < 4; ++m)
+#pragma unroll
+            for (int hf = 0; hf < 2; ++hf) {
+                const int i = 16 * m + r4 + hf * 8;
+                if (is_w) put_split(wb + Ws<DK>::W, Ws<DK>::PLANE, i * DK + cc, acc[m][hf * 2], acc[m][hf * 2 + 1]);
+                else *reinterpret_cast<float2*>(U0 + (long long)i * p.dvp + cc) = make_float2(acc[m][hf * 2], acc[m][hf * 2 + 1]);
+            }
+    }
+    // ---- Q~, K~, e^{b_C} --------------------------------------------------------------------------------------------------
+    for (int e = tid; e < kC * DK / 2; e += 128) {
+        const int t = e / (DK / 2), c = (e % (DK / 2)) * 2;
+        put_split(wb + Ws<DK>::Q, Ws<DK>::PLANE, t * DK + c, q_at(t, c) * ex2a(s.b[t][c]), q_at(t, c + 1) * ex2a(s.b[t][c + 1]));
+        put_split(wb + Ws<DK>::K, Ws<DK>::PLANE, t * DK + c, s.k[t][c] * ex2a(s.b[kC - 1][c] - s.b[t][c]),
+                  s.k[t][c + 1] * ex2a(s.b[kC - 1][c + 1] - s.b[t][c + 1]));
+    }
+    if (tid < DK) U0[(long long)kC * p.dvp + tid] = ex2a(s.b[kC - 1][tid]);
+}
+
+// ---------------------------------------------------------------------------------------------------------------------
+// decayed linear attention, per chunk
+// ---------------------------------------------------------------------------------------------------------------------
+template <int DK>
+struct DecaySmem {
+    static constexpr int PK = DK + 4;
+    float q[kC][PK], k[kC][PK];
+    float pw[kC + 1];               // powers of the decay
+};
+template <int DK>
+__global__ void __launch_bounds__(128)
+decay_chunk_kernel(const ChunkParams p) {
+    extern __shared__ uint8_t sm_raw[];
+    DecaySmem<DK>& s = *reinterpret_cast<DecaySmem<DK>*>(sm_raw);
+    constexpr int KS = DK / 16;
+    const int tid = threadIdx.x, w = tid >> 5, lane = tid & 31, r4 = lane >> 2, c2 = (lane & 3) * 2;
+    const int ch = blockIdx.x, h = blockIdx.y, b = blockIdx.z;
+    const int t0 = p.t_begin + ch * kC, L = min(kC, p.n - t0);
+    const long long row0 = (long long)b * p.n + t0;
+    uint8_t* ws = p.ws + (((long long)b * p.H + h) * p.chunks + ch) * p.ws_stride;
+    __nv_bfloat16* wb = reinterpret_cast<__nv_bfloat16*>(ws);
+    float* U0 = reinterpret_cast<float*>(ws + Ws<DK>::U_BYTES);
+    const __nv_bfloat16* qg = (const __nv_bfloat16*)p.q + row0 * p.ld + (long long)h * p.dk;
+    const __nv_bfloat16* kg = (const __nv_bfloat16*)p.k + row0 * p.ld + (long long)h * p.dk;
+    const __nv_bfloat16* vg = (const __nv_bfloat16*)p.v + row0 * p.ld + (long long)h * p.dv;
+    if (tid <= kC) s.pw[tid] = powf(p.decay[h], (float)tid);
+    for (int e = tid; e < kC * DK; e += 128) {
+        const int t = e / DK, c = e % DK;
+        const bool in = t < L && c < p.dk;
+        s.q[t][c] = in ? silu_f(to_f(qg[t * p.ld + c])) : 0.f;
+        s.k[t][c] = in ? silu_f(to_f(kg[t * p.ld + c])) : 0.f;
+    }
+    for (int e = tid; e < kC * p.dvp; e += 128) {
+        const int t = e / p.dvp, c = e % p.dvp;
+        U0[e] = (t < L && c < p.dv) ? silu_f(to_f(vg[t * p.ld + c])) : 0.f;
+    }
+    __syncthreads();
+    float acc[8][4];
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
+#pragma unroll 1
+    for (int ks = 0; ks < KS; ++ks) {
+        AFrag a;
+#pragma unroll
+        for (int x = 0; x < 4; ++x) {
+            const int i = 16 * w + r4 + (x & 1) * 8, c = ks * 16 + c2 + (x >> 1) * 8;
+            split2(s.q[i][c], s.q[i][c + 1], a.h[x], a.l[x]);
+        }
+#pragma unroll
+        for (int nt = 0; nt < 8; ++nt) {
+            if (nt < 2 * w + 2) {
+                const int j = nt * 8 + r4, c = ks * 16 + c2;
+                uint32_t bh0, bl0, bh1, bl1;
+                split2(s.k[j][c], s.k[j][c + 1], bh0, bl0);
+                split2(s.k[j][c + 8], s.k[j][c + 9], bh1, bl1);
+                mma_split(acc[nt], a, bh0, bh1, bl0, bl1);
+            }
+        }
+    }
+#pragma unroll
+    for (int nt = 0; nt < 8; ++nt) {
+        if (nt < 2 * w + 2) {
+#pragma unroll
+            for (int hf = 0; hf < 2; ++hf) {
+                const int i = 16 * w + r4 + hf * 8, j = nt * 8 + c2;
+                const float m0 = i >= j ? acc[nt][hf * 2] * s.pw[i - j] : 0.f, m1 = i >= j + 1 ? acc[nt][hf * 2 + 1] * s.pw[i - j - 1] : 0.f;
+                put_split(wb + Ws<DK>::M, kC * kC, i * kC + j, m0, m1);
+            }
+        }
+    }
+    for (int e = tid; e < kC * DK / 2; e += 128) {
+        const int t = e / (DK / 2), c = (e % (DK / 2)) * 2;
+        const float fq = s.pw[t + 1], fk = t < L ? s.pw[L - 1 - t] : 0.f;
+        put_split(wb + Ws<DK>::Q, Ws<DK>::PLANE, t * DK + c, s.q[t][c] * fq, s.q[t][c + 1] * fq);
+        put_split(wb + Ws<DK>::K, Ws<DK>::PLANE, t * DK + c, s.k[t][c] * fk, s.k[t][c + 1] * fk);
+    }
+    if (tid < DK) U0[(long long)kC * p.dvp + tid] = s.pw[L];
+}
+
+// ---------------------------------------------------------------------------------------------------------------------
+// the scan: a warp owns 16 value columns of one head, S^T [16][DK] in its accumulators
+// ---------------------------------------------------------------------------------------------------------------------
+template <int DK, bool HASW>
+struct ScanSmem {
+    static constexpr int P = DK + 8, PM = kC + 8;      // padded rows: ldmatrix without bank conflicts
+    __nv_bfloat16 wq[HASW ? 4 : 2][kC][P];             // -W hi, lo, Q~ hi, lo
+    __nv_bfloat16 k[2][kC][P];
+    __nv_bfloat16 m[2][kC][PM];
+    float dec[DK];
+};
+
+template <int DK, bool HASW>
+__global__ void __launch_bounds__(256)
+chunk_scan_kernel(const ChunkParams p) {
+    extern __shared__ uint8_t sm_raw[];
+    using SM = ScanSmem<DK, HASW>;
+    SM& s = *reinterpret_cast<SM*>(sm_raw);
+    constexpr int KS = DK / 16, NT = DK / 8;
+    const int tid = threadIdx.x, w = tid >> 5, lane = tid & 31, r4 = lane >> 2, c2 = (lane & 3) * 2;
+    const int h = blockIdx.y, b = blockIdx.z;
+    const int col0 = ((int)blockIdx.x * (int)(blockDim.x >> 5) + w) * 16;             // first value column of the warp
+    const bool act = col0 < p.dv;                               // an idle warp still helps to load
+    const int d0 = col0 + r4, d1 = d0 + 8;
+    const uint8_t* ws0 = p.ws + ((long long)b * p.H + h) * p.chunks * p.ws_stride;
+    float* Sg = p.state + ((long long)b * p.H + h) * p.dk * (long long)p.dv;
+
+    auto load_rows = [&](__nv_bfloat16* dst, int pitch, const __nv_bfloat16* src, int width, int planes) {   // planes of [64][width]
+        const int per = width / 8, total = planes * kC * per;
+        for (int e = tid; e < total; e += (int)blockDim.x) {
+            const int row = e / per, c = e - row * per;
+            cp16(smem_u32(dst + (long long)row * pitch + c * 8), src + (long long)row * width + c * 8);
+        }
+    };
+    auto load_wq = [&](int ch) {
+        const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(ws0 + (long long)ch * p.ws_stride);
+        load_rows(&s.wq[0][0][0], SM::P, src + (HASW ? Ws<DK>::W : Ws<DK>::Q), DK, HASW ? 4 : 2);
+    };
+    auto load_mk = [&](int ch) {
+        const uint8_t* base = ws0 + (long long)ch * p.ws_stride;
+        const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(base);
+        load_rows(&s.m[0][0][0], SM::PM, src + Ws<DK>::M, kC, 2);
+        load_rows(&s.k[0][0][0], SM::P, src + Ws<DK>::K, DK, 2);
+        const float* dsrc = reinterpret_cast<const float*>(base + Ws<DK>::U_BYTES) + (long long)kC * p.dvp;
+        if (tid < DK / 4) cp16(smem_u32(&s.dec[tid * 4]), dsrc + tid * 4);
+    };
+    float S[NT][4];
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int c = nt * 8 + c2 + (e & 1), d = e < 2 ? d0 : d1;
+            S[nt][e] = (act && c < p.dk && d < p.dv) ? Sg[(long long)c * p.dv + d] : 0.f;
+        }
+    float u[8][4];
+    auto load_u0 = [&](int ch) {
+        const float* U0 = reinterpret_cast<const float*>(ws0 + (long long)ch * p.ws_stride + Ws<DK>::U_BYTES);
+#pragma unroll
+        for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+                u[nt][e] = act ? __ldcs(U0 + (long long)(nt * 8 + c2 + (e & 1)) * p.dvp + (e < 2 ? d0 : d1)) : 0.f;
+    };
+    load_wq(0); cp_commit();
+    load_mk(0); cp_commit();
+    load_u0(0);
+    // ldmatrix lane addresses: token rows x 16 key columns (two 8-token groups), and for the transposed read 16 tokens x 16 columns
+    const uint32_t lrow = (uint32_t)((lane >> 4) * 8 + (lane & 7)), lcol = (uint32_t)(((lane >> 3) & 1) * 8);
+    const uint32_t trow = (uint32_t)(((lane >> 3) & 1) * 8 + (lane & 7)), tcol = (uint32_t)((lane >> 4) * 8);
+    const uint32_t aWQ = smem_u32(&s.wq[0][lrow][lcol]), aM = smem_u32(&s.m[0][lrow][lcol]), aK = smem_u32(&s.k[0][trow][tcol]);
+    constexpr uint32_t PLANE_B = kC * SM::P * 2, PLANE_M = kC * SM::PM * 2;
+
+    for (int ch = 0; ch < p.chunks; ++ch) {
+        float o[8][4];
+#pragma unroll
+        for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) o[nt][e] = 0.f;
+        cp_wait<1>();
+        __syncthreads();
+        if (act) {
+#pragma unroll
+            for (int ks = 0; ks < KS; ++ks) {
+                AFrag a;
+                split2(S[2 * ks][0], S[2 * ks][1], a.h[0], a.l[0]);
+                split2(S[2 * ks][2], S[2 * ks][3], a.h[1], a.l[1]);
+                split2(S[2 * ks + 1][0], S[2 * ks + 1][1], a.h[2], a.l[2]);
+                split2(S[2 * ks + 1][2], S[2 * ks + 1][3], a.h[3], a.l[3]);
+#pragma unroll
+                for (int np = 0; np < 4; ++np) {
+                    const uint32_t at = aWQ + (uint32_t)(np * 16 * SM::P + ks * 16) * 2;
+                    uint32_t bh[4], bl[4];
+                    if (HASW) {
+                        ldsm4(bh, at); ldsm4(bl, at + PLANE_B);
+                        mma_split(u[2 * np], a, bh[0], bh[1], bl[0], bl[1]);
+                        mma_split(u[2 * np + 1], a, bh[2], bh[3], bl[2], bl[3]);
+                    }
+                    ldsm4(bh, at + (HASW ? 2 : 0) * PLANE_B); ldsm4(bl, at + (HASW ? 3 : 1) * PLANE_B);
+                    mma_split(o[2 * np], a, bh[0], bh[1], bl[0], bl[1]);
+                    mma_split(o[2 * np + 1], a, bh[2], bh[3], bl[2], bl[3]);
+                }
+            }
+        }
+        __syncthreads();
+        if (ch + 1 < p.chunks) load_wq(ch + 1);
+        cp_commit();
+        cp_wait<1>();
+        __syncthreads();
+        if (act) {
+            AFrag ua[4];
+#pragma unroll
+            for (int ks = 0; ks < 4; ++ks) {
+                split2(u[2 * ks][0], u[2 * ks][1], ua[ks].h[0], ua[ks].l[0]);
+                split2(u[2 * ks][2], u[2 * ks][3], ua[ks].h[1], ua[ks].l[1]);
+                split2(u[2 * ks + 1][0], u[2 * ks + 1][1], ua[ks].h[2], ua[ks].l[2]);
+                split2(u[2 * ks + 1][2], u[2 * ks + 1][3], ua[ks].h[3], ua[ks].l[3]);
+            }
+            if (ch + 1 < p.chunks) load_u0(ch + 1);          // lands under the products below
+#pragma unroll
+            for (int ks = 0; ks < 4; ++ks)
+#pragma unroll
+                for (int np = ks; np < 4; ++np) {            // queries at or after the keys' block
+                    const uint32_t at = aM + (uint32_t)(np * 16 * SM::PM + ks * 16) * 2;
+                    uint32_t bh[4], bl[4];
+                    ldsm4(bh, at); ldsm4(bl, at + PLANE_M);
+                    mma_split(o[2 * np], ua[ks], bh[0], bh[1], bl[0], bl[1]);
+                    mma_split(o[2 * np + 1], ua[ks], bh[2], bh[3], bl[2], bl[3]);
+                }
+            const int t0 = p.t_begin + ch * kC, L = min(kC, p.n - t0);
+            float* og = p.o + (((long long)b * p.n + t0) * p.H + h) * p.dv;
+#pragma unroll
+            for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int t = nt * 8 + c2 + (e & 1), d = e < 2 ? d0 : d1;
+                    if (t < L && d < p.dv) og[(long long)t * p.H * p.dv + d] = o[nt][e];
+                }
+#pragma unroll
+            for (int np = 0; np < NT / 2; ++np) {
+#pragma unroll
+                for (int x = 0; x < 2; ++x) {
+                    const float2 dc = *reinterpret_cast<const float2*>(&s.dec[(2 * np + x) * 8 + c2]);
+                    S[2 * np + x][0] *= dc.x; S[2 * np + x][1] *= dc.y; S[2 * np + x][2] *= dc.x; S[2 * np + x][3] *= dc.y;
+                }
+#pragma unroll
+                for (int ks = 0; ks < 4; ++ks) {
+                    const uint32_t at = aK + (uint32_t)(ks * 16 * SM::P + np * 16) * 2;
+                    uint32_t bh[4], bl[4];
+                    ldsm4t(bh, at); ldsm4t(bl, at + PLANE_B);
+                    mma_split(S[2 * np], ua[ks], bh[0], bh[1], bl[0], bl[1]);
+                    mma_split(S[2 * np + 1], ua[ks], bh[2], bh[3], bl[2], bl[3]);
+                }
+            }
+        }
+        __syncthreads();
+        if (ch + 1 < p.chunks) load_mk(ch + 1);
+        cp_commit();
+    }
+    if (act) {
+#pragma unroll
+        for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int c = nt * 8 + c2 + (e & 1), d = e < 2 ? d0 : d1;
+                if (c < p.dk && d < p.dv) Sg[(long long)c * p.dv + d] = S[nt][e];
+            }
+    }
+}
+
+template <int DK, bool DELTA>
+int launch_chunked(ChunkParams p, int B, void* ws, long long ws_bytes, cudaStream_t stream) {
+    p.dvp = (p.dv + 15) / 16 * 16;
+    p.ws = (uint8_t*)ws;
+    p.ws_stride = Ws<DK>::bytes(p.dvp);
+    const long long per_chunk = p.ws_stride * B * p.H;
+    const int all = (p.n + kC - 1) / kC;
+    long long seg = ws_bytes / per_chunk;
+    if (seg < 1) { set_last_error("chunked recurrence: workspace of %lld bytes holds no chunk (%lld needed)", ws_bytes, per_chunk); return PLZ_ERR_WORKSPACE; }
+    if (seg > all) seg = all;
+    const long long rounds = (all + seg - 1) / seg;
+    seg = (all + rounds - 1) / rounds;
+    const int smem1 = DELTA ? (int)sizeof(DeltaSmem<DK>) : (int)sizeof(DecaySmem<DK>), smem2 = (int)sizeof(ScanSmem<DK, DELTA>);
+    static bool once[64] = {};
+    int dev = 0;
+    PLZ_CUDA_CHECK(cudaGetDevice(&dev));
+    if (!once[dev & 63]) {
+        if (DELTA) PLZ_CUDA_CHECK(cudaFuncSetAttribute(delta_chunk_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem1));
+        else PLZ_CUDA_CHECK(cudaFuncSetAttribute(decay_chunk_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem1));
+        PLZ_CUDA_CHECK(cudaFuncSetAttribute((chunk_scan_kernel<DK, DELTA>), cudaFuncAttributeMaxDynamicSharedMemorySize, smem2));
+        once[dev & 63] = true;
+    }
+    for (int c0 = 0; c0 < all; c0 += (int)seg) {
+        p.t_begin = c0 * kC;
+        p.chunks = all - c0 < (int)seg ? all - c0 : (int)seg;
+        if (DELTA) delta_chunk_kernel<DK><<<dim3(p.chunks, p.H, B), 128, smem1, stream>>>(p);
+        else decay_chunk_kernel<DK><<<dim3(p.chunks, p.H, B), 128, smem1, stream>>>(p);
+        PLZ_LAUNCH_CHECK();
+        // four warps (64 value columns) per CTA while that leaves SMs free, else eight on one copy of the chunk's operands
+        const int warps = (long long)B * p.H * ((p.dv + 63) / 64) > seq_sm_count() && p.dv > 64 ? 8 : 4;
+        chunk_scan_kernel<DK, DELTA><<<dim3((p.dv + 16 * warps - 1) / (16 * warps), p.H, B), 32 * warps, smem2, stream>>>(p);
+        PLZ_LAUNCH_CHECK();
+    }
+    return PLZ_OK;
+}
+template <bool DELTA>
+int launch_dk(const ChunkParams& p, int B, void* ws, long long ws_bytes, cudaStream_t stream) {
+    if (p.dk <= 32) return launch_chunked<32, DELTA>(p, B, ws, ws_bytes, stream);
+    if (p.dk <= 64) return launch_chunked<64, DELTA>(p, B, ws, ws_bytes, stream);
+    if (p.dk <= 128) return launch_chunked<128, DELTA>(p, B, ws, ws_bytes, stream);
+    set_last_error("chunked recurrence: key size %d (at most 128)", p.dk);
+    return PLZ_ERR_UNSUPPORTED;
+}
+
+}  // namespace
+
+// bytes that hold every chunk of n tokens; any amount down to one chunk of all heads works (the scan then runs in segments)
+long long chunk_ws_bytes(int B, int n, int H, int dk, int dv) {
+    if (dk > 128) return 0;
+    const int dvp = (dv + 15) / 16 * 16, DK = dk <= 32 ? 32 : (dk <= 64 ? 64 : 128);
+    const long long per = DK == 32 ? Ws<32>::bytes(dvp) : (DK == 64 ? Ws<64>::bytes(dvp) : Ws<128>::bytes(dvp));
+    const long long one = per * B * H, all = one * ((n + kC - 1) / kC), cap = 96ll << 20;   // stay inside L2 when there is a choice
+    return all <= cap ? all : (one > cap ? one : cap / one * one);
+}
+
+int launch_chunk_decay(const DecayAttnArgs& a, void* ws, long long ws_bytes, cudaStream_t stream) {
+    ChunkParams p = {};
+    p.q = a.q; p.k = a.k; p.v = a.v; p.ld = a.ld; p.decay = a.decay; p.state = a.state; p.o = a.o;
+    p.n = a.n; p.H = a.H; p.G = a.H; p.dk = a.dk; p.dv = a.dv;
+    return launch_dk<false>(p, a.B, ws, ws_bytes, stream);
+}
+int launch_chunk_delta(const DeltaRuleArgs& a, void* ws, long long ws_bytes, cudaStream_t stream) {
+    ChunkParams p = {};
+    p.q = a.q; p.k = a.k; p.v = a.v; p.logg = a.logg; p.beta = a.beta; p.state = a.state; p.o = a.o;
+    p.n = a.n; p.H = a.H; p.G = a.G; p.dk = a.dk; p.dv = a.dv;
+    return launch_dk<true>(p, a.B, ws, ws_bytes, stream);
+}
+
+}  // namespace plz

@@ -75,6 +75,13 @@ class Loader:
         return w, b, offs
 
 
+CHUNK_FROM = 64     # portions of at least this many tokens take the chunked recurrence (bf16 models)
+
+
+def _chunked(x: torch.Tensor, n: int) -> bool:
+    return n >= CHUNK_FROM and x.dtype == torch.bfloat16
+
+
 class Lightning:
     """Per head S <- decay S + k v^T, o = S^T q, with q, k, v = silu of their projections."""
 
@@ -93,7 +100,8 @@ class Lightning:
     def forward(self, x: torch.Tensor, st: dict, ctx: StepContext) -> torch.Tensor:
         qk, v, (oq, ok, ov, og) = self.H * self.dk, self.H * self.dv, self.off
         p = S.linear(x, self.w_in)
-        o = S.decay_attention(p[:, oq:oq + qk], p[:, ok:ok + qk], p[:, ov:ov + v], self.decay, st["S"], ctx.B, ctx.n, self.H, self.dk, self.dv)
+        o = S.decay_attention(p[:, oq:oq + qk], p[:, ok:ok + qk], p[:, ov:ov + v], self.decay, st["S"], ctx.B, ctx.n, self.H, self.dk, self.dv,
+                              _chunked(x, ctx.n))
         return S.linear(S.norm_gate(o, p[:, og:og + v], self.norm, ctx.eps, 1), self.w_out)
 
 
@@ -127,7 +135,7 @@ class ChannelDelta:
         gate = S.linear(p[:, og:og + self.rg], self.w_g2)
         q, k, v, logg, beta = S.delta_prep(p, (oq, ok, ov, ob), a, self.conv, self.A_log, self.dt_bias, st.get("conv"), ctx.B, ctx.n, self.H, self.G,
                                            self.dk, self.dv, self.dk ** -0.5)
-        o = S.delta_rule(q, k, v, logg, beta, st["S"], ctx.B, ctx.n, self.H, self.G, self.dk, self.dv)
+        o = S.delta_rule(q, k, v, logg, beta, st["S"], ctx.B, ctx.n, self.H, self.G, self.dk, self.dv, _chunked(x, ctx.n))
         return S.linear(S.norm_gate(o, gate, self.norm, ctx.eps, self.H), self.w_out)
 
 

@@ -143,8 +143,9 @@ SIGNATURES = {
     "plz_seq_rows_norm": [_I32, _P, _P, _P, _F, _F, _I64, _I32, _P, _P],
     "plz_seq_norm_gate": [_I32, _P, _P, _I64, _P, _F, _I64, _I32, _I32, _P, _P],
     "plz_delta_prep": [_I32, C.POINTER(DeltaPrep), _P],
-    "plz_delta_rule": [C.POINTER(DeltaRule), _P],
-    "plz_decay_attn": [_I32, C.POINTER(DecayAttn), _P],
+    "plz_chunk_ws_bytes": [_I32, _I32, _I32, _I32, _I32],
+    "plz_delta_rule": [C.POINTER(DeltaRule), _P, _I64, _P],
+    "plz_decay_attn": [_I32, C.POINTER(DecayAttn), _P, _I64, _P],
     "plz_attn_prep": [_I32, C.POINTER(AttnPrep), _P],
     "plz_attn_bias_ws_bytes": [_I32, _I32, _I32, _I32, _I32],
     "plz_attn_bias": [_I32, C.POINTER(AttnBias), _P, _I64, _P],
@@ -153,7 +154,7 @@ SIGNATURES = {
     "plz_distill_loss": [_P, _I64, _P, _I64, _I32, _I32, _F, _F, _F, _P, _P, _P, _I64, _I32, _P],
 }
 _RESTYPES = {"plz_last_error": C.c_char_p, "plz_launch_count": C.c_uint64, "plz_attn_decode_ws_bytes": C.c_int64,
-             "plz_attn_bias_ws_bytes": C.c_int64}
+             "plz_attn_bias_ws_bytes": C.c_int64, "plz_chunk_ws_bytes": C.c_int64}
 
 
 def lib():

@@ -83,21 +83,30 @@ def delta_prep(proj: torch.Tensor, offs, a: torch.Tensor, taps: torch.Tensor, A_
     return q, k, v, lg, beta
 
 
-def delta_rule(q, k, v, logg, beta, state: torch.Tensor, B: int, n: int, H: int, G: int, dk: int, dv: int) -> torch.Tensor:
-    """o fp32 [B * n, H * dv]; state fp32 [B, H, dk, dv] in place."""
+def _chunk_ws(chunked: bool, B, n, H, dk, dv, device):
+    need = P.lib().plz_chunk_ws_bytes(B, n, H, dk, dv) if chunked else 0
+    return (torch.empty(need, dtype=torch.uint8, device=device), need) if need else (None, 0)
+
+
+def delta_rule(q, k, v, logg, beta, state: torch.Tensor, B: int, n: int, H: int, G: int, dk: int, dv: int, chunked: bool = False) -> torch.Tensor:
+    """o fp32 [B * n, H * dv]; state fp32 [B, H, dk, dv] in place. chunked: 64 tokens at a time on the tensor cores (dk <= 128; larger
+    key sizes run token by token)."""
+    ws, need = _chunk_ws(chunked, B, n, H, dk, dv, state.device)
     o = torch.empty(B * n, H * dv, dtype=torch.float32, device=state.device)
     d = P.DeltaRule(q.data_ptr(), k.data_ptr(), v.data_ptr(), logg.data_ptr(), beta.data_ptr(), state.data_ptr(), o.data_ptr(), B, n, H, G, dk, dv)
-    P.check(P.lib().plz_delta_rule(C.byref(d), P.stream_ptr()), "plz_delta_rule")
+    P.check(P.lib().plz_delta_rule(C.byref(d), _ptr(ws), need, P.stream_ptr()), "plz_delta_rule")
     return o
 
 
 def decay_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, B: int, n: int, H: int, dk: int,
-                    dv: int) -> torch.Tensor:
-    """q, k, v: slices (before silu) of one projection; o fp32 [B * n, H * dv]; state fp32 [B, H, dk, dv] in place."""
+                    dv: int, chunked: bool = False) -> torch.Tensor:
+    """q, k, v: slices (before silu) of one projection; o fp32 [B * n, H * dv]; state fp32 [B, H, dk, dv] in place. chunked: as in
+    delta_rule (bf16 projections)."""
+    ws, need = _chunk_ws(chunked, B, n, H, dk, dv, state.device)
     assert q.stride(0) == k.stride(0) == v.stride(0)
     o = torch.empty(B * n, H * dv, dtype=torch.float32, device=state.device)
     d = P.DecayAttn(q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), decay.data_ptr(), state.data_ptr(), o.data_ptr(), B, n, H, dk, dv)
-    P.check(P.lib().plz_decay_attn(code(q.dtype), C.byref(d), P.stream_ptr()), "plz_decay_attn")
+    P.check(P.lib().plz_decay_attn(code(q.dtype), C.byref(d), _ptr(ws), need, P.stream_ptr()), "plz_decay_attn")
     return o
 
 
