@@ -1170,8 +1170,10 @@ def main():
     ap.add_argument("--no-parity", action="store_true", help="N > 1: skip the correctness check of the fused exchange that runs before the timed region")
     ap.add_argument("--sustained-s", type=float, default=3.0, help="length of the sustained leg in seconds (0 = off)")
     ap.add_argument("--pair-gemm", type=int, default=1, help="0: keep the large products on the one-CTA-per-tile kernels (comparison)")
-    ap.add_argument("--workload", default="linear", choices=["linear", "distill"],
-                    help="linear (default): the benchmark step of one Linear; distill: the super-block distillation step (its own JSON line)")
+    ap.add_argument("--workload", default="linear", choices=["linear", "distill", "hybrid"],
+                    help="linear (default): the benchmark step of one Linear; distill: the super-block distillation step (its own JSON line); "
+                         "hybrid: prefill and decode of the Gopunex decoder beside PalettizedQwen at equal size, and a per-kernel table (JSON lines)")
+    ap.add_argument("--sizes", default="small,medium,large", help="--workload hybrid: which of the sizes small, medium, large")
     ap.add_argument("--case", default=None, help="run ONE kernel of the hot path a few times on a small case and exit (for ncu captures)")
     ap.add_argument("--kernels", action="store_true", help="per-kernel table: one JSON line per measurement")
     ap.add_argument("--M", type=int, default=4096)
@@ -1189,6 +1191,9 @@ def main():
     args = ap.parse_args()
     if args.workload == "distill":
         run_distill(args)
+    elif args.workload == "hybrid":
+        import bench_hybrid
+        bench_hybrid.run(args, peaks(), ClockSampler)
     elif args.case:
         run_case(args)
     elif args.kernels:

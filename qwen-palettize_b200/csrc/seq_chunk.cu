@@ -29,6 +29,8 @@ constexpr float kL2e = 1.4426950408889634f;
 
 __device__ __forceinline__ float ex2a(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
 
+// z / (1 + e^-z) of a bf16 input, about 2^-21 relative
+__device__ __forceinline__ float silu_fast(float z) { return __fdividef(z, 1.0f + ex2a(-z * kL2e)); }
 // (x, y) -> bf16 pairs hi, lo with x ~ hi.x + lo.x
 __device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
     hi = pack_bf16x2(x, y);
@@ -69,6 +71,14 @@ __device__ __forceinline__ void put_split(__nv_bfloat16* plane, int stride, int 
     *reinterpret_cast<uint32_t*>(plane + stride + at) = l;
 }
 
+__device__ __forceinline__ void put_split4(__nv_bfloat16* plane, int stride, int at, float x, float y, float z, float w) {
+    uint2 h, l;
+    split2(x, y, h.x, l.x);
+    split2(z, w, h.y, l.y);
+    *reinterpret_cast<uint2*>(plane + at) = h;
+    *reinterpret_cast<uint2*>(plane + stride + at) = l;
+}
+
 struct ChunkParams {
     // delta: fp32 q, k [rows, G * dk], v [rows, H * dv], logg [rows, H * dk], beta [rows, H]; decay: bf16 slices, pitch ld
     const void* q; const void* k; const void* v; long long ld;
@@ -77,6 +87,7 @@ struct ChunkParams {
     uint8_t* ws; long long ws_stride;
     int n, t_begin, chunks;      // tokens per sequence; first token and number of chunks of this segment
     int H, G, dk, dv, dvp;
+    int vec;                     // rows allow 16-byte loads
 };
 
 // ---------------------------------------------------------------------------------------------------------------------
@@ -107,22 +118,48 @@ delta_chunk_kernel(const ChunkParams p) {
     const float* qg = (const float*)p.q + (row0 * p.G + hk) * p.dk;        // row pitch G * dk
     const long long ldq = (long long)p.G * p.dk;
 
-    for (int e = tid; e < kC * DK; e += 128) {
-        const int t = e / DK, c = e % DK;
-        const bool in = t < L && c < p.dk;
-        s.k[t][c] = in ? ((const float*)p.k)[((row0 + t) * p.G + hk) * p.dk + c] : 0.f;
-        s.b[t][c] = in ? p.logg[((row0 + t) * p.H + h) * p.dk + c] * kL2e : 0.f;
+    const float* kg = (const float*)p.k + (row0 * p.G + hk) * p.dk;
+    const float* gg = p.logg + (row0 * p.H + h) * p.dk;
+    const long long ldg = (long long)p.H * p.dk;
+    if (p.vec) {
+#pragma unroll 8
+        for (int e = tid; e < kC * DK / 4; e += 128) {
+            const int t = e / (DK / 4), c = (e % (DK / 4)) * 4;
+            float4 kv = make_float4(0.f, 0.f, 0.f, 0.f), gv = kv;
+            if (t < L && c < p.dk) {
+                kv = __ldg(reinterpret_cast<const float4*>(kg + t * ldq + c));
+                gv = __ldg(reinterpret_cast<const float4*>(gg + t * ldg + c));
+            }
+            *reinterpret_cast<float4*>(&s.k[t][c]) = kv;
+            *reinterpret_cast<float4*>(&s.b[t][c]) = make_float4(gv.x * kL2e, gv.y * kL2e, gv.z * kL2e, gv.w * kL2e);
+        }
+    } else {
+        for (int e = tid; e < kC * DK; e += 128) {
+            const int t = e / DK, c = e % DK;
+            const bool in = t < L && c < p.dk;
+            s.k[t][c] = in ? kg[t * ldq + c] : 0.f;
+            s.b[t][c] = in ? gg[t * ldg + c] * kL2e : 0.f;
+        }
     }
     if (tid < kC) s.beta[tid] = tid < L ? p.beta[(row0 + tid) * p.H + h] : 0.f;
     __syncthreads();
     if (tid < DK) {
         float run = 0.f;
+#pragma unroll 16
         for (int t = 0; t < kC; ++t) { run += s.b[t][tid]; s.b[t][tid] = run; }
     }
     __syncthreads();
 
     // ---- A' and M: warp w takes rows 16 w .. 16 w + 15 -----------------------------------------------------------------
     auto q_at = [&](int t, int c) { return (t < L && c < p.dk) ? __ldg(qg + t * ldq + c) : 0.f; };
+    auto q_at2 = [&](int t, int c) {      // c even
+        if (!p.vec) return make_float2(q_at(t, c), q_at(t, c + 1));
+        return (t < L && c < p.dk) ? __ldg(reinterpret_cast<const float2*>(qg + t * ldq + c)) : make_float2(0.f, 0.f);
+    };
+    auto q_at4 = [&](int t, int c) {      // c a multiple of four
+        if (!p.vec) return make_float4(q_at(t, c), q_at(t, c + 1), q_at(t, c + 2), q_at(t, c + 3));
+        return (t < L && c < p.dk) ? __ldg(reinterpret_cast<const float4*>(qg + t * ldq + c)) : make_float4(0.f, 0.f, 0.f, 0.f);
+    };
     const int i0 = 16 * w + r4, i1 = i0 + 8;
     // blocks left of the diagonal blocks of this warp (reference: token 16 w - 1), then rows 8..15 against columns 0..7 (reference 16 w + 7)
     for (int part = 0; part < 2; ++part) {
@@ -148,8 +185,9 @@ delta_chunk_kernel(const ChunkParams p) {
                 const float e10 = ex2a(s.b[i1][c] - rr[half * 2]), e11 = ex2a(s.b[i1][c + 1] - rr[half * 2 + 1]);
                 split2(s.k[i0][c] * e00, s.k[i0][c + 1] * e01, ak.h[half * 2], ak.l[half * 2]);
                 split2(s.k[i1][c] * e10, s.k[i1][c + 1] * e11, ak.h[half * 2 + 1], ak.l[half * 2 + 1]);
-                split2(q_at(i0, c) * e00, q_at(i0, c + 1) * e01, aq.h[half * 2], aq.l[half * 2]);
-                split2(q_at(i1, c) * e10, q_at(i1, c + 1) * e11, aq.h[half * 2 + 1], aq.l[half * 2 + 1]);
+                const float2 qa = q_at2(i0, c), qb = q_at2(i1, c);
+                split2(qa.x * e00, qa.y * e01, aq.h[half * 2], aq.l[half * 2]);
+                split2(qb.x * e10, qb.y * e11, aq.h[half * 2 + 1], aq.l[half * 2 + 1]);
             }
 #pragma unroll
             for (int i = 0; i < 6; ++i) {
@@ -186,7 +224,7 @@ delta_chunk_kernel(const ChunkParams p) {
         for (int c4 = quarter; c4 < DK / 4; c4 += 4) {
             const int c = c4 * 4;
             const float4 bi = *reinterpret_cast<const float4*>(&s.b[row][c]), ki = *reinterpret_cast<const float4*>(&s.k[row][c]);
-            const float q0 = q_at(row, c), q1 = q_at(row, c + 1), q2 = q_at(row, c + 2), q3 = q_at(row, c + 3);
+            const float4 qi = q_at4(row, c);
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
                 const float4 bj = *reinterpret_cast<const float4*>(&s.b[base + j][c]), kj = *reinterpret_cast<const float4*>(&s.k[base + j][c]);
@@ -194,7 +232,7 @@ delta_chunk_kernel(const ChunkParams p) {
                 const float e0 = ex2a(fminf(bi.x - bj.x, 0.f)) * kj.x, e1 = ex2a(fminf(bi.y - bj.y, 0.f)) * kj.y;
                 const float e2 = ex2a(fminf(bi.z - bj.z, 0.f)) * kj.z, e3 = ex2a(fminf(bi.w - bj.w, 0.f)) * kj.w;
                 ak[j] += ki.x * e0 + ki.y * e1 + ki.z * e2 + ki.w * e3;
-                aq[j] += q0 * e0 + q1 * e1 + q2 * e2 + q3 * e3;
+                aq[j] += qi.x * e0 + qi.y * e1 + qi.z * e2 + qi.w * e3;
             }
         }
 #pragma unroll
@@ -312,11 +350,14 @@ delta_chunk_kernel(const ChunkParams p) {
             }
     }
     // ---- Q~, K~, e^{b_C} --------------------------------------------------------------------------------------------------
-    for (int e = tid; e < kC * DK / 2; e += 128) {
-        const int t = e / (DK / 2), c = (e % (DK / 2)) * 2;
-        put_split(wb + Ws<DK>::Q, Ws<DK>::PLANE, t * DK + c, q_at(t, c) * ex2a(s.b[t][c]), q_at(t, c + 1) * ex2a(s.b[t][c + 1]));
-        put_split(wb + Ws<DK>::K, Ws<DK>::PLANE, t * DK + c, s.k[t][c] * ex2a(s.b[kC - 1][c] - s.b[t][c]),
-                  s.k[t][c + 1] * ex2a(s.b[kC - 1][c + 1] - s.b[t][c + 1]));
+#pragma unroll 4
+    for (int e = tid; e < kC * DK / 4; e += 128) {
+        const int t = e / (DK / 4), c = (e % (DK / 4)) * 4;
+        const float4 qv = q_at4(t, c), bt = *reinterpret_cast<const float4*>(&s.b[t][c]), be = *reinterpret_cast<const float4*>(&s.b[kC - 1][c]);
+        const float4 kv = *reinterpret_cast<const float4*>(&s.k[t][c]);
+        put_split4(wb + Ws<DK>::Q, Ws<DK>::PLANE, t * DK + c, qv.x * ex2a(bt.x), qv.y * ex2a(bt.y), qv.z * ex2a(bt.z), qv.w * ex2a(bt.w));
+        put_split4(wb + Ws<DK>::K, Ws<DK>::PLANE, t * DK + c, kv.x * ex2a(be.x - bt.x), kv.y * ex2a(be.y - bt.y), kv.z * ex2a(be.z - bt.z),
+                   kv.w * ex2a(be.w - bt.w));
     }
     if (tid < DK) U0[(long long)kC * p.dvp + tid] = ex2a(s.b[kC - 1][tid]);
 }
@@ -347,15 +388,39 @@ decay_chunk_kernel(const ChunkParams p) {
     const __nv_bfloat16* kg = (const __nv_bfloat16*)p.k + row0 * p.ld + (long long)h * p.dk;
     const __nv_bfloat16* vg = (const __nv_bfloat16*)p.v + row0 * p.ld + (long long)h * p.dv;
     if (tid <= kC) s.pw[tid] = powf(p.decay[h], (float)tid);
-    for (int e = tid; e < kC * DK; e += 128) {
-        const int t = e / DK, c = e % DK;
-        const bool in = t < L && c < p.dk;
-        s.q[t][c] = in ? silu_f(to_f(qg[t * p.ld + c])) : 0.f;
-        s.k[t][c] = in ? silu_f(to_f(kg[t * p.ld + c])) : 0.f;
-    }
-    for (int e = tid; e < kC * p.dvp; e += 128) {
-        const int t = e / p.dvp, c = e % p.dvp;
-        U0[e] = (t < L && c < p.dv) ? silu_f(to_f(vg[t * p.ld + c])) : 0.f;
+    if (p.vec) {
+#pragma unroll 4
+        for (int e = tid; e < kC * DK / 8; e += 128) {
+            const int t = e / (DK / 8), c = (e % (DK / 8)) * 8;
+            float fq[8], fk[8];
+            const bool in = t < L && c < p.dk;
+            if (in) { load8(qg + t * p.ld + c, fq); load8(kg + t * p.ld + c, fk); }
+#pragma unroll
+            for (int i = 0; i < 8; ++i) { s.q[t][c + i] = in ? silu_fast(fq[i]) : 0.f; s.k[t][c + i] = in ? silu_fast(fk[i]) : 0.f; }
+        }
+        const int v8 = p.dvp / 8;
+#pragma unroll 4
+        for (int e = tid; e < kC * v8; e += 128) {
+            const int t = e / v8, c = (e - t * v8) * 8;
+            float f[8];
+            const bool in = t < L && c < p.dv;
+            if (in) load8(vg + t * p.ld + c, f);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) f[i] = in ? silu_fast(f[i]) : 0.f;
+            *reinterpret_cast<float4*>(U0 + (long long)t * p.dvp + c) = make_float4(f[0], f[1], f[2], f[3]);
+            *reinterpret_cast<float4*>(U0 + (long long)t * p.dvp + c + 4) = make_float4(f[4], f[5], f[6], f[7]);
+        }
+    } else {
+        for (int e = tid; e < kC * DK; e += 128) {
+            const int t = e / DK, c = e % DK;
+            const bool in = t < L && c < p.dk;
+            s.q[t][c] = in ? silu_fast(to_f(qg[t * p.ld + c])) : 0.f;
+            s.k[t][c] = in ? silu_fast(to_f(kg[t * p.ld + c])) : 0.f;
+        }
+        for (int e = tid; e < kC * p.dvp; e += 128) {
+            const int t = e / p.dvp, c = e % p.dvp;
+            U0[e] = (t < L && c < p.dv) ? silu_fast(to_f(vg[t * p.ld + c])) : 0.f;
+        }
     }
     __syncthreads();
     float acc[8][4];
@@ -393,11 +458,13 @@ decay_chunk_kernel(const ChunkParams p) {
             }
         }
     }
-    for (int e = tid; e < kC * DK / 2; e += 128) {
-        const int t = e / (DK / 2), c = (e % (DK / 2)) * 2;
+#pragma unroll 4
+    for (int e = tid; e < kC * DK / 4; e += 128) {
+        const int t = e / (DK / 4), c = (e % (DK / 4)) * 4;
         const float fq = s.pw[t + 1], fk = t < L ? s.pw[L - 1 - t] : 0.f;
-        put_split(wb + Ws<DK>::Q, Ws<DK>::PLANE, t * DK + c, s.q[t][c] * fq, s.q[t][c + 1] * fq);
-        put_split(wb + Ws<DK>::K, Ws<DK>::PLANE, t * DK + c, s.k[t][c] * fk, s.k[t][c + 1] * fk);
+        const float4 qv = *reinterpret_cast<const float4*>(&s.q[t][c]), kv = *reinterpret_cast<const float4*>(&s.k[t][c]);
+        put_split4(wb + Ws<DK>::Q, Ws<DK>::PLANE, t * DK + c, qv.x * fq, qv.y * fq, qv.z * fq, qv.w * fq);
+        put_split4(wb + Ws<DK>::K, Ws<DK>::PLANE, t * DK + c, kv.x * fk, kv.y * fk, kv.z * fk, kv.w * fk);
     }
     if (tid < DK) U0[(long long)kC * p.dvp + tid] = s.pw[L];
 }
@@ -630,12 +697,14 @@ int launch_chunk_decay(const DecayAttnArgs& a, void* ws, long long ws_bytes, cud
     ChunkParams p = {};
     p.q = a.q; p.k = a.k; p.v = a.v; p.ld = a.ld; p.decay = a.decay; p.state = a.state; p.o = a.o;
     p.n = a.n; p.H = a.H; p.G = a.H; p.dk = a.dk; p.dv = a.dv;
+    p.vec = a.dk % 8 == 0 && a.dv % 8 == 0 && a.ld % 8 == 0 && !(((uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.v) & 15);
     return launch_dk<false>(p, a.B, ws, ws_bytes, stream);
 }
 int launch_chunk_delta(const DeltaRuleArgs& a, void* ws, long long ws_bytes, cudaStream_t stream) {
     ChunkParams p = {};
     p.q = a.q; p.k = a.k; p.v = a.v; p.logg = a.logg; p.beta = a.beta; p.state = a.state; p.o = a.o;
     p.n = a.n; p.H = a.H; p.G = a.G; p.dk = a.dk; p.dv = a.dv;
+    p.vec = a.dk % 4 == 0 && !(((uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.logg) & 15);
     return launch_dk<true>(p, a.B, ws, ws_bytes, stream);
 }
 

@@ -55,6 +55,39 @@ class HybridConfig:
         return cls(c["width"], c["vocab"], layers, c["norm"]["eps"], c["embedding"]["scale"], c["residual_mult"])
 
 
+def tensor_shapes(config: dict) -> dict:
+    """Stored name -> shape of every tensor of a model with this config.json (ranks and table sizes that only the tensors give take
+    their defaults)."""
+    w, out = config["width"], {"embed": (config["vocab"], config["width"])}
+    for i, e in enumerate(config["layers"]):
+        out[f"l{i}.norm1"] = (w,)
+        out.update({f"l{i}.mix.{k}": s for k, s in M.MIXERS[e["type"]].shapes(e["mixer"], w).items()})
+        if e.get("mlp") is not None:
+            out[f"l{i}.norm2"] = (w,)
+            out.update({f"l{i}.mlp.{k}": s for k, s in M.MLPS[e["mlp"]["kind"]].shapes(e["mlp"], w).items()})
+    out["final.norm"] = (w,)
+    out["head"] = (config["vocab"], w)
+    return out
+
+
+def random_tensors(config: dict, seed: int = 0, device="cpu") -> dict:
+    """Synthetic bf16 weights: matrices N(0, 1 / columns), plain norm weights 1 + N(0, 0.1^2), everything else N(0, 0.3^2)."""
+    g = torch.Generator(device=device).manual_seed(seed)
+    out = {}
+    for name, shape in tensor_shapes(config).items():
+        t = torch.randn(shape, generator=g, device=device)
+        if name in ("embed",):
+            pass
+        elif name.endswith((".mix.norm", ".q.norm", ".k.norm")):
+            t = 1.0 + 0.1 * t
+        elif len(shape) == 2 and not name.endswith((".rel", ".conv")):
+            t = t * shape[1] ** -0.5
+        else:
+            t = t * 0.3
+        out[name] = t.to(torch.bfloat16)
+    return out
+
+
 class _Layer:
     def __init__(self, spec: LayerSpec, tensors, prefix: str, width: int, dtype, device):
         L = M.Loader(tensors, prefix, dtype, device)
@@ -86,9 +119,20 @@ class HybridModel:
     def from_config(cls, config: dict, tensors, dtype=torch.bfloat16, device="cuda"):
         return cls(HybridConfig.from_dict(config), tensors, dtype, device)
 
+    @classmethod
+    def random(cls, config: dict, device="cuda", seed: int = 0, dtype=torch.bfloat16):
+        return cls.from_config(config, random_tensors(config, seed, device), dtype, device)
+
     @property
     def vocab(self) -> int:
         return self.cfg.vocab
+
+    def weight_bytes(self) -> int:
+        """Bytes of the matrices a decode step reads (embedding table aside)."""
+        seen = [self.head]
+        for l in self.layers:
+            seen += [t for m in (l.mixer, l.mlp) if m is not None for t in vars(m).values() if isinstance(t, torch.Tensor) and t.dim() == 2 and t.dtype == self.dtype]
+        return sum(t.numel() * t.element_size() for t in seen)
 
     def new_cache(self, B: int, T_max: int) -> SequenceState:
         return SequenceState([l.mixer.state_spec() for l in self.layers], B, T_max, self.dtype, self.device)

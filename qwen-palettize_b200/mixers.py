@@ -94,6 +94,11 @@ class Lightning:
         self.w_out, self.norm = L.mat("o", (width, v)), L.f32("norm", (v,))
         self.decay = torch.tensor(mc["decay"], dtype=torch.float32, device=L.device)
 
+    @staticmethod
+    def shapes(mc: dict, width: int) -> dict:
+        qk, v = mc["heads"] * mc["dim"], mc["heads"] * mc["vdim"]
+        return {"q": (qk, width), "k": (qk, width), "v": (v, width), "g": (v, width), "o": (width, v), "norm": (v,)}
+
     def state_spec(self):
         return {"S": StateSpec((self.H, self.dk, self.dv), fp32=True, zero=True)}
 
@@ -121,6 +126,15 @@ class ChannelDelta:
         self.conv = torch.cat([L.f32(n + ".conv", (c, self.taps)) for n, c in (("q", qk), ("k", qk), ("v", v))]).contiguous()
         self.A_log, self.dt_bias = L.f32("A_log", (self.H,)), L.f32("dt_bias", (self.H * self.dk,))
         self.norm, self.w_out = L.f32("norm", (self.dv,)), L.mat("o", (width, v))
+
+    @staticmethod
+    def shapes(mc: dict, width: int, rank: int | None = None) -> dict:
+        H, dk, dv = mc["heads"], mc["dim"], mc["vdim"]
+        qk, v, r = mc["kv_heads"] * dk, H * dv, rank or dv
+        out = {"q": (qk, width), "k": (qk, width), "v": (v, width), "b": (H, width), "A_log": (H,), "norm": (dv,), "a1": (r, width),
+               "a2": (H * dk, r), "dt_bias": (H * dk,), "g1": (r, width), "g2": (v, r), "o": (width, v)}
+        out.update({n + ".conv": (out[n][0], mc["conv"]) for n in ("q", "k", "v")})
+        return out
 
     def state_spec(self):
         spec = {"S": StateSpec((self.H, self.dk, self.dv), fp32=True, zero=True)}
@@ -176,6 +190,12 @@ class BiasAttention:
         self.mix = L.f32("vmix").reshape(1) if self.v_mix and L.has("vmix") else None
         self.w_out = L.mat("o", (width, self.H * self.dv))
 
+    @staticmethod
+    def shapes(mc: dict, width: int, buckets: int = 32) -> dict:
+        q, k, v = mc["heads"] * mc["dim"], mc["kv_heads"] * mc["dim"], mc["kv_heads"] * mc["vdim"]
+        return {"q": (q, width), "q.b": (q,), "k": (k, width), "k.b": (k,), "v": (v, width), "v.b": (v,), "q.norm": (q,), "k.norm": (k,),
+                "rel": (buckets, mc["heads"]), "vmix": (), "o": (width, mc["heads"] * mc["vdim"])}
+
     def state_spec(self):
         return {"k": StateSpec(("T_max", self.G * self.dk)), "v": StateSpec(("T_max", self.G * self.dv))}
 
@@ -195,6 +215,10 @@ class BiasAttention:
 class DenseMlp:
     def __init__(self, fc: dict, L: Loader, width: int):
         self.up, self.down = L.mat("up", (fc["ff"], width)), L.mat("down", (width, fc["ff"]))
+
+    @staticmethod
+    def shapes(fc: dict, width: int) -> dict:
+        return {"up": (fc["ff"], width), "down": (width, fc["ff"])}
 
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         return S.linear(S.linear(x, self.up, act=S.ACT_RELU2), self.down)
