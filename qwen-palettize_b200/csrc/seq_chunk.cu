@@ -95,17 +95,21 @@ struct ChunkParams {
 // ---------------------------------------------------------------------------------------------------------------------
 template <int DK>
 struct DeltaSmem {
-    static constexpr int PK = DK + 4, PT = kC + 4;
-    float k[kC][PK], b[kC][PK];      // keys; cumulative log2 decay
-    float a[kC][PT], t[kC][PT];      // beta A' (strictly lower); T
-    float tmp[4][16][20];
+    static constexpr int PK = DK + 4, PB = 17, PT = kC + 4;
+    float q[kC][PK], k[kC][PK];      // k turns into Kbar = k e^b once A' and M are done
+    union {
+        float b[kC][PK];             // cumulative log2 decay
+        struct { float t[kC][PT], tmp[4][16][20]; } inv;   // afterwards: T, and a block product per warp
+    };
+    float a[10][16][PB];             // beta A', strictly lower, as 16 x 16 blocks (I, J <= I) at I (I + 1) / 2 + J
     float beta[kC];
 };
 
+// 256 threads: warps 0-3 the products between blocks, warps 4-7 the 8 x 8 diagonal blocks, then all of them.
 template <int DK>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(256, 2)
 delta_chunk_kernel(const ChunkParams p) {
-    extern __shared__ uint8_t sm_raw[];
+    extern __shared__ __align__(16) uint8_t sm_raw[];
     DeltaSmem<DK>& s = *reinterpret_cast<DeltaSmem<DK>*>(sm_raw);
     constexpr int KS = DK / 16;
     const int tid = threadIdx.x, w = tid >> 5, lane = tid & 31, r4 = lane >> 2, c2 = (lane & 3) * 2;
@@ -115,251 +119,278 @@ delta_chunk_kernel(const ChunkParams p) {
     uint8_t* ws = p.ws + (((long long)b * p.H + h) * p.chunks + ch) * p.ws_stride;
     __nv_bfloat16* wb = reinterpret_cast<__nv_bfloat16*>(ws);
     float* U0 = reinterpret_cast<float*>(ws + Ws<DK>::U_BYTES);
-    const float* qg = (const float*)p.q + (row0 * p.G + hk) * p.dk;        // row pitch G * dk
-    const long long ldq = (long long)p.G * p.dk;
-
+    const long long ldq = (long long)p.G * p.dk, ldg = (long long)p.H * p.dk;
+    const float* qg = (const float*)p.q + (row0 * p.G + hk) * p.dk;
     const float* kg = (const float*)p.k + (row0 * p.G + hk) * p.dk;
     const float* gg = p.logg + (row0 * p.H + h) * p.dk;
-    const long long ldg = (long long)p.H * p.dk;
+
     if (p.vec) {
-#pragma unroll 8
-        for (int e = tid; e < kC * DK / 4; e += 128) {
-            const int t = e / (DK / 4), c = (e % (DK / 4)) * 4;
-            float4 kv = make_float4(0.f, 0.f, 0.f, 0.f), gv = kv;
+#pragma unroll
+        for (int i = 0; i < kC * DK / 4 / 256; ++i) {
+            const int e = tid + i * 256, t = e / (DK / 4), c = (e % (DK / 4)) * 4;
+            float4 qv = make_float4(0.f, 0.f, 0.f, 0.f), kv = qv, gv = qv;
             if (t < L && c < p.dk) {
+                qv = __ldg(reinterpret_cast<const float4*>(qg + t * ldq + c));
                 kv = __ldg(reinterpret_cast<const float4*>(kg + t * ldq + c));
                 gv = __ldg(reinterpret_cast<const float4*>(gg + t * ldg + c));
             }
+            *reinterpret_cast<float4*>(&s.q[t][c]) = qv;
             *reinterpret_cast<float4*>(&s.k[t][c]) = kv;
             *reinterpret_cast<float4*>(&s.b[t][c]) = make_float4(gv.x * kL2e, gv.y * kL2e, gv.z * kL2e, gv.w * kL2e);
         }
     } else {
-        for (int e = tid; e < kC * DK; e += 128) {
+        for (int e = tid; e < kC * DK; e += 256) {
             const int t = e / DK, c = e % DK;
             const bool in = t < L && c < p.dk;
+            s.q[t][c] = in ? qg[t * ldq + c] : 0.f;
             s.k[t][c] = in ? kg[t * ldq + c] : 0.f;
             s.b[t][c] = in ? gg[t * ldg + c] * kL2e : 0.f;
         }
     }
     if (tid < kC) s.beta[tid] = tid < L ? p.beta[(row0 + tid) * p.H + h] : 0.f;
     __syncthreads();
-    if (tid < DK) {
+    // inclusive sum over the 64 tokens, two threads per channel (the second half adds the first half's total)
+    if (tid < 2 * DK) {
+        const int c = tid % DK, h0 = tid / DK * 32;
         float run = 0.f;
 #pragma unroll 16
-        for (int t = 0; t < kC; ++t) { run += s.b[t][tid]; s.b[t][tid] = run; }
+        for (int t = 0; t < 32; ++t) { run += s.b[h0 + t][c]; s.b[h0 + t][c] = run; }
     }
     __syncthreads();
+    for (int e = tid; e < 32 * DK; e += 256) s.b[32 + e / DK][e % DK] += s.b[31][e % DK];
+    __syncthreads();
 
-    // ---- A' and M: warp w takes rows 16 w .. 16 w + 15 -----------------------------------------------------------------
-    auto q_at = [&](int t, int c) { return (t < L && c < p.dk) ? __ldg(qg + t * ldq + c) : 0.f; };
-    auto q_at2 = [&](int t, int c) {      // c even
-        if (!p.vec) return make_float2(q_at(t, c), q_at(t, c + 1));
-        return (t < L && c < p.dk) ? __ldg(reinterpret_cast<const float2*>(qg + t * ldq + c)) : make_float2(0.f, 0.f);
-    };
-    auto q_at4 = [&](int t, int c) {      // c a multiple of four
-        if (!p.vec) return make_float4(q_at(t, c), q_at(t, c + 1), q_at(t, c + 2), q_at(t, c + 3));
-        return (t < L && c < p.dk) ? __ldg(reinterpret_cast<const float4*>(qg + t * ldq + c)) : make_float4(0.f, 0.f, 0.f, 0.f);
-    };
-    const int i0 = 16 * w + r4, i1 = i0 + 8;
-    // blocks left of the diagonal blocks of this warp (reference: token 16 w - 1), then rows 8..15 against columns 0..7 (reference 16 w + 7)
-    for (int part = 0; part < 2; ++part) {
-        if (part == 0 && w == 0) continue;
-        const int ref = part == 0 ? 16 * w - 1 : 16 * w + 7;
-        const int nt0 = part == 0 ? 0 : 2 * w, ntn = part == 0 ? 2 * w : 1;
-        float kk[6][4], qk[6][4];
+    if (w < 4) {
+        // ---- products between blocks. job = 16-row block rb against 8-column tiles nt0 .. nt0 + ntn - 1:
+        //   part 0  tiles left of the diagonal 16-block, reference token 16 rb - 1
+        //   part 1  rows 8..15 against columns 0..7 of the diagonal 16-block, reference token 16 rb + 7
+        const int n_jobs = (w & 1) ? 3 : 1;
+        for (int job = 0; job < n_jobs; ++job) {
+            int rb, part = 0, nt0 = 0, ntn = 4;
+            if (w == 0) rb = 3;
+            else if (w == 2) rb = 2;
+            else if (w == 1) { rb = job < 2 ? 3 : 0; part = job > 0; nt0 = 4; ntn = 2; }
+            else { rb = job < 2 ? 1 : 2; part = job > 0; ntn = 2; }
+            if (part) { nt0 = 2 * rb; ntn = 1; }
+            const int ref = part == 0 ? 16 * rb - 1 : 16 * rb + 7;
+            const int i0 = 16 * rb + r4, i1 = i0 + 8;
+            float kk[4][4], qk[4][4];
 #pragma unroll
-        for (int i = 0; i < 6; ++i)
+            for (int i = 0; i < 4; ++i)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) { kk[i][e] = 0.f; qk[i][e] = 0.f; }
+                for (int e = 0; e < 4; ++e) { kk[i][e] = 0.f; qk[i][e] = 0.f; }
 #pragma unroll 1
-        for (int ks = 0; ks < KS; ++ks) {
-            AFrag ak, aq;
-            float rr[4];
+            for (int ks = 0; ks < KS; ++ks) {
+                AFrag ak, aq;
+                float2 rr[2];
 #pragma unroll
-            for (int x = 0; x < 4; ++x) rr[x] = s.b[ref][ks * 16 + c2 + (x & 1) + (x >> 1) * 8];
+                for (int half = 0; half < 2; ++half) {          // k columns c2, c2 + 1 and + 8
+                    const int c = ks * 16 + c2 + half * 8;
+                    const float2 rf = *reinterpret_cast<const float2*>(&s.b[ref][c]);
+                    rr[half] = rf;
+                    float2 ka = make_float2(0.f, 0.f), qa = ka;
+                    if (part == 0) {
+                        const float2 bb = *reinterpret_cast<const float2*>(&s.b[i0][c]);
+                        const float2 kv = *reinterpret_cast<const float2*>(&s.k[i0][c]), qv = *reinterpret_cast<const float2*>(&s.q[i0][c]);
+                        const float e0 = ex2a(bb.x - rf.x), e1 = ex2a(bb.y - rf.y);
+                        ka = make_float2(kv.x * e0, kv.y * e1); qa = make_float2(qv.x * e0, qv.y * e1);
+                    }
+                    split2(ka.x, ka.y, ak.h[half * 2], ak.l[half * 2]);
+                    split2(qa.x, qa.y, aq.h[half * 2], aq.l[half * 2]);
+                    const float2 bb = *reinterpret_cast<const float2*>(&s.b[i1][c]);
+                    const float2 kv = *reinterpret_cast<const float2*>(&s.k[i1][c]), qv = *reinterpret_cast<const float2*>(&s.q[i1][c]);
+                    const float e0 = ex2a(bb.x - rf.x), e1 = ex2a(bb.y - rf.y);
+                    split2(kv.x * e0, kv.y * e1, ak.h[half * 2 + 1], ak.l[half * 2 + 1]);
+                    split2(qv.x * e0, qv.y * e1, aq.h[half * 2 + 1], aq.l[half * 2 + 1]);
+                }
 #pragma unroll
-            for (int half = 0; half < 2; ++half) {          // k columns c2, c2 + 1 and + 8
-                const int c = ks * 16 + c2 + half * 8;
-                float e00 = 0.f, e01 = 0.f;
-                if (part == 0) { e00 = ex2a(s.b[i0][c] - rr[half * 2]); e01 = ex2a(s.b[i0][c + 1] - rr[half * 2 + 1]); }
-                const float e10 = ex2a(s.b[i1][c] - rr[half * 2]), e11 = ex2a(s.b[i1][c + 1] - rr[half * 2 + 1]);
-                split2(s.k[i0][c] * e00, s.k[i0][c + 1] * e01, ak.h[half * 2], ak.l[half * 2]);
-                split2(s.k[i1][c] * e10, s.k[i1][c + 1] * e11, ak.h[half * 2 + 1], ak.l[half * 2 + 1]);
-                const float2 qa = q_at2(i0, c), qb = q_at2(i1, c);
-                split2(qa.x * e00, qa.y * e01, aq.h[half * 2], aq.l[half * 2]);
-                split2(qb.x * e10, qb.y * e11, aq.h[half * 2 + 1], aq.l[half * 2 + 1]);
+                for (int i = 0; i < 4; ++i) {
+                    if (i < ntn) {
+                        const int j = (nt0 + i) * 8 + r4, c = ks * 16 + c2;
+                        const float2 k0 = *reinterpret_cast<const float2*>(&s.k[j][c]), k1 = *reinterpret_cast<const float2*>(&s.k[j][c + 8]);
+                        const float2 b0 = *reinterpret_cast<const float2*>(&s.b[j][c]), b1 = *reinterpret_cast<const float2*>(&s.b[j][c + 8]);
+                        uint32_t bh0, bl0, bh1, bl1;
+                        split2(k0.x * ex2a(rr[0].x - b0.x), k0.y * ex2a(rr[0].y - b0.y), bh0, bl0);
+                        split2(k1.x * ex2a(rr[1].x - b1.x), k1.y * ex2a(rr[1].y - b1.y), bh1, bl1);
+                        mma_split(kk[i], ak, bh0, bh1, bl0, bl1);
+                        mma_split(qk[i], aq, bh0, bh1, bl0, bl1);
+                    }
+                }
             }
 #pragma unroll
-            for (int i = 0; i < 6; ++i) {
+            for (int i = 0; i < 4; ++i) {
                 if (i < ntn) {
-                    const int j = (nt0 + i) * 8 + r4, c = ks * 16 + c2;
-                    uint32_t bh0, bl0, bh1, bl1;
-                    split2(s.k[j][c] * ex2a(rr[0] - s.b[j][c]), s.k[j][c + 1] * ex2a(rr[1] - s.b[j][c + 1]), bh0, bl0);
-                    split2(s.k[j][c + 8] * ex2a(rr[2] - s.b[j][c + 8]), s.k[j][c + 9] * ex2a(rr[3] - s.b[j][c + 9]), bh1, bl1);
-                    mma_split(kk[i], ak, bh0, bh1, bl0, bl1);
-                    mma_split(qk[i], aq, bh0, bh1, bl0, bl1);
+                    const int j = (nt0 + i) * 8 + c2, blk = rb * (rb + 1) / 2 + (nt0 + i) / 2, jj = ((nt0 + i) & 1) * 8 + c2;
+                    if (part == 0) {
+                        s.a[blk][r4][jj] = kk[i][0] * s.beta[i0]; s.a[blk][r4][jj + 1] = kk[i][1] * s.beta[i0];
+                        put_split(wb + Ws<DK>::M, kC * kC, i0 * kC + j, qk[i][0], qk[i][1]);
+                    }
+                    s.a[blk][r4 + 8][jj] = kk[i][2] * s.beta[i1]; s.a[blk][r4 + 8][jj + 1] = kk[i][3] * s.beta[i1];
+                    put_split(wb + Ws<DK>::M, kC * kC, i1 * kC + j, qk[i][2], qk[i][3]);
                 }
             }
         }
+    } else {
+        // ---- pairs inside the 8-row diagonal blocks: lane = (row, one of four channel slices), all exponents explicit
+        const int rb = w - 4;
+        for (int blk = 0; blk < 2; ++blk) {
+            const int base = 16 * rb + 8 * blk, ri = lane & 7, row = base + ri, quarter = lane >> 3;
+            float ak[8], aq[8];
 #pragma unroll
-        for (int i = 0; i < 6; ++i) {
-            if (i < ntn) {
-                const int j = (nt0 + i) * 8 + c2;
-                if (part == 0) {
-                    s.a[i0][j] = kk[i][0] * s.beta[i0]; s.a[i0][j + 1] = kk[i][1] * s.beta[i0];
-                    put_split(wb + Ws<DK>::M, kC * kC, i0 * kC + j, qk[i][0], qk[i][1]);
-                }
-                s.a[i1][j] = kk[i][2] * s.beta[i1]; s.a[i1][j + 1] = kk[i][3] * s.beta[i1];
-                put_split(wb + Ws<DK>::M, kC * kC, i1 * kC + j, qk[i][2], qk[i][3]);
-            }
-        }
-    }
-    // pairs inside the two 8-row diagonal blocks: lane = (row, one of four channel slices), all exponents explicit
-    for (int blk = 0; blk < 2; ++blk) {
-        const int base = 16 * w + 8 * blk, row = base + (lane & 7), quarter = lane >> 3;
-        float ak[8], aq[8];
-#pragma unroll
-        for (int j = 0; j < 8; ++j) { ak[j] = 0.f; aq[j] = 0.f; }
+            for (int j = 0; j < 8; ++j) { ak[j] = 0.f; aq[j] = 0.f; }
 #pragma unroll 1
-        for (int c4 = quarter; c4 < DK / 4; c4 += 4) {
-            const int c = c4 * 4;
-            const float4 bi = *reinterpret_cast<const float4*>(&s.b[row][c]), ki = *reinterpret_cast<const float4*>(&s.k[row][c]);
-            const float4 qi = q_at4(row, c);
+            for (int c4 = quarter; c4 < DK / 4; c4 += 4) {
+                const int c = c4 * 4;
+                const float4 bi = *reinterpret_cast<const float4*>(&s.b[row][c]), ki = *reinterpret_cast<const float4*>(&s.k[row][c]);
+                const float4 qi = *reinterpret_cast<const float4*>(&s.q[row][c]);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) {
+                    const float4 bj = *reinterpret_cast<const float4*>(&s.b[base + j][c]), kj = *reinterpret_cast<const float4*>(&s.k[base + j][c]);
+                    // j > row: discarded below (the exponent would be positive; clamp it so that nothing overflows)
+                    const float e0 = ex2a(fminf(bi.x - bj.x, 0.f)) * kj.x, e1 = ex2a(fminf(bi.y - bj.y, 0.f)) * kj.y;
+                    const float e2 = ex2a(fminf(bi.z - bj.z, 0.f)) * kj.z, e3 = ex2a(fminf(bi.w - bj.w, 0.f)) * kj.w;
+                    ak[j] += ki.x * e0 + ki.y * e1 + ki.z * e2 + ki.w * e3;
+                    aq[j] += qi.x * e0 + qi.y * e1 + qi.z * e2 + qi.w * e3;
+                }
+            }
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
-                const float4 bj = *reinterpret_cast<const float4*>(&s.b[base + j][c]), kj = *reinterpret_cast<const float4*>(&s.k[base + j][c]);
-                // j > row: discarded below (the exponent would be positive; clamp it so that nothing overflows)
-                const float e0 = ex2a(fminf(bi.x - bj.x, 0.f)) * kj.x, e1 = ex2a(fminf(bi.y - bj.y, 0.f)) * kj.y;
-                const float e2 = ex2a(fminf(bi.z - bj.z, 0.f)) * kj.z, e3 = ex2a(fminf(bi.w - bj.w, 0.f)) * kj.w;
-                ak[j] += ki.x * e0 + ki.y * e1 + ki.z * e2 + ki.w * e3;
-                aq[j] += qi.x * e0 + qi.y * e1 + qi.z * e2 + qi.w * e3;
+                ak[j] += __shfl_xor_sync(0xFFFFFFFFu, ak[j], 8); ak[j] += __shfl_xor_sync(0xFFFFFFFFu, ak[j], 16);
+                aq[j] += __shfl_xor_sync(0xFFFFFFFFu, aq[j], 8); aq[j] += __shfl_xor_sync(0xFFFFFFFFu, aq[j], 16);
+            }
+            if (quarter == 0) {
+#pragma unroll
+                for (int j = 0; j < 8; ++j) s.a[rb * (rb + 1) / 2 + rb][8 * blk + ri][8 * blk + j] = j < ri ? ak[j] * s.beta[row] : 0.f;
+            } else if (quarter == 1) {
+#pragma unroll
+                for (int j = 0; j < 8; j += 2)
+                    put_split(wb + Ws<DK>::M, kC * kC, row * kC + base + j, j <= ri ? aq[j] : 0.f, j + 1 <= ri ? aq[j + 1] : 0.f);
+            } else if (quarter == 2 && blk == 0) {
+                // rows 0..7 against columns 8..15 of the 16-row block lie above the diagonal
+#pragma unroll
+                for (int j = 0; j < 8; j += 2) put_split(wb + Ws<DK>::M, kC * kC, row * kC + base + 8 + j, 0.f, 0.f);
             }
         }
-#pragma unroll
-        for (int j = 0; j < 8; ++j) {
-            ak[j] += __shfl_xor_sync(0xFFFFFFFFu, ak[j], 8); ak[j] += __shfl_xor_sync(0xFFFFFFFFu, ak[j], 16);
-            aq[j] += __shfl_xor_sync(0xFFFFFFFFu, aq[j], 8); aq[j] += __shfl_xor_sync(0xFFFFFFFFu, aq[j], 16);
-        }
-        const int ri = lane & 7;
-        if (quarter == 0) {
-#pragma unroll
-            for (int j = 0; j < 8; ++j) s.a[row][base + j] = j < ri ? ak[j] * s.beta[row] : 0.f;
-        } else if (quarter == 1) {
-#pragma unroll
-            for (int j = 0; j < 8; j += 2)
-                put_split(wb + Ws<DK>::M, kC * kC, row * kC + base + j, j <= ri ? aq[j] : 0.f, j + 1 <= ri ? aq[j + 1] : 0.f);
-        } else if (quarter == 2 && blk == 0) {
-            // rows 0..7 against columns 8..15 of the 16-row block lie above the diagonal
-#pragma unroll
-            for (int j = 0; j < 8; j += 2) put_split(wb + Ws<DK>::M, kC * kC, row * kC + base + 8 + j, 0.f, 0.f);
-        }
     }
+    __syncthreads();
+    // ---- Q~, K~, e^{b_C}; k -> Kbar ---------------------------------------------------------------------------------------
+#pragma unroll 2
+    for (int e = tid; e < kC * DK / 4; e += 256) {
+        const int t = e / (DK / 4), c = (e % (DK / 4)) * 4;
+        const float4 qv = *reinterpret_cast<const float4*>(&s.q[t][c]), kv = *reinterpret_cast<const float4*>(&s.k[t][c]);
+        const float4 bt = *reinterpret_cast<const float4*>(&s.b[t][c]), be = *reinterpret_cast<const float4*>(&s.b[kC - 1][c]);
+        const float4 x = make_float4(ex2a(bt.x), ex2a(bt.y), ex2a(bt.z), ex2a(bt.w));
+        put_split4(wb + Ws<DK>::Q, Ws<DK>::PLANE, t * DK + c, qv.x * x.x, qv.y * x.y, qv.z * x.z, qv.w * x.w);
+        put_split4(wb + Ws<DK>::K, Ws<DK>::PLANE, t * DK + c, kv.x * ex2a(be.x - bt.x), kv.y * ex2a(be.y - bt.y), kv.z * ex2a(be.z - bt.z),
+                   kv.w * ex2a(be.w - bt.w));
+        *reinterpret_cast<float4*>(&s.k[t][c]) = make_float4(kv.x * x.x, kv.y * x.y, kv.z * x.z, kv.w * x.w);
+    }
+    if (tid < DK) U0[(long long)kC * p.dvp + tid] = ex2a(s.b[kC - 1][tid]);
     __syncthreads();
 
     // ---- T = (I + a)^{-1}: 16-row diagonal blocks by substitution, then block diagonals outwards -------------------------
-    if (lane < 16) {
+    if (w < 4 && lane < 16) {
+        const int blk = w * (w + 1) / 2 + w;
         float x[16];
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
             float v = i == lane ? 1.f : 0.f;
 #pragma unroll
-            for (int j = 0; j < i; ++j) v = fmaf(-s.a[16 * w + i][16 * w + j], x[j], v);
+            for (int j = 0; j < i; ++j) v = fmaf(-s.a[blk][i][j], x[j], v);
             x[i] = v;
         }
 #pragma unroll
-        for (int i = 0; i < 16; ++i) s.t[16 * w + i][16 * w + lane] = x[i];
+        for (int i = 0; i < 16; ++i) s.inv.t[16 * w + i][16 * w + lane] = x[i];
     }
     __syncthreads();
+    // a block takes two warps: 16 columns x 8 rows each
     for (int d = 1; d < 4; ++d) {
-        if (w + d < 4) {
-            const int J = w, I = w + d, col = lane & 15, rh = (lane >> 4) * 8;
-            float acc[8];
+        const int J = w >> 1, I = J + d, col = lane & 15, rh = (w & 1) * 8 + (lane >> 4) * 4;
+        float acc[4] = {0.f, 0.f, 0.f, 0.f};
+        if (I < 4) {
+            for (int K = J; K < I; ++K) {
+                const float(*ab)[DeltaSmem<DK>::PB] = s.a[I * (I + 1) / 2 + K];
 #pragma unroll
-            for (int i = 0; i < 8; ++i) acc[i] = 0.f;
-            for (int K = J; K < I; ++K)
-#pragma unroll 4
                 for (int kk = 0; kk < 16; ++kk) {
-                    const float tv = s.t[16 * K + kk][16 * J + col];
+                    const float tv = s.inv.t[16 * K + kk][16 * J + col];
 #pragma unroll
-                    for (int i = 0; i < 8; ++i) acc[i] = fmaf(s.a[16 * I + rh + i][16 * K + kk], tv, acc[i]);
+                    for (int i = 0; i < 4; ++i) acc[i] = fmaf(ab[rh + i][kk], tv, acc[i]);
                 }
-#pragma unroll
-            for (int i = 0; i < 8; ++i) s.tmp[w][rh + i][col] = acc[i];
-            __syncwarp();
-#pragma unroll
-            for (int i = 0; i < 8; ++i) acc[i] = 0.f;
-#pragma unroll 4
-            for (int kk = 0; kk < 16; ++kk) {
-                const float pv = s.tmp[w][kk][col];
-#pragma unroll
-                for (int i = 0; i < 8; ++i) acc[i] = fmaf(s.t[16 * I + rh + i][16 * I + kk], pv, acc[i]);
             }
 #pragma unroll
-            for (int i = 0; i < 8; ++i) s.t[16 * I + rh + i][16 * J + col] = -acc[i];
+            for (int i = 0; i < 4; ++i) s.inv.tmp[J][rh + i][col] = acc[i];
+        }
+        __syncthreads();
+        if (I < 4) {
+#pragma unroll
+            for (int i = 0; i < 4; ++i) acc[i] = 0.f;
+#pragma unroll
+            for (int kk = 0; kk < 16; ++kk) {
+                const float pv = s.inv.tmp[J][kk][col];
+#pragma unroll
+                for (int i = 0; i < 4; ++i) acc[i] = fmaf(s.inv.t[16 * I + rh + i][16 * I + kk], pv, acc[i]);
+            }
+#pragma unroll
+            for (int i = 0; i < 4; ++i) s.inv.t[16 * I + rh + i][16 * J + col] = -acc[i];
         }
         __syncthreads();
     }
 
-    // ---- -W = -(T beta) Kbar and U0 = (T beta) V; a warp takes every fourth 8-column tile ---------------------------------
-    AFrag at[10];     // (m, ks) with ks <= m
+    // ---- -W = -(T beta) Kbar and U0 = (T beta) V. Warps w and w + 4 share an 8-column tile: row blocks {0, 3} and {1, 2} ------
+    const int half_m = w >> 2;
+    const int m0 = half_m ? 1 : 0, m1 = half_m ? 2 : 3;
+    AFrag at[5];      // blocks (m0, 0 .. m0), then (m1, 0 .. m1)
 #pragma unroll
-    for (int m = 0; m < 4; ++m)
+    for (int f = 0; f < 5; ++f) {
+        const int m = f <= m0 ? m0 : m1, ks = f <= m0 ? f : f - m0 - 1;
 #pragma unroll
-        for (int ks = 0; ks <= m; ++ks) {
-            AFrag& f = at[m * (m + 1) / 2 + ks];
-#pragma unroll
-            for (int x = 0; x < 4; ++x) {
-                const int i = 16 * m + r4 + (x & 1) * 8, j = 16 * ks + c2 + (x >> 1) * 8;
-                split2(s.t[i][j] * s.beta[j], s.t[i][j + 1] * s.beta[j + 1], f.h[x], f.l[x]);
-            }
+        for (int x = 0; x < 4; ++x) {
+            const int i = 16 * m + r4 + (x & 1) * 8, j = 16 * ks + c2 + (x >> 1) * 8;
+            split2(s.inv.t[i][j] * s.beta[j], s.inv.t[i][j + 1] * s.beta[j + 1], at[f].h[x], at[f].l[x]);
         }
+    }
     const int nt_w = DK / 8, nt_all = nt_w + p.dvp / 8;
 #pragma unroll 1
-    for (int nt = w; nt < nt_all; nt += 4) {
+    for (int nt = w & 3; nt < nt_all; nt += 4) {
         const bool is_w = nt < nt_w;
         const int c = (is_w ? nt : nt - nt_w) * 8 + r4;
-        float acc[4][4];
+        float f[4][4];
 #pragma unroll
-        for (int m = 0; m < 4; ++m)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) acc[m][e] = 0.f;
-#pragma unroll
-        for (int ks = 0; ks < 4; ++ks) {
-            float f[4];
+        for (int ks = 0; ks < 4; ++ks)
 #pragma unroll
             for (int x = 0; x < 4; ++x) {
                 const int j = 16 * ks + c2 + (x & 1) + (x >> 1) * 8;
-                if (is_w) f[x] = -s.k[j][c] * ex2a(s.b[j][c]);
-                else f[x] = (j < L && c < p.dv) ? __ldg((const float*)p.v + ((row0 + j) * p.H + h) * (long long)p.dv + c) : 0.f;
+                f[ks][x] = 0.f;
+                if (ks <= m1) {
+                    if (is_w) f[ks][x] = -s.k[j][c];
+                    else if (j < L && c < p.dv) f[ks][x] = __ldg((const float*)p.v + ((row0 + j) * p.H + h) * (long long)p.dv + c);
+                }
             }
-            uint32_t bh0, bl0, bh1, bl1;
-            split2(f[0], f[1], bh0, bl0);
-            split2(f[2], f[3], bh1, bl1);
+        float acc0[4] = {0.f, 0.f, 0.f, 0.f}, acc1[4] = {0.f, 0.f, 0.f, 0.f};
+        uint32_t bh[4][2], bl[4][2];
 #pragma unroll
-            for (int m = 0; m < 4; ++m)
-                if (ks <= m) mma_split(acc[m], at[m * (m + 1) / 2 + ks], bh0, bh1, bl0, bl1);
+        for (int ks = 0; ks < 4; ++ks) { split2(f[ks][0], f[ks][1], bh[ks][0], bl[ks][0]); split2(f[ks][2], f[ks][3], bh[ks][1], bl[ks][1]); }
+        if (half_m == 0) {
+            mma_split(acc0, at[0], bh[0][0], bh[0][1], bl[0][0], bl[0][1]);
+#pragma unroll
+            for (int ks = 0; ks < 4; ++ks) mma_split(acc1, at[1 + ks], bh[ks][0], bh[ks][1], bl[ks][0], bl[ks][1]);
+        } else {
+#pragma unroll
+            for (int ks = 0; ks < 2; ++ks) mma_split(acc0, at[ks], bh[ks][0], bh[ks][1], bl[ks][0], bl[ks][1]);
+#pragma unroll
+            for (int ks = 0; ks < 3; ++ks) mma_split(acc1, at[2 + ks], bh[ks][0], bh[ks][1], bl[ks][0], bl[ks][1]);
         }
         const int cc = (is_w ? nt : nt - nt_w) * 8 + c2;
 #pragma unroll
-        for (int m = 0; m < 4; ++m)
+        for (int mm = 0; mm < 2; ++mm)
 #pragma unroll
             for (int hf = 0; hf < 2; ++hf) {
-                const int i = 16 * m + r4 + hf * 8;
-                if (is_w) put_split(wb + Ws<DK>::W, Ws<DK>::PLANE, i * DK + cc, acc[m][hf * 2], acc[m][hf * 2 + 1]);
-                else *reinterpret_cast<float2*>(U0 + (long long)i * p.dvp + cc) = make_float2(acc[m][hf * 2], acc[m][hf * 2 + 1]);
+                const int i = 16 * (mm ? m1 : m0) + r4 + hf * 8;
+                const float x = mm ? acc1[hf * 2] : acc0[hf * 2], y = mm ? acc1[hf * 2 + 1] : acc0[hf * 2 + 1];
+                if (is_w) put_split(wb + Ws<DK>::W, Ws<DK>::PLANE, i * DK + cc, x, y);
+                else *reinterpret_cast<float2*>(U0 + (long long)i * p.dvp + cc) = make_float2(x, y);
             }
     }
-    // ---- Q~, K~, e^{b_C} --------------------------------------------------------------------------------------------------
-#pragma unroll 4
-    for (int e = tid; e < kC * DK / 4; e += 128) {
-        const int t = e / (DK / 4), c = (e % (DK / 4)) * 4;
-        const float4 qv = q_at4(t, c), bt = *reinterpret_cast<const float4*>(&s.b[t][c]), be = *reinterpret_cast<const float4*>(&s.b[kC - 1][c]);
-        const float4 kv = *reinterpret_cast<const float4*>(&s.k[t][c]);
-        put_split4(wb + Ws<DK>::Q, Ws<DK>::PLANE, t * DK + c, qv.x * ex2a(bt.x), qv.y * ex2a(bt.y), qv.z * ex2a(bt.z), qv.w * ex2a(bt.w));
-        put_split4(wb + Ws<DK>::K, Ws<DK>::PLANE, t * DK + c, kv.x * ex2a(be.x - bt.x), kv.y * ex2a(be.y - bt.y), kv.z * ex2a(be.z - bt.z),
-                   kv.w * ex2a(be.w - bt.w));
-    }
-    if (tid < DK) U0[(long long)kC * p.dvp + tid] = ex2a(s.b[kC - 1][tid]);
 }
 
 // ---------------------------------------------------------------------------------------------------------------------
@@ -663,7 +694,7 @@ int launch_chunked(ChunkParams p, int B, void* ws, long long ws_bytes, cudaStrea
     for (int c0 = 0; c0 < all; c0 += (int)seg) {
         p.t_begin = c0 * kC;
         p.chunks = all - c0 < (int)seg ? all - c0 : (int)seg;
-        if (DELTA) delta_chunk_kernel<DK><<<dim3(p.chunks, p.H, B), 128, smem1, stream>>>(p);
+        if (DELTA) delta_chunk_kernel<DK><<<dim3(p.chunks, p.H, B), 256, smem1, stream>>>(p);
         else decay_chunk_kernel<DK><<<dim3(p.chunks, p.H, B), 128, smem1, stream>>>(p);
         PLZ_LAUNCH_CHECK();
         // four warps (64 value columns) per CTA while that leaves SMs free, else eight on one copy of the chunk's operands

@@ -3,6 +3,7 @@
 //   linear_rows_kernel   a handful of rows (token decode): bound by streaming W once. KS warps of a block share the reduction of
 //                        two output rows, chosen so that the launch has enough loads in flight whatever N is; the first
 //                        weights are requested before the wait on the previous kernel of the stream.
+//   linear_skinny_kernel 2 .. 16 rows, bf16: the same streaming with mma.sync fragments loaded straight from memory.
 //   linear_tile_kernel   any shape and both types on the CUDA cores, fp32 products and sums: the 32-bit mode, and bf16 shapes
 //                        that the tensor-core path's 16-byte rows exclude.
 //   launch_seq_linear    picks one of them or the tcgen05 GEMM (lut_gemm.cu, dense B, bias and activation in its epilogue).
@@ -107,6 +108,77 @@ linear_rows_kernel(const LinParams p, int ks) {
     }
 }
 
+// 2 .. 16 rows of x, bf16: a warp takes 16 output rows (weight rows) as the A operand of m16n8k16 mma.sync, x as B. The order of the
+// reduction index inside a product is free, so lane (r, q) loads 16 contiguous bytes of weight rows r and r + 8 and of x row r at
+// k0 + 8 q and uses them as the fragments of two products: no shuffle, no shared memory, no unpacking. KS warps share the reduction.
+template <typename TO, int NT>     // NT: groups of eight x rows
+__global__ void __launch_bounds__(256)
+linear_skinny_kernel(const LinParams p, int ks) {
+    __shared__ float part[8][16][8 * NT + 1];
+    constexpr int U = 4;           // 32-wide steps in flight
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, r4 = lane >> 2, q8 = (lane & 3) * 8;
+    const int groups = 8 / ks, grp = warp / ks, kw = warp % ks;
+    const int n0 = ((int)blockIdx.x * groups + grp) * 16;
+    const __nv_bfloat16* w0 = (const __nv_bfloat16*)p.w + (long long)(n0 + r4) * p.ldw;
+    const __nv_bfloat16* w1 = w0 + 8 * p.ldw;
+    const bool has0 = n0 + r4 < p.N, has1 = n0 + r4 + 8 < p.N;
+    const uint4 z = make_uint4(0u, 0u, 0u, 0u);
+    uint4 a[U], b[U];
+    auto fetch = [&](int k) {
+#pragma unroll
+        for (int i = 0; i < U; ++i) {
+            const int kk = k + i * 32 * ks + q8;
+            a[i] = has0 && kk < p.K ? __ldg(reinterpret_cast<const uint4*>(w0 + kk)) : z;
+            b[i] = has1 && kk < p.K ? __ldg(reinterpret_cast<const uint4*>(w1 + kk)) : z;
+        }
+    };
+    int k = kw * 32;
+    fetch(k);                          // weights do not depend on the previous kernel
+    pdl_launch_dependents();
+    pdl_wait();
+    float acc[NT][4];
+#pragma unroll
+    for (int t = 0; t < NT; ++t)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[t][e] = 0.f;
+    auto mma = [&](float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+        asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                     : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+    };
+    while (k < p.K) {
+        uint4 xv[U][NT];
+#pragma unroll
+        for (int i = 0; i < U; ++i)
+#pragma unroll
+            for (int t = 0; t < NT; ++t) {
+                const int kk = k + i * 32 * ks + q8, m = t * 8 + r4;
+                xv[i][t] = m < p.M && kk < p.K ? *reinterpret_cast<const uint4*>((const __nv_bfloat16*)p.x + (long long)m * p.ldx + kk) : z;
+            }
+#pragma unroll
+        for (int i = 0; i < U; ++i)
+#pragma unroll
+            for (int t = 0; t < NT; ++t) {
+                mma(acc[t], a[i].x, b[i].x, a[i].y, b[i].y, xv[i][t].x, xv[i][t].y);
+                mma(acc[t], a[i].z, b[i].z, a[i].w, b[i].w, xv[i][t].z, xv[i][t].w);
+            }
+        k += U * 32 * ks;
+        if (k < p.K) fetch(k);
+    }
+#pragma unroll
+    for (int t = 0; t < NT; ++t)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) part[warp][r4 + (e >> 1) * 8][t * 8 + (lane & 3) * 2 + (e & 1)] = acc[t][e];
+    __syncthreads();
+    for (int e = threadIdx.x; e < groups * 16 * 8 * NT; e += 256) {
+        const int g = e / (16 * 8 * NT), r = e % 16, m = (e / 16) % (8 * NT), n = ((int)blockIdx.x * groups + g) * 16 + r;
+        if (m >= p.M || n >= p.N) continue;
+        float v = 0.f;
+        for (int i = 0; i < ks; ++i) v += part[g * ks + i][r][m];
+        if (p.bias) v += to_f(((const __nv_bfloat16*)p.bias)[n]);
+        ((TO*)p.y)[(long long)m * p.ldy + n] = from_f<TO>(activate(v, p.act));
+    }
+}
+
 template <typename T, typename TO>
 __global__ void __launch_bounds__(256)
 linear_tile_kernel(const LinParams p) {
@@ -166,6 +238,16 @@ int launch_rows(const LinParams& p, cudaStream_t stream) {
     else PLZ_LAUNCH_CHAIN((linear_rows_kernel<T, TO, 8>), grid, dim3(256), 0, stream, p, ks);
     return PLZ_OK;
 }
+template <typename TO>
+int launch_skinny(const LinParams& p, cudaStream_t stream) {
+    const int tiles = (p.N + 15) / 16;
+    int ks = 1;
+    while (ks < 8 && (long long)tiles * ks < 16ll * seq_sm_count() && p.K > 128 * ks) ks *= 2;
+    const dim3 grid((tiles + 8 / ks - 1) / (8 / ks));
+    if (p.M <= 8) PLZ_LAUNCH_CHAIN((linear_skinny_kernel<TO, 1>), grid, dim3(256), 0, stream, p, ks);
+    else PLZ_LAUNCH_CHAIN((linear_skinny_kernel<TO, 2>), grid, dim3(256), 0, stream, p, ks);
+    return PLZ_OK;
+}
 template <typename T, typename TO>
 int launch_tile(const LinParams& p, cudaStream_t stream) {
     const long long my = (p.M + 63) / 64;
@@ -184,6 +266,7 @@ int launch_seq_linear(int dtype, const void* x, long long ldx, int M, int K, con
     const LinParams p = {x, ldx, w, ldw, bias, y, ldy, M, N, K, act};
     const int per16 = dtype == 0 ? 8 : 4;
     const bool vec = K % 8 == 0 && ldx % per16 == 0 && ldw % per16 == 0 && !((uintptr_t)x & 15) && !((uintptr_t)w & 15);
+    if (dtype == 0 && M > 1 && M <= 16 && vec) return y_f32 ? launch_skinny<float>(p, stream) : launch_skinny<__nv_bfloat16>(p, stream);
     if (M <= 8 && vec) {
         if (dtype == 1) return launch_rows<float, float>(p, stream);
         return y_f32 ? launch_rows<__nv_bfloat16, float>(p, stream) : launch_rows<__nv_bfloat16, __nv_bfloat16>(p, stream);

@@ -203,6 +203,95 @@ delta_prep_kernel(const DeltaPrep p) {
     for (int c = lane; c < L; c += 32) dst[c] *= f;      // this lane's own elements
 }
 
+// The same for portions: a warp takes one item over kPrepRows consecutive tokens, four channels per lane (head sizes up to 128, a
+// multiple of 4), the convolution's inputs sliding through registers. Up to four taps (missing ones count as zero weights).
+constexpr int kPrepRows = 16;
+__device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
+    const uint2 r = *reinterpret_cast<const uint2*>(p);
+    return make_float4(__uint_as_float(r.x << 16), __uint_as_float(r.x & 0xFFFF0000u), __uint_as_float(r.y << 16), __uint_as_float(r.y & 0xFFFF0000u));
+}
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+template <typename T>
+__global__ void __launch_bounds__(256)
+delta_prep_rows_kernel(const DeltaPrep p) {
+    const int lane = threadIdx.x & 31, item = (int)blockIdx.y * 8 + (threadIdx.x >> 5);
+    const int blocks = (p.n + kPrepRows - 1) / kPrepRows;
+    const long long b = blockIdx.x / blocks;
+    const int t0 = (int)(blockIdx.x % blocks) * kPrepRows, t1 = min(p.n, t0 + kPrepRows);
+    const long long r0 = b * p.n;
+    pdl_launch_dependents();
+    pdl_wait();
+    if (item >= 2 * p.G + 2 * p.H) return;
+    const int c = lane * 4;
+    if (item >= 2 * p.G + p.H) {
+        const int h = item - 2 * p.G - p.H;
+        const float rate = -expf(p.A_log[h]);
+        float4 bias = make_float4(0.f, 0.f, 0.f, 0.f);
+        const bool in = c < p.dk;
+        if (in) bias = make_float4(p.dt_bias[h * p.dk + c], p.dt_bias[h * p.dk + c + 1], p.dt_bias[h * p.dk + c + 2], p.dt_bias[h * p.dk + c + 3]);
+        for (int tb = t0; tb < t1; tb += 4) {
+            float4 x[4];
+#pragma unroll
+            for (int u = 0; u < 4; ++u)
+                if (in && tb + u < t1) x[u] = load4((const T*)p.a + (r0 + tb + u) * p.lda + (long long)h * p.dk + c);
+#pragma unroll
+            for (int u = 0; u < 4; ++u)
+                if (in && tb + u < t1)
+                    *reinterpret_cast<float4*>(p.logg + ((r0 + tb + u) * p.H + h) * p.dk + c) =
+                        make_float4(rate * softplus_f(x[u].x + bias.x), rate * softplus_f(x[u].y + bias.y), rate * softplus_f(x[u].z + bias.z),
+                                    rate * softplus_f(x[u].w + bias.w));
+        }
+        if (lane < kPrepRows && t0 + lane < t1)
+            p.beta[(r0 + t0 + lane) * p.H + h] = sigmoid_f(to_f(((const T*)p.proj)[(r0 + t0 + lane) * p.ldp + p.off_b + h]));
+        return;
+    }
+    const int kind = item < p.G ? 0 : (item < 2 * p.G ? 1 : 2);
+    const int head = kind == 0 ? item : (kind == 1 ? item - p.G : item - 2 * p.G);
+    const int L = kind == 2 ? p.dv : p.dk;
+    const int off = (kind == 0 ? p.off_q : (kind == 1 ? p.off_k : p.off_v)) + head * L;
+    const int ch0 = (kind == 0 ? 0 : (kind == 1 ? p.G * p.dk : 2 * p.G * p.dk)) + head * L;
+    const int C = 2 * p.G * p.dk + p.H * p.dv, keep = p.n_taps - 1;
+    const bool in = c < L;
+    float w[4][4];                                    // [tap looking back 3 - j tokens][channel]
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const int k = j - (4 - p.n_taps);         // stored column of this tap
+            w[j][e] = in && k >= 0 ? p.taps[(long long)(ch0 + c + e) * p.n_taps + k] : 0.f;
+        }
+    auto input = [&](int t) {                         // tokens before the portion come from the kept inputs, before those zero
+        if (!in) return make_float4(0.f, 0.f, 0.f, 0.f);
+        if (t >= 0) return load4((const T*)p.proj + (r0 + t) * p.ldp + off + c);
+        if (t + keep < 0) return make_float4(0.f, 0.f, 0.f, 0.f);
+        return load4((const T*)p.conv + (b * keep + t + keep) * (long long)C + ch0 + c);
+    };
+    float4 x0 = input(t0 - 3), x1 = input(t0 - 2), x2 = input(t0 - 1);
+    float* dst = kind == 0 ? p.q + head * p.dk : (kind == 1 ? p.k + head * p.dk : p.v + head * p.dv);
+    const long long ldd = kind == 2 ? (long long)p.H * p.dv : (long long)p.G * p.dk;
+    for (int tb = t0; tb < t1; tb += 4) {
+        float4 nx[4];
+#pragma unroll
+        for (int u = 0; u < 4; ++u) nx[u] = tb + u < t1 ? input(tb + u) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+            const float4 x3 = nx[u];
+            float4 y;
+            y.x = silu_f(w[0][0] * x0.x + w[1][0] * x1.x + w[2][0] * x2.x + w[3][0] * x3.x);
+            y.y = silu_f(w[0][1] * x0.y + w[1][1] * x1.y + w[2][1] * x2.y + w[3][1] * x3.y);
+            y.z = silu_f(w[0][2] * x0.z + w[1][2] * x1.z + w[2][2] * x2.z + w[3][2] * x3.z);
+            y.w = silu_f(w[0][3] * x0.w + w[1][3] * x1.w + w[2][3] * x2.w + w[3][3] * x3.w);
+            x0 = x1; x1 = x2; x2 = x3;
+            float f = 1.f;
+            if (kind != 2) {
+                const float ss = warp_sum(y.x * y.x + y.y * y.y + y.z * y.z + y.w * y.w);
+                f = (kind == 0 ? p.q_scale : 1.0f) / sqrtf(ss + 1e-6f);
+            }
+            if (in && tb + u < t1) *reinterpret_cast<float4*>(dst + (r0 + tb + u) * ldd + c) = make_float4(y.x * f, y.y * f, y.z * f, y.w * f);
+        }
+    }
+}
+
 // the last n_taps - 1 inputs after a portion of n tokens (n >= 1)
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -387,7 +476,14 @@ int launch_delta_prep(int dtype, const DeltaPrepArgs& a, cudaStream_t stream) {
     p.q = a.q; p.k = a.k; p.v = a.v; p.logg = a.logg; p.beta = a.beta;
     p.update = a.n == 1;
     const dim3 grid((unsigned)rows, (2 * a.G + 2 * a.H + 7) / 8);
-    if (dtype == 1) PLZ_LAUNCH_CHAIN(delta_prep_kernel<float>, grid, dim3(256), 0, stream, p);
+    const int C4 = 2 * a.G * a.dk + a.H * a.dv;
+    const bool rows4 = a.n >= 8 && a.n_taps <= 4 && a.dk % 4 == 0 && a.dv % 4 == 0 && a.dk <= 128 && a.dv <= 128 && C4 % 4 == 0 && a.ldp % 4 == 0 && a.lda % 4 == 0 &&
+                       a.off_q % 4 == 0 && a.off_k % 4 == 0 && a.off_v % 4 == 0 && !(((uintptr_t)a.proj | (uintptr_t)a.a | (uintptr_t)a.conv | (uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.v | (uintptr_t)a.logg) & 15);
+    if (rows4) {
+        const dim3 g4((unsigned)((long long)a.B * ((a.n + kPrepRows - 1) / kPrepRows)), grid.y);
+        if (dtype == 1) PLZ_LAUNCH_CHAIN(delta_prep_rows_kernel<float>, g4, dim3(256), 0, stream, p);
+        else PLZ_LAUNCH_CHAIN(delta_prep_rows_kernel<bf>, g4, dim3(256), 0, stream, p);
+    } else if (dtype == 1) PLZ_LAUNCH_CHAIN(delta_prep_kernel<float>, grid, dim3(256), 0, stream, p);
     else PLZ_LAUNCH_CHAIN(delta_prep_kernel<bf>, grid, dim3(256), 0, stream, p);
     if (a.n > 1 && a.n_taps > 1) {
         const int qk = a.G * a.dk, C = 2 * qk + a.H * a.dv;

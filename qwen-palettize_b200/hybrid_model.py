@@ -156,7 +156,7 @@ class HybridModel:
     def logits(self, x: torch.Tensor, rows=None) -> torch.Tensor:
         """fp32 logits of the given rows (int64 device tensor; None: all) of the residual stream."""
         h = S.rows_norm(x, rows, self.final_norm, self.DESIGN.norm_offset, self.cfg.eps, self.dtype)
-        return S.linear(h, self.head, out_f32=True) if h.shape[0] <= 8 else S.linear(h, self.head).float()
+        return S.linear(h, self.head, out_f32=True) if h.shape[0] <= 16 else S.linear(h, self.head).float()
 
     def forward(self, ids: torch.Tensor, cache: SequenceState, want=None):
         """Run ids int64 [B, n] from the state in `cache`; want: rows (b * n + t) whose logits are returned, fp32 [len(want), vocab]
