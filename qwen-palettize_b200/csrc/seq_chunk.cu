@@ -8,34 +8,27 @@
 //
 // (decayed linear attention: u = v, no W, scalar decay). Two launches per segment of chunks:
 //   delta_chunk_kernel / decay_chunk_kernel   one CTA per (chunk, head, sequence), all in parallel: -W, U0, Q~, K~, M, e^{b_C}
-//   chunk_scan_kernel                         one CTA per (64 value columns, head, sequence) walks the chunks in order.
+//   scan_kernel (seq_scan.cu)                 one CTA per (128 value columns, head, sequence) walks the chunks in order.
 //
 // Exponents of decays are never positive: products e^{b_i - b_j} = e^{b_i - r} e^{r - b_j} use a reference r between the two tokens (the
 // token before the 16- or 8-row block of i), and pairs inside one 8-row block are evaluated directly. So a decay of any strength
 // underflows to zero and nothing overflows.
 //
 // The recurrence is fp32: every operand of a product is split into two bf16 terms (hi + lo) and the product takes the three terms
-// hi hi + hi lo + lo hi, i.e. about 16 bits of mantissa, with fp32 accumulation and an fp32 state. The products are 16 x 8 x 16
-// mma.sync on register fragments: the blocks here are 8 to 16 rows, the state of the scan has to leave the accumulator and come back as
-// an operand at every chunk, and with the state held TRANSPOSED (value rows x key columns) the accumulator layout IS the operand layout,
-// so a chunk costs no trip of state or U through shared or tensor memory.
-#include "seq_math.cuh"
+// hi hi + hi lo + lo hi, i.e. about 16 bits of mantissa, with fp32 accumulation and an fp32 state. The scan's products (128 x 64 .. 128
+// x 64 .. 128) run on tcgen05 (seq_scan.cu); the 8- and 16-row blocks in here are 16 x 8 x 16 mma.sync on register fragments, whose
+// operands are formed in registers (decays times keys) and never stored.
+#include "seq_chunk.cuh"
 
 namespace plz {
 namespace {
 
-constexpr int kC = 64;                     // tokens per chunk
 constexpr float kL2e = 1.4426950408889634f;
 
 __device__ __forceinline__ float ex2a(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
 
 // z / (1 + e^-z) of a bf16 input, about 2^-21 relative
 __device__ __forceinline__ float silu_fast(float z) { return __fdividef(z, 1.0f + ex2a(-z * kL2e)); }
-// (x, y) -> bf16 pairs hi, lo with x ~ hi.x + lo.x
-__device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
-    hi = pack_bf16x2(x, y);
-    lo = pack_bf16x2(x - __uint_as_float(hi << 16), y - __uint_as_float(hi & 0xFFFF0000u));
-}
 __device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
     asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
                  : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
@@ -47,36 +40,16 @@ __device__ __forceinline__ void mma_split(float (&d)[4], const AFrag& a, uint32_
     mma16816(d, a.h, bl0, bl1);
     mma16816(d, a.l, bh0, bh1);
 }
-__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void cp16(uint32_t dst, const void* src) { asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory"); }
-__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
-
-// Workspace of one (sequence, head, chunk): bf16 planes (hi, lo) of -W, Q~, K~ [64][DK] and M [64][64], then fp32 U0 [64][DVP], e^{b_C} [DK]
-template <int DK>
-struct Ws {
-    static constexpr int PLANE = kC * DK;                      // bf16 elements
-    static constexpr int W = 0, Q = 2 * PLANE, M = 4 * PLANE, K = M + 2 * kC * kC, U_BYTES = (K + 2 * PLANE) * 2;
-    static __host__ __device__ long long bytes(int dvp) { return (long long)U_BYTES + (long long)kC * dvp * 4 + DK * 4; }
-};
-__device__ __forceinline__ void put_split(__nv_bfloat16* plane, int stride, int at, float x, float y) {
-    uint32_t h, l;
-    split2(x, y, h, l);
-    *reinterpret_cast<uint32_t*>(plane + at) = h;
-    *reinterpret_cast<uint32_t*>(plane + stride + at) = l;
-}
-
-__device__ __forceinline__ void put_split4(__nv_bfloat16* plane, int stride, int at, float x, float y, float z, float w) {
-    uint2 h, l;
-    split2(x, y, h.x, l.x);
-    split2(z, w, h.y, l.y);
-    *reinterpret_cast<uint2*>(plane + at) = h;
-    *reinterpret_cast<uint2*>(plane + stride + at) = l;
+// the 16 x 16 blocks of M above the diagonal (the scan multiplies the whole tile), 256 threads
+__device__ __forceinline__ void zero_upper(uint8_t* wM, uint32_t plane, int tid) {
+    for (int e = tid; e < kC * kC / 8; e += 256) {
+        const uint32_t r = e / (kC / 8), c = (e % (kC / 8)) * 8;
+        if ((c >> 4) > (r >> 4)) {
+            const uint32_t at = ChunkWs<1, 64>::at(kC, r, c);
+            *reinterpret_cast<uint4*>(wM + at) = make_uint4(0u, 0u, 0u, 0u);
+            *reinterpret_cast<uint4*>(wM + plane + at) = make_uint4(0u, 0u, 0u, 0u);
+        }
+    }
 }
 
 struct ChunkParams {
@@ -117,8 +90,9 @@ delta_chunk_kernel(const ChunkParams p) {
     const int t0 = p.t_begin + ch * kC, L = min(kC, p.n - t0);
     const long long row0 = (long long)b * p.n + t0;
     uint8_t* ws = p.ws + (((long long)b * p.H + h) * p.chunks + ch) * p.ws_stride;
-    __nv_bfloat16* wb = reinterpret_cast<__nv_bfloat16*>(ws);
-    float* U0 = reinterpret_cast<float*>(ws + Ws<DK>::U_BYTES);
+    using W = ChunkWs<DK / 64, 128>;
+    uint8_t* wM = ws + W::OFF_B;
+    float* U0 = reinterpret_cast<float*>(ws + W::OFF_U);
     const long long ldq = (long long)p.G * p.dk, ldg = (long long)p.H * p.dk;
     const float* qg = (const float*)p.q + (row0 * p.G + hk) * p.dk;
     const float* kg = (const float*)p.k + (row0 * p.G + hk) * p.dk;
@@ -223,10 +197,10 @@ delta_chunk_kernel(const ChunkParams p) {
                     const int j = (nt0 + i) * 8 + c2, blk = rb * (rb + 1) / 2 + (nt0 + i) / 2, jj = ((nt0 + i) & 1) * 8 + c2;
                     if (part == 0) {
                         s.a[blk][r4][jj] = kk[i][0] * s.beta[i0]; s.a[blk][r4][jj + 1] = kk[i][1] * s.beta[i0];
-                        put_split(wb + Ws<DK>::M, kC * kC, i0 * kC + j, qk[i][0], qk[i][1]);
+                        put_split(wM + W::at(kC, i0, j), W::M_PLANE, qk[i][0], qk[i][1]);
                     }
                     s.a[blk][r4 + 8][jj] = kk[i][2] * s.beta[i1]; s.a[blk][r4 + 8][jj + 1] = kk[i][3] * s.beta[i1];
-                    put_split(wb + Ws<DK>::M, kC * kC, i1 * kC + j, qk[i][2], qk[i][3]);
+                    put_split(wM + W::at(kC, i1, j), W::M_PLANE, qk[i][2], qk[i][3]);
                 }
             }
         }
@@ -246,9 +220,9 @@ delta_chunk_kernel(const ChunkParams p) {
 #pragma unroll
                 for (int j = 0; j < 8; ++j) {
                     const float4 bj = *reinterpret_cast<const float4*>(&s.b[base + j][c]), kj = *reinterpret_cast<const float4*>(&s.k[base + j][c]);
-                    // j > row: discarded below (the exponent would be positive; clamp it so that nothing overflows)
-                    const float e0 = ex2a(fminf(bi.x - bj.x, 0.f)) * kj.x, e1 = ex2a(fminf(bi.y - bj.y, 0.f)) * kj.y;
-                    const float e2 = ex2a(fminf(bi.z - bj.z, 0.f)) * kj.z, e3 = ex2a(fminf(bi.w - bj.w, 0.f)) * kj.w;
+                    // j > row: an exponent above zero, discarded below
+                    const float e0 = ex2a(bi.x - bj.x) * kj.x, e1 = ex2a(bi.y - bj.y) * kj.y;
+                    const float e2 = ex2a(bi.z - bj.z) * kj.z, e3 = ex2a(bi.w - bj.w) * kj.w;
                     ak[j] += ki.x * e0 + ki.y * e1 + ki.z * e2 + ki.w * e3;
                     aq[j] += qi.x * e0 + qi.y * e1 + qi.z * e2 + qi.w * e3;
                 }
@@ -264,11 +238,11 @@ delta_chunk_kernel(const ChunkParams p) {
             } else if (quarter == 1) {
 #pragma unroll
                 for (int j = 0; j < 8; j += 2)
-                    put_split(wb + Ws<DK>::M, kC * kC, row * kC + base + j, j <= ri ? aq[j] : 0.f, j + 1 <= ri ? aq[j + 1] : 0.f);
+                    put_split(wM + W::at(kC, row, base + j), W::M_PLANE, j <= ri ? aq[j] : 0.f, j + 1 <= ri ? aq[j + 1] : 0.f);
             } else if (quarter == 2 && blk == 0) {
                 // rows 0..7 against columns 8..15 of the 16-row block lie above the diagonal
 #pragma unroll
-                for (int j = 0; j < 8; j += 2) put_split(wb + Ws<DK>::M, kC * kC, row * kC + base + 8 + j, 0.f, 0.f);
+                for (int j = 0; j < 8; j += 2) put_split(wM + W::at(kC, row, base + 8 + j), W::M_PLANE, 0.f, 0.f);
             }
         }
     }
@@ -280,12 +254,13 @@ delta_chunk_kernel(const ChunkParams p) {
         const float4 qv = *reinterpret_cast<const float4*>(&s.q[t][c]), kv = *reinterpret_cast<const float4*>(&s.k[t][c]);
         const float4 bt = *reinterpret_cast<const float4*>(&s.b[t][c]), be = *reinterpret_cast<const float4*>(&s.b[kC - 1][c]);
         const float4 x = make_float4(ex2a(bt.x), ex2a(bt.y), ex2a(bt.z), ex2a(bt.w));
-        put_split4(wb + Ws<DK>::Q, Ws<DK>::PLANE, t * DK + c, qv.x * x.x, qv.y * x.y, qv.z * x.z, qv.w * x.w);
-        put_split4(wb + Ws<DK>::K, Ws<DK>::PLANE, t * DK + c, kv.x * ex2a(be.x - bt.x), kv.y * ex2a(be.y - bt.y), kv.z * ex2a(be.z - bt.z),
+        put_split4(ws + W::at(128, 64 + t, c), W::A_PLANE, qv.x * x.x, qv.y * x.y, qv.z * x.z, qv.w * x.w);
+        put_split4(ws + W::OFF_K + W::at(kC, t, c), W::K_PLANE, kv.x * ex2a(be.x - bt.x), kv.y * ex2a(be.y - bt.y), kv.z * ex2a(be.z - bt.z),
                    kv.w * ex2a(be.w - bt.w));
         *reinterpret_cast<float4*>(&s.k[t][c]) = make_float4(kv.x * x.x, kv.y * x.y, kv.z * x.z, kv.w * x.w);
     }
-    if (tid < DK) U0[(long long)kC * p.dvp + tid] = ex2a(s.b[kC - 1][tid]);
+    if (tid < DK) reinterpret_cast<float*>(ws + W::OFF_DEC)[tid] = ex2a(s.b[kC - 1][tid]);
+    zero_upper(wM, W::M_PLANE, tid);
     __syncthreads();
 
     // ---- T = (I + a)^{-1}: 16-row diagonal blocks by substitution, then block diagonals outwards -------------------------
@@ -387,7 +362,7 @@ delta_chunk_kernel(const ChunkParams p) {
             for (int hf = 0; hf < 2; ++hf) {
                 const int i = 16 * (mm ? m1 : m0) + r4 + hf * 8;
                 const float x = mm ? acc1[hf * 2] : acc0[hf * 2], y = mm ? acc1[hf * 2 + 1] : acc0[hf * 2 + 1];
-                if (is_w) put_split(wb + Ws<DK>::W, Ws<DK>::PLANE, i * DK + cc, x, y);
+                if (is_w) put_split(ws + W::at(128, i, cc), W::A_PLANE, x, y);
                 else *reinterpret_cast<float2*>(U0 + (long long)i * p.dvp + cc) = make_float2(x, y);
             }
     }
@@ -403,7 +378,7 @@ struct DecaySmem {
     float pw[kC + 1];               // powers of the decay
 };
 template <int DK>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(256)
 decay_chunk_kernel(const ChunkParams p) {
     extern __shared__ uint8_t sm_raw[];
     DecaySmem<DK>& s = *reinterpret_cast<DecaySmem<DK>*>(sm_raw);
@@ -413,15 +388,16 @@ decay_chunk_kernel(const ChunkParams p) {
     const int t0 = p.t_begin + ch * kC, L = min(kC, p.n - t0);
     const long long row0 = (long long)b * p.n + t0;
     uint8_t* ws = p.ws + (((long long)b * p.H + h) * p.chunks + ch) * p.ws_stride;
-    __nv_bfloat16* wb = reinterpret_cast<__nv_bfloat16*>(ws);
-    float* U0 = reinterpret_cast<float*>(ws + Ws<DK>::U_BYTES);
+    using W = ChunkWs<DK / 64, 64>;
+    uint8_t* wM = ws + W::OFF_B;
+    float* U0 = reinterpret_cast<float*>(ws + W::OFF_U);
     const __nv_bfloat16* qg = (const __nv_bfloat16*)p.q + row0 * p.ld + (long long)h * p.dk;
     const __nv_bfloat16* kg = (const __nv_bfloat16*)p.k + row0 * p.ld + (long long)h * p.dk;
     const __nv_bfloat16* vg = (const __nv_bfloat16*)p.v + row0 * p.ld + (long long)h * p.dv;
     if (tid <= kC) s.pw[tid] = powf(p.decay[h], (float)tid);
     if (p.vec) {
 #pragma unroll 4
-        for (int e = tid; e < kC * DK / 8; e += 128) {
+        for (int e = tid; e < kC * DK / 8; e += 256) {
             const int t = e / (DK / 8), c = (e % (DK / 8)) * 8;
             float fq[8], fk[8];
             const bool in = t < L && c < p.dk;
@@ -431,7 +407,7 @@ decay_chunk_kernel(const ChunkParams p) {
         }
         const int v8 = p.dvp / 8;
 #pragma unroll 4
-        for (int e = tid; e < kC * v8; e += 128) {
+        for (int e = tid; e < kC * v8; e += 256) {
             const int t = e / v8, c = (e - t * v8) * 8;
             float f[8];
             const bool in = t < L && c < p.dv;
@@ -442,271 +418,105 @@ decay_chunk_kernel(const ChunkParams p) {
             *reinterpret_cast<float4*>(U0 + (long long)t * p.dvp + c + 4) = make_float4(f[4], f[5], f[6], f[7]);
         }
     } else {
-        for (int e = tid; e < kC * DK; e += 128) {
+        for (int e = tid; e < kC * DK; e += 256) {
             const int t = e / DK, c = e % DK;
             const bool in = t < L && c < p.dk;
             s.q[t][c] = in ? silu_fast(to_f(qg[t * p.ld + c])) : 0.f;
             s.k[t][c] = in ? silu_fast(to_f(kg[t * p.ld + c])) : 0.f;
         }
-        for (int e = tid; e < kC * p.dvp; e += 128) {
+        for (int e = tid; e < kC * p.dvp; e += 256) {
             const int t = e / p.dvp, c = e % p.dvp;
             U0[e] = (t < L && c < p.dv) ? silu_fast(to_f(vg[t * p.ld + c])) : 0.f;
         }
     }
     __syncthreads();
-    float acc[8][4];
+    // M: warps w and w + 4 share 16 rows, taking the 8-column tiles of either half
+    const int rb = w & 3, nh = w >> 2, ntn = rb + 1;
+    float acc[4][4];
 #pragma unroll
-    for (int i = 0; i < 8; ++i)
+    for (int i = 0; i < 4; ++i)
 #pragma unroll
         for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
-#pragma unroll 1
+#pragma unroll 2
     for (int ks = 0; ks < KS; ++ks) {
         AFrag a;
 #pragma unroll
         for (int x = 0; x < 4; ++x) {
-            const int i = 16 * w + r4 + (x & 1) * 8, c = ks * 16 + c2 + (x >> 1) * 8;
-            split2(s.q[i][c], s.q[i][c + 1], a.h[x], a.l[x]);
+            const int i = 16 * rb + r4 + (x & 1) * 8, c = ks * 16 + c2 + (x >> 1) * 8;
+            const float2 f = *reinterpret_cast<const float2*>(&s.q[i][c]);
+            split2(f.x, f.y, a.h[x], a.l[x]);
         }
 #pragma unroll
-        for (int nt = 0; nt < 8; ++nt) {
-            if (nt < 2 * w + 2) {
-                const int j = nt * 8 + r4, c = ks * 16 + c2;
+        for (int nt = 0; nt < 4; ++nt) {
+            if (nt < ntn) {
+                const int j = (nh * ntn + nt) * 8 + r4, c = ks * 16 + c2;
+                const float2 f0 = *reinterpret_cast<const float2*>(&s.k[j][c]), f1 = *reinterpret_cast<const float2*>(&s.k[j][c + 8]);
                 uint32_t bh0, bl0, bh1, bl1;
-                split2(s.k[j][c], s.k[j][c + 1], bh0, bl0);
-                split2(s.k[j][c + 8], s.k[j][c + 9], bh1, bl1);
+                split2(f0.x, f0.y, bh0, bl0);
+                split2(f1.x, f1.y, bh1, bl1);
                 mma_split(acc[nt], a, bh0, bh1, bl0, bl1);
             }
         }
     }
 #pragma unroll
-    for (int nt = 0; nt < 8; ++nt) {
-        if (nt < 2 * w + 2) {
+    for (int nt = 0; nt < 4; ++nt) {
+        if (nt < ntn) {
 #pragma unroll
             for (int hf = 0; hf < 2; ++hf) {
-                const int i = 16 * w + r4 + hf * 8, j = nt * 8 + c2;
+                const int i = 16 * rb + r4 + hf * 8, j = (nh * ntn + nt) * 8 + c2;
                 const float m0 = i >= j ? acc[nt][hf * 2] * s.pw[i - j] : 0.f, m1 = i >= j + 1 ? acc[nt][hf * 2 + 1] * s.pw[i - j - 1] : 0.f;
-                put_split(wb + Ws<DK>::M, kC * kC, i * kC + j, m0, m1);
+                put_split(wM + W::at(kC, i, j), W::M_PLANE, m0, m1);
             }
         }
     }
+    zero_upper(wM, W::M_PLANE, tid);
 #pragma unroll 4
-    for (int e = tid; e < kC * DK / 4; e += 128) {
+    for (int e = tid; e < kC * DK / 4; e += 256) {
         const int t = e / (DK / 4), c = (e % (DK / 4)) * 4;
         const float fq = s.pw[t + 1], fk = t < L ? s.pw[L - 1 - t] : 0.f;
         const float4 qv = *reinterpret_cast<const float4*>(&s.q[t][c]), kv = *reinterpret_cast<const float4*>(&s.k[t][c]);
-        put_split4(wb + Ws<DK>::Q, Ws<DK>::PLANE, t * DK + c, qv.x * fq, qv.y * fq, qv.z * fq, qv.w * fq);
-        put_split4(wb + Ws<DK>::K, Ws<DK>::PLANE, t * DK + c, kv.x * fk, kv.y * fk, kv.z * fk, kv.w * fk);
+        put_split4(ws + W::at(64, t, c), W::A_PLANE, qv.x * fq, qv.y * fq, qv.z * fq, qv.w * fq);
+        put_split4(ws + W::OFF_K + W::at(kC, t, c), W::K_PLANE, kv.x * fk, kv.y * fk, kv.z * fk, kv.w * fk);
     }
-    if (tid < DK) U0[(long long)kC * p.dvp + tid] = s.pw[L];
-}
-
-// ---------------------------------------------------------------------------------------------------------------------
-// the scan: a warp owns 16 value columns of one head, S^T [16][DK] in its accumulators
-// ---------------------------------------------------------------------------------------------------------------------
-template <int DK, bool HASW>
-struct ScanSmem {
-    static constexpr int P = DK + 8, PM = kC + 8;      // padded rows: ldmatrix without bank conflicts
-    __nv_bfloat16 wq[HASW ? 4 : 2][kC][P];             // -W hi, lo, Q~ hi, lo
-    __nv_bfloat16 k[2][kC][P];
-    __nv_bfloat16 m[2][kC][PM];
-    float dec[DK];
-};
-
-template <int DK, bool HASW>
-__global__ void __launch_bounds__(256)
-chunk_scan_kernel(const ChunkParams p) {
-    extern __shared__ uint8_t sm_raw[];
-    using SM = ScanSmem<DK, HASW>;
-    SM& s = *reinterpret_cast<SM*>(sm_raw);
-    constexpr int KS = DK / 16, NT = DK / 8;
-    const int tid = threadIdx.x, w = tid >> 5, lane = tid & 31, r4 = lane >> 2, c2 = (lane & 3) * 2;
-    const int h = blockIdx.y, b = blockIdx.z;
-    const int col0 = ((int)blockIdx.x * (int)(blockDim.x >> 5) + w) * 16;             // first value column of the warp
-    const bool act = col0 < p.dv;                               // an idle warp still helps to load
-    const int d0 = col0 + r4, d1 = d0 + 8;
-    const uint8_t* ws0 = p.ws + ((long long)b * p.H + h) * p.chunks * p.ws_stride;
-    float* Sg = p.state + ((long long)b * p.H + h) * p.dk * (long long)p.dv;
-
-    auto load_rows = [&](__nv_bfloat16* dst, int pitch, const __nv_bfloat16* src, int width, int planes) {   // planes of [64][width]
-        const int per = width / 8, total = planes * kC * per;
-        for (int e = tid; e < total; e += (int)blockDim.x) {
-            const int row = e / per, c = e - row * per;
-            cp16(smem_u32(dst + (long long)row * pitch + c * 8), src + (long long)row * width + c * 8);
-        }
-    };
-    auto load_wq = [&](int ch) {
-        const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(ws0 + (long long)ch * p.ws_stride);
-        load_rows(&s.wq[0][0][0], SM::P, src + (HASW ? Ws<DK>::W : Ws<DK>::Q), DK, HASW ? 4 : 2);
-    };
-    auto load_mk = [&](int ch) {
-        const uint8_t* base = ws0 + (long long)ch * p.ws_stride;
-        const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(base);
-        load_rows(&s.m[0][0][0], SM::PM, src + Ws<DK>::M, kC, 2);
-        load_rows(&s.k[0][0][0], SM::P, src + Ws<DK>::K, DK, 2);
-        const float* dsrc = reinterpret_cast<const float*>(base + Ws<DK>::U_BYTES) + (long long)kC * p.dvp;
-        if (tid < DK / 4) cp16(smem_u32(&s.dec[tid * 4]), dsrc + tid * 4);
-    };
-    float S[NT][4];
-#pragma unroll
-    for (int nt = 0; nt < NT; ++nt)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int c = nt * 8 + c2 + (e & 1), d = e < 2 ? d0 : d1;
-            S[nt][e] = (act && c < p.dk && d < p.dv) ? Sg[(long long)c * p.dv + d] : 0.f;
-        }
-    float u[8][4];
-    auto load_u0 = [&](int ch) {
-        const float* U0 = reinterpret_cast<const float*>(ws0 + (long long)ch * p.ws_stride + Ws<DK>::U_BYTES);
-#pragma unroll
-        for (int nt = 0; nt < 8; ++nt)
-#pragma unroll
-            for (int e = 0; e < 4; ++e)
-                u[nt][e] = act ? __ldcs(U0 + (long long)(nt * 8 + c2 + (e & 1)) * p.dvp + (e < 2 ? d0 : d1)) : 0.f;
-    };
-    load_wq(0); cp_commit();
-    load_mk(0); cp_commit();
-    load_u0(0);
-    // ldmatrix lane addresses: token rows x 16 key columns (two 8-token groups), and for the transposed read 16 tokens x 16 columns
-    const uint32_t lrow = (uint32_t)((lane >> 4) * 8 + (lane & 7)), lcol = (uint32_t)(((lane >> 3) & 1) * 8);
-    const uint32_t trow = (uint32_t)(((lane >> 3) & 1) * 8 + (lane & 7)), tcol = (uint32_t)((lane >> 4) * 8);
-    const uint32_t aWQ = smem_u32(&s.wq[0][lrow][lcol]), aM = smem_u32(&s.m[0][lrow][lcol]), aK = smem_u32(&s.k[0][trow][tcol]);
-    constexpr uint32_t PLANE_B = kC * SM::P * 2, PLANE_M = kC * SM::PM * 2;
-
-    for (int ch = 0; ch < p.chunks; ++ch) {
-        float o[8][4];
-#pragma unroll
-        for (int nt = 0; nt < 8; ++nt)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) o[nt][e] = 0.f;
-        cp_wait<1>();
-        __syncthreads();
-        if (act) {
-#pragma unroll
-            for (int ks = 0; ks < KS; ++ks) {
-                AFrag a;
-                split2(S[2 * ks][0], S[2 * ks][1], a.h[0], a.l[0]);
-                split2(S[2 * ks][2], S[2 * ks][3], a.h[1], a.l[1]);
-                split2(S[2 * ks + 1][0], S[2 * ks + 1][1], a.h[2], a.l[2]);
-                split2(S[2 * ks + 1][2], S[2 * ks + 1][3], a.h[3], a.l[3]);
-#pragma unroll
-                for (int np = 0; np < 4; ++np) {
-                    const uint32_t at = aWQ + (uint32_t)(np * 16 * SM::P + ks * 16) * 2;
-                    uint32_t bh[4], bl[4];
-                    if (HASW) {
-                        ldsm4(bh, at); ldsm4(bl, at + PLANE_B);
-                        mma_split(u[2 * np], a, bh[0], bh[1], bl[0], bl[1]);
-                        mma_split(u[2 * np + 1], a, bh[2], bh[3], bl[2], bl[3]);
-                    }
-                    ldsm4(bh, at + (HASW ? 2 : 0) * PLANE_B); ldsm4(bl, at + (HASW ? 3 : 1) * PLANE_B);
-                    mma_split(o[2 * np], a, bh[0], bh[1], bl[0], bl[1]);
-                    mma_split(o[2 * np + 1], a, bh[2], bh[3], bl[2], bl[3]);
-                }
-            }
-        }
-        __syncthreads();
-        if (ch + 1 < p.chunks) load_wq(ch + 1);
-        cp_commit();
-        cp_wait<1>();
-        __syncthreads();
-        if (act) {
-            AFrag ua[4];
-#pragma unroll
-            for (int ks = 0; ks < 4; ++ks) {
-                split2(u[2 * ks][0], u[2 * ks][1], ua[ks].h[0], ua[ks].l[0]);
-                split2(u[2 * ks][2], u[2 * ks][3], ua[ks].h[1], ua[ks].l[1]);
-                split2(u[2 * ks + 1][0], u[2 * ks + 1][1], ua[ks].h[2], ua[ks].l[2]);
-                split2(u[2 * ks + 1][2], u[2 * ks + 1][3], ua[ks].h[3], ua[ks].l[3]);
-            }
-            if (ch + 1 < p.chunks) load_u0(ch + 1);          // lands under the products below
-#pragma unroll
-            for (int ks = 0; ks < 4; ++ks)
-#pragma unroll
-                for (int np = ks; np < 4; ++np) {            // queries at or after the keys' block
-                    const uint32_t at = aM + (uint32_t)(np * 16 * SM::PM + ks * 16) * 2;
-                    uint32_t bh[4], bl[4];
-                    ldsm4(bh, at); ldsm4(bl, at + PLANE_M);
-                    mma_split(o[2 * np], ua[ks], bh[0], bh[1], bl[0], bl[1]);
-                    mma_split(o[2 * np + 1], ua[ks], bh[2], bh[3], bl[2], bl[3]);
-                }
-            const int t0 = p.t_begin + ch * kC, L = min(kC, p.n - t0);
-            float* og = p.o + (((long long)b * p.n + t0) * p.H + h) * p.dv;
-#pragma unroll
-            for (int nt = 0; nt < 8; ++nt)
-#pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const int t = nt * 8 + c2 + (e & 1), d = e < 2 ? d0 : d1;
-                    if (t < L && d < p.dv) og[(long long)t * p.H * p.dv + d] = o[nt][e];
-                }
-#pragma unroll
-            for (int np = 0; np < NT / 2; ++np) {
-#pragma unroll
-                for (int x = 0; x < 2; ++x) {
-                    const float2 dc = *reinterpret_cast<const float2*>(&s.dec[(2 * np + x) * 8 + c2]);
-                    S[2 * np + x][0] *= dc.x; S[2 * np + x][1] *= dc.y; S[2 * np + x][2] *= dc.x; S[2 * np + x][3] *= dc.y;
-                }
-#pragma unroll
-                for (int ks = 0; ks < 4; ++ks) {
-                    const uint32_t at = aK + (uint32_t)(ks * 16 * SM::P + np * 16) * 2;
-                    uint32_t bh[4], bl[4];
-                    ldsm4t(bh, at); ldsm4t(bl, at + PLANE_B);
-                    mma_split(S[2 * np], ua[ks], bh[0], bh[1], bl[0], bl[1]);
-                    mma_split(S[2 * np + 1], ua[ks], bh[2], bh[3], bl[2], bl[3]);
-                }
-            }
-        }
-        __syncthreads();
-        if (ch + 1 < p.chunks) load_mk(ch + 1);
-        cp_commit();
-    }
-    if (act) {
-#pragma unroll
-        for (int nt = 0; nt < NT; ++nt)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int c = nt * 8 + c2 + (e & 1), d = e < 2 ? d0 : d1;
-                if (c < p.dk && d < p.dv) Sg[(long long)c * p.dv + d] = S[nt][e];
-            }
-    }
+    if (tid < DK) reinterpret_cast<float*>(ws + W::OFF_DEC)[tid] = s.pw[L];
 }
 
 template <int DK, bool DELTA>
 int launch_chunked(ChunkParams p, int B, void* ws, long long ws_bytes, cudaStream_t stream) {
     p.dvp = (p.dv + 15) / 16 * 16;
     p.ws = (uint8_t*)ws;
-    p.ws_stride = Ws<DK>::bytes(p.dvp);
+    p.ws_stride = ChunkWs<DK / 64, DELTA ? 128 : 64>::bytes(p.dvp);
     const long long per_chunk = p.ws_stride * B * p.H;
     const int all = (p.n + kC - 1) / kC;
     long long seg = ws_bytes / per_chunk;
     if (seg < 1) { set_last_error("chunked recurrence: workspace of %lld bytes holds no chunk (%lld needed)", ws_bytes, per_chunk); return PLZ_ERR_WORKSPACE; }
+    if ((uintptr_t)ws & 15) { set_last_error("chunked recurrence: workspace must be 16-byte aligned"); return PLZ_ERR_BAD_ALIGN; }
     if (seg > all) seg = all;
     const long long rounds = (all + seg - 1) / seg;
     seg = (all + rounds - 1) / rounds;
-    const int smem1 = DELTA ? (int)sizeof(DeltaSmem<DK>) : (int)sizeof(DecaySmem<DK>), smem2 = (int)sizeof(ScanSmem<DK, DELTA>);
+    const int smem = DELTA ? (int)sizeof(DeltaSmem<DK>) : (int)sizeof(DecaySmem<DK>);
     static bool once[64] = {};
     int dev = 0;
     PLZ_CUDA_CHECK(cudaGetDevice(&dev));
     if (!once[dev & 63]) {
-        if (DELTA) PLZ_CUDA_CHECK(cudaFuncSetAttribute(delta_chunk_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem1));
-        else PLZ_CUDA_CHECK(cudaFuncSetAttribute(decay_chunk_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem1));
-        PLZ_CUDA_CHECK(cudaFuncSetAttribute((chunk_scan_kernel<DK, DELTA>), cudaFuncAttributeMaxDynamicSharedMemorySize, smem2));
+        if (DELTA) PLZ_CUDA_CHECK(cudaFuncSetAttribute(delta_chunk_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+        else PLZ_CUDA_CHECK(cudaFuncSetAttribute(decay_chunk_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
         once[dev & 63] = true;
     }
     for (int c0 = 0; c0 < all; c0 += (int)seg) {
         p.t_begin = c0 * kC;
         p.chunks = all - c0 < (int)seg ? all - c0 : (int)seg;
-        if (DELTA) delta_chunk_kernel<DK><<<dim3(p.chunks, p.H, B), 256, smem1, stream>>>(p);
-        else decay_chunk_kernel<DK><<<dim3(p.chunks, p.H, B), 128, smem1, stream>>>(p);
+        if (DELTA) delta_chunk_kernel<DK><<<dim3(p.chunks, p.H, B), 256, smem, stream>>>(p);
+        else decay_chunk_kernel<DK><<<dim3(p.chunks, p.H, B), 256, smem, stream>>>(p);
         PLZ_LAUNCH_CHECK();
-        // four warps (64 value columns) per CTA while that leaves SMs free, else eight on one copy of the chunk's operands
-        const int warps = (long long)B * p.H * ((p.dv + 63) / 64) > seq_sm_count() && p.dv > 64 ? 8 : 4;
-        chunk_scan_kernel<DK, DELTA><<<dim3((p.dv + 16 * warps - 1) / (16 * warps), p.H, B), 32 * warps, smem2, stream>>>(p);
-        PLZ_LAUNCH_CHECK();
+        const ScanArgs a = {p.ws, p.ws_stride, p.state, p.o, B, p.n, p.t_begin, p.chunks, p.H, p.dk, p.dv, p.dvp};
+        const int rc = launch_chunk_scan(a, DELTA, DK / 64, stream);
+        if (rc) return rc;
     }
     return PLZ_OK;
 }
 template <bool DELTA>
 int launch_dk(const ChunkParams& p, int B, void* ws, long long ws_bytes, cudaStream_t stream) {
-    if (p.dk <= 32) return launch_chunked<32, DELTA>(p, B, ws, ws_bytes, stream);
     if (p.dk <= 64) return launch_chunked<64, DELTA>(p, B, ws, ws_bytes, stream);
     if (p.dk <= 128) return launch_chunked<128, DELTA>(p, B, ws, ws_bytes, stream);
     set_last_error("chunked recurrence: key size %d (at most 128)", p.dk);
@@ -718,8 +528,8 @@ int launch_dk(const ChunkParams& p, int B, void* ws, long long ws_bytes, cudaStr
 // bytes that hold every chunk of n tokens; any amount down to one chunk of all heads works (the scan then runs in segments)
 long long chunk_ws_bytes(int B, int n, int H, int dk, int dv) {
     if (dk > 128) return 0;
-    const int dvp = (dv + 15) / 16 * 16, DK = dk <= 32 ? 32 : (dk <= 64 ? 64 : 128);
-    const long long per = DK == 32 ? Ws<32>::bytes(dvp) : (DK == 64 ? Ws<64>::bytes(dvp) : Ws<128>::bytes(dvp));
+    const int dvp = (dv + 15) / 16 * 16;
+    const long long per = dk <= 64 ? ChunkWs<1, 128>::bytes(dvp) : ChunkWs<2, 128>::bytes(dvp);
     const long long one = per * B * H, all = one * ((n + kC - 1) / kC), cap = 96ll << 20;   // stay inside L2 when there is a choice
     return all <= cap ? all : (one > cap ? one : cap / one * one);
 }

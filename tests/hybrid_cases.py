@@ -26,7 +26,7 @@ def config(layers, width=56, vocab=73, ff=88, eps=3e-5, scale=1.7, mult=0.6):
 
 CONFIGS = {
     "all": config([lightning(), delta(), attention(), delta(heads=3, kv_heads=3), attention(), lightning(heads=1)]),
-    "attention_first": config([attention(v_mix=False), attention(heads=4, kv_heads=4, dim=40), attention(heads=2, kv_heads=2, dim=8, vdim=32), attention()], width=64),
+    "attention_first": config([attention(v_mix=False), attention(heads=4, kv_heads=4, dim=40), attention(heads=2, kv_heads=2, dim=8, vdim=32), attention(vdim=32)], width=64),
     "no_mlp": config([dict(delta(conv=1), mlp=None), lightning(heads=3, dim=8, vdim=40), dict(attention(heads=1, kv_heads=1), mlp=None)], width=48, mult=1.0, scale=1.0),
     "odd_sizes": config([attention(heads=3, kv_heads=1, dim=10, vdim=7), delta(heads=2, kv_heads=1, dim=5, vdim=9, conv=4), lightning(heads=3, dim=6, vdim=11)],
                         width=30, vocab=41, ff=34),

@@ -114,7 +114,7 @@ def test_interleaved_requests_and_reused_slots(dt):
         got[r].append(eng.step(r, part, range(len(part)), end=at + len(part) == len(reqs[r])))
     for r, n in (("a", 70), ("b", 30), ("a", 1), ("b", 1), ("c", 2), ("a", 1), ("d", 3), ("a", 66), ("d", 1), ("e", 1), ("d", 93), ("a", 12), ("f", 64)):
         step(r, n)
-    assert not eng.pool.live and len(eng.pool.free) == 2          # never more than two at once
+    assert not eng.pool.live and len(eng.pool.free) == 3          # three slots served six requests
     for r in reqs:
         assert H.error(torch.cat(got[r]), H.expected(cfg, W, reqs[r])) < H.TOL[dt], r
 
