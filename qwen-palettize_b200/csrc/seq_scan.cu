@@ -162,10 +162,15 @@ scan_kernel(const ScanArgs p, StatusWord* status) {
             for (int cb = 0; cb < 2; ++cb) {
                 uint32_t v[32];
                 tmem_ld_32x32(tmem + lo + C::T_UO + 128u * (ch & 1) + 64u + cb * 32u, v);
-                if (live) {
+                if (!live) continue;
+                float* at = og + (long long)cb * 32 * pitch;
+                if (L == kC) {
 #pragma unroll
-                    for (int i = 0; i < 32; ++i)
-                        if (cb * 32 + i < L) og[(long long)(cb * 32 + i) * pitch] = __uint_as_float(v[i]);
+                    for (int i = 0; i < 32; ++i, at += pitch) __stcs(at, __uint_as_float(v[i]));
+                } else {
+#pragma unroll
+                    for (int i = 0; i < 32; ++i, at += pitch)
+                        if (cb * 32 + i < L) *at = __uint_as_float(v[i]);
                 }
             }
         };
