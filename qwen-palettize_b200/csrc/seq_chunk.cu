@@ -29,6 +29,18 @@ __device__ __forceinline__ float ex2a(float x) { float y; asm("ex2.approx.ftz.f3
 
 // z / (1 + e^-z) of a bf16 input, about 2^-21 relative
 __device__ __forceinline__ float silu_fast(float z) { return __fdividef(z, 1.0f + ex2a(-z * kL2e)); }
+// two fp32 per instruction
+struct F2x2 { uint64_t a, b; };
+__device__ __forceinline__ F2x2 ld_f2x2(const float* p) {
+    const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(p);
+    return {v.x, v.y};
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) { uint64_t d; asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c)); return d; }
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) { uint64_t d; asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b)); return d; }
+__device__ __forceinline__ uint64_t sub2(uint64_t a, uint64_t b) { uint64_t d; asm("sub.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b)); return d; }
+__device__ __forceinline__ uint64_t ex2_2(uint64_t a) {
+    return (uint64_t)__float_as_uint(ex2a(__uint_as_float((uint32_t)a))) | ((uint64_t)__float_as_uint(ex2a(__uint_as_float((uint32_t)(a >> 32)))) << 32);
+}
 __device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
     asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
                  : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
@@ -102,12 +114,12 @@ delta_chunk_kernel(const ChunkParams p) {
 #pragma unroll
         for (int i = 0; i < kC * DK / 4 / 256; ++i) {
             const int e = tid + i * 256, t = e / (DK / 4), c = (e % (DK / 4)) * 4;
-            float4 qv = make_float4(0.f, 0.f, 0.f, 0.f), kv = qv, gv = qv;
-            if (t < L && c < p.dk) {
-                qv = __ldg(reinterpret_cast<const float4*>(qg + t * ldq + c));
-                kv = __ldg(reinterpret_cast<const float4*>(kg + t * ldq + c));
-                gv = __ldg(reinterpret_cast<const float4*>(gg + t * ldg + c));
-            }
+            // unconditional loads from a clamped place: a branch around each would serialise them
+            const int tc = min(t, L - 1), cc = min(c, p.dk - 4);
+            const float m = t < L && c < p.dk ? 1.f : 0.f;
+            float4 qv = __ldg(reinterpret_cast<const float4*>(qg + tc * ldq + cc)), kv = __ldg(reinterpret_cast<const float4*>(kg + tc * ldq + cc));
+            float4 gv = __ldg(reinterpret_cast<const float4*>(gg + tc * ldg + cc));
+            if (m == 0.f) { qv = make_float4(0.f, 0.f, 0.f, 0.f); kv = qv; gv = qv; }
             *reinterpret_cast<float4*>(&s.q[t][c]) = qv;
             *reinterpret_cast<float4*>(&s.k[t][c]) = kv;
             *reinterpret_cast<float4*>(&s.b[t][c]) = make_float4(gv.x * kL2e, gv.y * kL2e, gv.z * kL2e, gv.w * kL2e);
@@ -209,36 +221,40 @@ delta_chunk_kernel(const ChunkParams p) {
         const int rb = w - 4;
         for (int blk = 0; blk < 2; ++blk) {
             const int base = 16 * rb + 8 * blk, ri = lane & 7, row = base + ri, quarter = lane >> 3;
-            float ak[8], aq[8];
+            uint64_t ak[8], aq[8];          // pairs of partial sums
 #pragma unroll
-            for (int j = 0; j < 8; ++j) { ak[j] = 0.f; aq[j] = 0.f; }
+            for (int j = 0; j < 8; ++j) { ak[j] = 0ull; aq[j] = 0ull; }
 #pragma unroll 1
             for (int c4 = quarter; c4 < DK / 4; c4 += 4) {
                 const int c = c4 * 4;
-                const float4 bi = *reinterpret_cast<const float4*>(&s.b[row][c]), ki = *reinterpret_cast<const float4*>(&s.k[row][c]);
-                const float4 qi = *reinterpret_cast<const float4*>(&s.q[row][c]);
+                const F2x2 bi = ld_f2x2(&s.b[row][c]), ki = ld_f2x2(&s.k[row][c]), qi = ld_f2x2(&s.q[row][c]);
 #pragma unroll
                 for (int j = 0; j < 8; ++j) {
-                    const float4 bj = *reinterpret_cast<const float4*>(&s.b[base + j][c]), kj = *reinterpret_cast<const float4*>(&s.k[base + j][c]);
+                    const F2x2 bj = ld_f2x2(&s.b[base + j][c]), kj = ld_f2x2(&s.k[base + j][c]);
                     // j > row: an exponent above zero, discarded below
-                    const float e0 = ex2a(bi.x - bj.x) * kj.x, e1 = ex2a(bi.y - bj.y) * kj.y;
-                    const float e2 = ex2a(bi.z - bj.z) * kj.z, e3 = ex2a(bi.w - bj.w) * kj.w;
-                    ak[j] += ki.x * e0 + ki.y * e1 + ki.z * e2 + ki.w * e3;
-                    aq[j] += qi.x * e0 + qi.y * e1 + qi.z * e2 + qi.w * e3;
+                    const uint64_t e0 = mul2(ex2_2(sub2(bi.a, bj.a)), kj.a), e1 = mul2(ex2_2(sub2(bi.b, bj.b)), kj.b);
+                    ak[j] = fma2(ki.a, e0, ak[j]); ak[j] = fma2(ki.b, e1, ak[j]);
+                    aq[j] = fma2(qi.a, e0, aq[j]); aq[j] = fma2(qi.b, e1, aq[j]);
                 }
+            }
+            float sk[8], sq[8];
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                sk[j] = __uint_as_float((uint32_t)ak[j]) + __uint_as_float((uint32_t)(ak[j] >> 32));
+                sq[j] = __uint_as_float((uint32_t)aq[j]) + __uint_as_float((uint32_t)(aq[j] >> 32));
             }
 #pragma unroll
             for (int j = 0; j < 8; ++j) {
-                ak[j] += __shfl_xor_sync(0xFFFFFFFFu, ak[j], 8); ak[j] += __shfl_xor_sync(0xFFFFFFFFu, ak[j], 16);
-                aq[j] += __shfl_xor_sync(0xFFFFFFFFu, aq[j], 8); aq[j] += __shfl_xor_sync(0xFFFFFFFFu, aq[j], 16);
+                sk[j] += __shfl_xor_sync(0xFFFFFFFFu, sk[j], 8); sk[j] += __shfl_xor_sync(0xFFFFFFFFu, sk[j], 16);
+                sq[j] += __shfl_xor_sync(0xFFFFFFFFu, sq[j], 8); sq[j] += __shfl_xor_sync(0xFFFFFFFFu, sq[j], 16);
             }
             if (quarter == 0) {
 #pragma unroll
-                for (int j = 0; j < 8; ++j) s.a[rb * (rb + 1) / 2 + rb][8 * blk + ri][8 * blk + j] = j < ri ? ak[j] * s.beta[row] : 0.f;
+                for (int j = 0; j < 8; ++j) s.a[rb * (rb + 1) / 2 + rb][8 * blk + ri][8 * blk + j] = j < ri ? sk[j] * s.beta[row] : 0.f;
             } else if (quarter == 1) {
 #pragma unroll
                 for (int j = 0; j < 8; j += 2)
-                    put_split(wM + W::at(kC, row, base + j), W::M_PLANE, j <= ri ? aq[j] : 0.f, j + 1 <= ri ? aq[j + 1] : 0.f);
+                    put_split(wM + W::at(kC, row, base + j), W::M_PLANE, j <= ri ? sq[j] : 0.f, j + 1 <= ri ? sq[j + 1] : 0.f);
             } else if (quarter == 2 && blk == 0) {
                 // rows 0..7 against columns 8..15 of the 16-row block lie above the diagonal
 #pragma unroll
@@ -325,6 +341,8 @@ delta_chunk_kernel(const ChunkParams p) {
         }
     }
     const int nt_w = DK / 8, nt_all = nt_w + p.dvp / 8;
+    const float* vg = (const float*)p.v + (row0 * p.H + h) * (long long)p.dv;
+    const long long ldv = (long long)p.H * p.dv;
 #pragma unroll 1
     for (int nt = w & 3; nt < nt_all; nt += 4) {
         const bool is_w = nt < nt_w;
@@ -335,11 +353,8 @@ delta_chunk_kernel(const ChunkParams p) {
 #pragma unroll
             for (int x = 0; x < 4; ++x) {
                 const int j = 16 * ks + c2 + (x & 1) + (x >> 1) * 8;
-                f[ks][x] = 0.f;
-                if (ks <= m1) {
-                    if (is_w) f[ks][x] = -s.k[j][c];
-                    else if (j < L && c < p.dv) f[ks][x] = __ldg((const float*)p.v + ((row0 + j) * p.H + h) * (long long)p.dv + c);
-                }
+                // past the last token T's column has beta = 0, past the last value column nobody reads: any finite value will do
+                f[ks][x] = is_w ? -s.k[j][c] : __ldg(vg + (long long)min(j, L - 1) * ldv + min(c, p.dv - 1));
             }
         float acc0[4] = {0.f, 0.f, 0.f, 0.f}, acc1[4] = {0.f, 0.f, 0.f, 0.f};
         uint32_t bh[4][2], bl[4][2];
@@ -401,7 +416,8 @@ decay_chunk_kernel(const ChunkParams p) {
             const int t = e / (DK / 8), c = (e % (DK / 8)) * 8;
             float fq[8], fk[8];
             const bool in = t < L && c < p.dk;
-            if (in) { load8(qg + t * p.ld + c, fq); load8(kg + t * p.ld + c, fk); }
+            const long long at = min(t, L - 1) * p.ld + min(c, p.dk - 8);      // unconditional loads
+            load8(qg + at, fq); load8(kg + at, fk);
 #pragma unroll
             for (int i = 0; i < 8; ++i) { s.q[t][c + i] = in ? silu_fast(fq[i]) : 0.f; s.k[t][c + i] = in ? silu_fast(fk[i]) : 0.f; }
         }
@@ -411,7 +427,7 @@ decay_chunk_kernel(const ChunkParams p) {
             const int t = e / v8, c = (e - t * v8) * 8;
             float f[8];
             const bool in = t < L && c < p.dv;
-            if (in) load8(vg + t * p.ld + c, f);
+            load8(vg + min(t, L - 1) * p.ld + min(c, p.dv - 8), f);
 #pragma unroll
             for (int i = 0; i < 8; ++i) f[i] = in ? silu_fast(f[i]) : 0.f;
             *reinterpret_cast<float4*>(U0 + (long long)t * p.dvp + c) = make_float4(f[0], f[1], f[2], f[3]);
@@ -530,7 +546,7 @@ long long chunk_ws_bytes(int B, int n, int H, int dk, int dv) {
     if (dk > 128) return 0;
     const int dvp = (dv + 15) / 16 * 16;
     const long long per = dk <= 64 ? ChunkWs<1, 128>::bytes(dvp) : ChunkWs<2, 128>::bytes(dvp);
-    const long long one = per * B * H, all = one * ((n + kC - 1) / kC), cap = 96ll << 20;   // stay inside L2 when there is a choice
+    const long long one = per * B * H, all = one * ((n + kC - 1) / kC), cap = 512ll << 20;
     return all <= cap ? all : (one > cap ? one : cap / one * one);
 }
 
