@@ -65,7 +65,7 @@ __device__ __forceinline__ void mma_pv(uint32_t d, uint32_t sP, uint32_t sV, boo
 }
 
 struct Group {
-    uint32_t tS, tO, s_full, p_full, o_full;
+    uint32_t tS, tO, s_full, p_full, o_full, out_ready;
     uint8_t* pP; uint32_t sP;
     int qt, n_kv;              // query tile; key tiles it walks
 };
@@ -104,7 +104,7 @@ __device__ __forceinline__ float exp_pass(const Group& G, uint32_t lane_off, int
 
 template <int DVB>
 __device__ __forceinline__ void softmax_group(const Group& G, const TcParams& p, const CUtensorMap* tmO, int h, int b, int warp_in_group, int lane,
-                                              int bar_id, volatile uint32_t* abort_flag) {
+                                              volatile uint32_t* abort_flag) {
     const int r = warp_in_group * 32 + lane;
     const uint32_t lane_off = (uint32_t)(warp_in_group * 32) << 16;
     const float c = p.scale_log2e;
@@ -178,8 +178,9 @@ __device__ __forceinline__ void softmax_group(const Group& G, const TcParams& p,
             }
         }
         fence_proxy_async_smem();
-        asm volatile("bar.sync %0, 128;" ::"r"(bar_id) : "memory");
-        if (r == 0) {
+        __syncwarp();
+        if (lane == 0) mbar_arrive(G.out_ready);
+        if (r == 0 && mbar_wait(G.out_ready, 0, abort_flag, p.status, ST_TIMEOUT_ACCUM, 23)) {
             for (int i = 0; i < p.dv_blocks; ++i) tma_store_4d(tmO, G.sP + i * kBlk, i * 64, h, G.qt * kT, b);
             tma_store_commit();
             tma_store_wait_all();
@@ -202,7 +203,8 @@ attn_bias_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     auto s_full = [&](int g) { return bar + 56u + 8u * g; };
     auto p_full = [&](int g) { return bar + 72u + 8u * g; };
     auto o_full = [&](int g) { return bar + 88u + 8u * g; };
-    volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(smem + C::OFF_BAR + 112);
+    auto out_ready = [&](int g) { return bar + 104u + 8u * g; };
+    volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(smem + C::OFF_BAR + 128);
     volatile uint32_t* abort_flag = tmem_slot + 1;
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -221,7 +223,7 @@ attn_bias_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         mbar_init(q_full, 1); mbar_init(v_full, 1); mbar_init(v_empty, 1);
         for (int i = 0; i < 2; ++i) {
             mbar_init(k_full0 + 8 * i, 1); mbar_init(k_empty0 + 8 * i, 1);
-            mbar_init(s_full(i), 1); mbar_init(p_full(i), 4); mbar_init(o_full(i), 1);
+            mbar_init(s_full(i), 1); mbar_init(p_full(i), 4); mbar_init(o_full(i), 1); mbar_init(out_ready(i), 4);
         }
         *abort_flag = 0;
         mbar_fence_init();
@@ -297,9 +299,9 @@ attn_bias_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         const int g = warp >> 2;
         if (g == 0 || hasB) {
             Group G;
-            G.tS = tS(g); G.tO = tO(g); G.s_full = s_full(g); G.p_full = p_full(g); G.o_full = o_full(g);
+            G.tS = tS(g); G.tO = tO(g); G.s_full = s_full(g); G.p_full = p_full(g); G.o_full = o_full(g); G.out_ready = out_ready(g);
             G.pP = smem + C::OFF_P + g * C::P; G.sP = sP0 + g * C::P; G.qt = g == 0 ? qtA : qtB; G.n_kv = g == 0 ? n_kvA : n_kv;
-            softmax_group<DVB>(G, p, &tmO, h, b, warp & 3, lane, 1 + g, abort_flag);
+            softmax_group<DVB>(G, p, &tmO, h, b, warp & 3, lane, abort_flag);
         }
     }
     tc_fence_before_sync();

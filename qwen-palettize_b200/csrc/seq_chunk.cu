@@ -41,6 +41,12 @@ __device__ __forceinline__ uint64_t sub2(uint64_t a, uint64_t b) { uint64_t d; a
 __device__ __forceinline__ uint64_t ex2_2(uint64_t a) {
     return (uint64_t)__float_as_uint(ex2a(__uint_as_float((uint32_t)a))) | ((uint64_t)__float_as_uint(ex2a(__uint_as_float((uint32_t)(a >> 32)))) << 32);
 }
+// 16 bytes global -> shared, zeros when !in (the address must be valid all the same)
+__device__ __forceinline__ void cp16z(uint32_t dst, const void* src, bool in) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(in ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+__device__ __forceinline__ void cp_wait_all() { asm volatile("cp.async.wait_all;" ::: "memory"); }
 __device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
     asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
                  : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
@@ -72,7 +78,7 @@ struct ChunkParams {
     uint8_t* ws; long long ws_stride;
     int n, t_begin, chunks;      // tokens per sequence; first token and number of chunks of this segment
     int H, G, dk, dv, dvp;
-    int vec;                     // rows allow 16-byte loads
+    int vec, vec_v;              // rows (of v) allow 16-byte loads
 };
 
 // ---------------------------------------------------------------------------------------------------------------------
@@ -114,33 +120,31 @@ delta_chunk_kernel(const ChunkParams p) {
 #pragma unroll
         for (int i = 0; i < kC * DK / 4 / 256; ++i) {
             const int e = tid + i * 256, t = e / (DK / 4), c = (e % (DK / 4)) * 4;
-            // unconditional loads from a clamped place: a branch around each would serialise them
+            const bool in = t < L && c < p.dk;
             const int tc = min(t, L - 1), cc = min(c, p.dk - 4);
-            const float m = t < L && c < p.dk ? 1.f : 0.f;
-            float4 qv = __ldg(reinterpret_cast<const float4*>(qg + tc * ldq + cc)), kv = __ldg(reinterpret_cast<const float4*>(kg + tc * ldq + cc));
-            float4 gv = __ldg(reinterpret_cast<const float4*>(gg + tc * ldg + cc));
-            if (m == 0.f) { qv = make_float4(0.f, 0.f, 0.f, 0.f); kv = qv; gv = qv; }
-            *reinterpret_cast<float4*>(&s.q[t][c]) = qv;
-            *reinterpret_cast<float4*>(&s.k[t][c]) = kv;
-            *reinterpret_cast<float4*>(&s.b[t][c]) = make_float4(gv.x * kL2e, gv.y * kL2e, gv.z * kL2e, gv.w * kL2e);
+            cp16z(smem_u32(&s.q[t][c]), qg + tc * ldq + cc, in);
+            cp16z(smem_u32(&s.k[t][c]), kg + tc * ldq + cc, in);
+            cp16z(smem_u32(&s.b[t][c]), gg + tc * ldg + cc, in);
         }
+        cp_commit();
     } else {
         for (int e = tid; e < kC * DK; e += 256) {
             const int t = e / DK, c = e % DK;
             const bool in = t < L && c < p.dk;
             s.q[t][c] = in ? qg[t * ldq + c] : 0.f;
             s.k[t][c] = in ? kg[t * ldq + c] : 0.f;
-            s.b[t][c] = in ? gg[t * ldg + c] * kL2e : 0.f;
+            s.b[t][c] = in ? gg[t * ldg + c] : 0.f;
         }
     }
     if (tid < kC) s.beta[tid] = tid < L ? p.beta[(row0 + tid) * p.H + h] : 0.f;
+    cp_wait_all();
     __syncthreads();
     // inclusive sum over the 64 tokens, two threads per channel (the second half adds the first half's total)
     if (tid < 2 * DK) {
         const int c = tid % DK, h0 = tid / DK * 32;
         float run = 0.f;
 #pragma unroll 16
-        for (int t = 0; t < 32; ++t) { run += s.b[h0 + t][c]; s.b[h0 + t][c] = run; }
+        for (int t = 0; t < 32; ++t) { run = fmaf(s.b[h0 + t][c], kL2e, run); s.b[h0 + t][c] = run; }
     }
     __syncthreads();
     for (int e = tid; e < 32 * DK; e += 256) s.b[32 + e / DK][e % DK] += s.b[31][e % DK];
@@ -278,6 +282,18 @@ delta_chunk_kernel(const ChunkParams p) {
     if (tid < DK) reinterpret_cast<float*>(ws + W::OFF_DEC)[tid] = ex2a(s.b[kC - 1][tid]);
     zero_upper(wM, W::M_PLANE, tid);
     __syncthreads();
+    // the values take the place of q while T is computed
+    const float* vg = (const float*)p.v + (row0 * p.H + h) * (long long)p.dv;
+    const long long ldv = (long long)p.H * p.dv;
+    const bool v_in_smem = p.vec_v && p.dv <= DK;
+    if (v_in_smem) {
+#pragma unroll
+        for (int i = 0; i < kC * DK / 4 / 256; ++i) {
+            const int e = tid + i * 256, t = e / (DK / 4), c = (e % (DK / 4)) * 4;
+            cp16z(smem_u32(&s.q[t][c]), vg + (long long)min(t, L - 1) * ldv + min(c, p.dv - 4), t < L && c < p.dv);
+        }
+        cp_commit();
+    }
 
     // ---- T = (I + a)^{-1}: 16-row diagonal blocks by substitution, then block diagonals outwards -------------------------
     if (w < 4 && lane < 16) {
@@ -341,8 +357,8 @@ delta_chunk_kernel(const ChunkParams p) {
         }
     }
     const int nt_w = DK / 8, nt_all = nt_w + p.dvp / 8;
-    const float* vg = (const float*)p.v + (row0 * p.H + h) * (long long)p.dv;
-    const long long ldv = (long long)p.H * p.dv;
+    cp_wait_all();
+    __syncthreads();
 #pragma unroll 1
     for (int nt = w & 3; nt < nt_all; nt += 4) {
         const bool is_w = nt < nt_w;
@@ -353,8 +369,10 @@ delta_chunk_kernel(const ChunkParams p) {
 #pragma unroll
             for (int x = 0; x < 4; ++x) {
                 const int j = 16 * ks + c2 + (x & 1) + (x >> 1) * 8;
+                if (is_w) f[ks][x] = -s.k[j][c];
+                else if (v_in_smem) f[ks][x] = s.q[j][c];
                 // past the last token T's column has beta = 0, past the last value column nobody reads: any finite value will do
-                f[ks][x] = is_w ? -s.k[j][c] : __ldg(vg + (long long)min(j, L - 1) * ldv + min(c, p.dv - 1));
+                else f[ks][x] = __ldg(vg + (long long)min(j, L - 1) * ldv + min(c, p.dv - 1));
             }
         float acc0[4] = {0.f, 0.f, 0.f, 0.f}, acc1[4] = {0.f, 0.f, 0.f, 0.f};
         uint32_t bh[4][2], bl[4][2];
@@ -561,6 +579,7 @@ int launch_chunk_delta(const DeltaRuleArgs& a, void* ws, long long ws_bytes, cud
     ChunkParams p = {};
     p.q = a.q; p.k = a.k; p.v = a.v; p.logg = a.logg; p.beta = a.beta; p.state = a.state; p.o = a.o;
     p.n = a.n; p.H = a.H; p.G = a.G; p.dk = a.dk; p.dv = a.dv;
+    p.vec_v = a.dv % 4 == 0 && !((uintptr_t)a.v & 15);
     p.vec = a.dk % 4 == 0 && !(((uintptr_t)a.q | (uintptr_t)a.k | (uintptr_t)a.logg) & 15);
     return launch_dk<true>(p, a.B, ws, ws_bytes, stream);
 }

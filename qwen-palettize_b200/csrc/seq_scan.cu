@@ -4,7 +4,7 @@
 // Everything is transposed: the state is S^T [value column = TMEM lane][key column], so the state and U are A operands of M = 128
 // products straight from tensor memory and only chunk constants come through shared memory. Per chunk
 //
-//   1. the four epilogue warps (thread = value column) read S^T, write it back times e^{b_C}, and write its bf16 halves hi + lo as an
+//   1. the eight epilogue warps (thread = value column and half of the columns) read S^T, write it back times e^{b_C}, and write its bf16 halves hi + lo as an
 //      A operand into TMEM
 //   2. MMA:  [U' | O] = S^T (-W | Q~)^T                        three products hi hi + hi lo + lo hi
 //   3. epilogue warps: U = U' + U0 (global memory), halves hi + lo over U' in place
@@ -19,7 +19,7 @@
 namespace plz {
 namespace {
 
-constexpr int kScanThreads = 192;   // warps 0-3 epilogue, 4 MMA, 5 copies
+constexpr int kScanThreads = 320;   // warps 0-7 epilogue (two per 32 value columns, half of the TMEM columns each), 8 MMA, 9 copies
 
 __device__ __forceinline__ void bulk_load(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {
     asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst), "l"(src), "r"(bytes), "r"(bar) : "memory");
@@ -64,7 +64,8 @@ scan_kernel(const ScanArgs p, StatusWord* status) {
     auto a_free = [&](int s) { return bar + 32u + 8u * s; };      // the products that read it have completed
     auto b_free = [&](int s) { return bar + 48u + 8u * s; };
     const uint32_t s_ready = bar + 64, uo_full = bar + 72, u_ready = bar + 80, fin_full = bar + 88;
-    volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(smem + C::OFF_BAR + 96);
+    auto u_read = [&](int q) { return bar + 96u + 8u * q; };      // both warps of a lane quarter have read U'
+    volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(smem + C::OFF_BAR + 128);
     volatile uint32_t* abort_flag = tmem_slot + 1;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int h = blockIdx.y, b = blockIdx.z;
@@ -72,17 +73,18 @@ scan_kernel(const ScanArgs p, StatusWord* status) {
 
     if (threadIdx.x == 0) {
         for (int s = 0; s < 2; ++s) { mbar_init(a_full(s), 1); mbar_init(b_full(s), 1); mbar_init(a_free(s), 1); mbar_init(b_free(s), 1); }
-        mbar_init(s_ready, 4); mbar_init(uo_full, 1); mbar_init(u_ready, 4); mbar_init(fin_full, 1);
+        for (int q = 0; q < 4; ++q) mbar_init(u_read(q), 2);
+        mbar_init(s_ready, 8); mbar_init(uo_full, 1); mbar_init(u_ready, 8); mbar_init(fin_full, 1);
         *abort_flag = 0;
         mbar_fence_init();
     }
-    if (warp == 4) { tmem_alloc(smem_u32((const void*)tmem_slot), 512); tmem_relinquish(); }
+    if (warp == 8) { tmem_alloc(smem_u32((const void*)tmem_slot), 512); tmem_relinquish(); }
     tc_fence_before_sync();
     __syncthreads();
     tc_fence_after_sync();
     const uint32_t tmem = *tmem_slot;
 
-    if (warp == 5) {
+    if (warp == 9) {
         if (lane == 0) {
             bool ok = true;
             int in_a = 0, in_b = 0;                       // chunks whose copies have been issued
@@ -108,7 +110,7 @@ scan_kernel(const ScanArgs p, StatusWord* status) {
             for (int ch = in_b > 2 ? in_b - 2 : 0; ch < in_b; ++ch)
                 while (!mbar_try_wait(b_full(ch & 1), (ch >> 1) & 1) && globaltimer_ns() - t0 < 100000000ull) {}
         }
-    } else if (warp == 4) {
+    } else if (warp == 8) {
         if (lane == 0) {
             bool ok = true;
             constexpr uint32_t n1 = HASW ? 128 : 64;
@@ -149,8 +151,9 @@ scan_kernel(const ScanArgs p, StatusWord* status) {
             }
         }
     } else {
-        const int d = (int)blockIdx.x * 128 + warp * 32 + lane;      // value column
-        const uint32_t lo = (uint32_t)(warp * 32) << 16;
+        const int quarter = warp & 3, half = warp >> 2;
+        const int d = (int)blockIdx.x * 128 + quarter * 32 + lane;   // value column
+        const uint32_t lo = (uint32_t)(quarter * 32) << 16;
         const bool live = d < p.dv, in_u = d < p.dvp;
         float* Sg = p.state + ((long long)b * p.H + h) * p.dk * (long long)p.dv + d;
         bool ok = true;
@@ -158,20 +161,17 @@ scan_kernel(const ScanArgs p, StatusWord* status) {
             const int t0 = p.t_begin + ch * kC, L = min(kC, p.n - t0);
             float* og = p.o + (((long long)b * p.n + t0) * p.H + h) * p.dv + d;
             const long long pitch = (long long)p.H * p.dv;
+            uint32_t v[32];
+            tmem_ld_32x32(tmem + lo + C::T_UO + 128u * (ch & 1) + 64u + half * 32u, v);
+            if (!live) return;
+            float* at = og + (long long)half * 32 * pitch;
+            if (L == kC) {
 #pragma unroll
-            for (int cb = 0; cb < 2; ++cb) {
-                uint32_t v[32];
-                tmem_ld_32x32(tmem + lo + C::T_UO + 128u * (ch & 1) + 64u + cb * 32u, v);
-                if (!live) continue;
-                float* at = og + (long long)cb * 32 * pitch;
-                if (L == kC) {
+                for (int i = 0; i < 32; ++i, at += pitch) __stcs(at, __uint_as_float(v[i]));
+            } else {
 #pragma unroll
-                    for (int i = 0; i < 32; ++i, at += pitch) __stcs(at, __uint_as_float(v[i]));
-                } else {
-#pragma unroll
-                    for (int i = 0; i < 32; ++i, at += pitch)
-                        if (cb * 32 + i < L) *at = __uint_as_float(v[i]);
-                }
+                for (int i = 0; i < 32; ++i, at += pitch)
+                    if (half * 32 + i < L) *at = __uint_as_float(v[i]);
             }
         };
         for (int ch = 0; ch < p.chunks && ok; ++ch) {
@@ -182,7 +182,7 @@ scan_kernel(const ScanArgs p, StatusWord* status) {
             tc_fence_after_sync();
             const float* dec = reinterpret_cast<const float*>(smem + C::OFF_DEC + s * 512);
 #pragma unroll 1
-            for (int cb = 0; cb < DK / 32; ++cb) {
+            for (int cb = half * KB; cb < (half + 1) * KB; ++cb) {
                 uint32_t v[32];
                 if (ch == 0) {
 #pragma unroll
@@ -210,36 +210,35 @@ scan_kernel(const ScanArgs p, StatusWord* status) {
             __syncwarp();
             if (lane == 0) mbar_arrive(s_ready);
             // while the first products run: U0 of this chunk, the finished output of the previous one
-            float u[kC];
+            float u[32];
             {
-                const float* U0 = reinterpret_cast<const float*>(ws0 + (long long)ch * p.ws_stride + W::OFF_U) + d;
+                const float* U0 = reinterpret_cast<const float*>(ws0 + (long long)ch * p.ws_stride + W::OFF_U) + (long long)half * 32 * p.dvp + (in_u ? d : 0);
 #pragma unroll
-                for (int t = 0; t < kC; ++t) u[t] = in_u ? __ldcs(U0 + (long long)t * p.dvp) : 0.f;
+                for (int t = 0; t < 32; ++t) u[t] = __ldcs(U0 + (long long)t * p.dvp);
             }
             if (ch > 0) store_o(ch - 1);
             if (HASW) {
                 ok = mbar_wait(uo_full, ch & 1, abort_flag, status, ST_TIMEOUT_ACCUM, 78);
                 if (!ok) break;
                 tc_fence_after_sync();
+                uint32_t v[32];
+                tmem_ld_32x32(tmem + lo + C::T_UO + 128u * s + half * 32u, v);
+#pragma unroll
+                for (int i = 0; i < 32; ++i) u[i] += __uint_as_float(v[i]);
+                // the other half's warp of these lanes has read its columns too before they are overwritten
+                tc_fence_before_sync();
+                __syncwarp();
+                if (lane == 0) mbar_arrive(u_read(quarter));
+                ok = mbar_wait(u_read(quarter), ch & 1, abort_flag, status, ST_TIMEOUT_ACCUM, 80);
+                if (!ok) break;
+                tc_fence_after_sync();
             }
+            // hi into columns 0..31, lo into 32..63 of the same region
+            uint32_t hh[16], ll[16];
 #pragma unroll
-            for (int cb = 0; cb < 2; ++cb) {
-                if (HASW) {
-                    uint32_t v[32];
-                    tmem_ld_32x32(tmem + lo + C::T_UO + 128u * s + cb * 32u, v);
-#pragma unroll
-                    for (int i = 0; i < 32; ++i) u[cb * 32 + i] += __uint_as_float(v[i]);
-                }
-            }
-            // both halves have been read: hi into columns 0..31, lo into 32..63 of the same region
-#pragma unroll
-            for (int cb = 0; cb < 2; ++cb) {
-                uint32_t hh[16], ll[16];
-#pragma unroll
-                for (int i = 0; i < 16; ++i) split2(u[cb * 32 + 2 * i], u[cb * 32 + 2 * i + 1], hh[i], ll[i]);
-                tmem_st_32x16(tmem + lo + C::T_UO + 128u * s + cb * 16u, hh);
-                tmem_st_32x16(tmem + lo + C::T_UO + 128u * s + 32u + cb * 16u, ll);
-            }
+            for (int i = 0; i < 16; ++i) split2(u[2 * i], u[2 * i + 1], hh[i], ll[i]);
+            tmem_st_32x16(tmem + lo + C::T_UO + 128u * s + half * 16u, hh);
+            tmem_st_32x16(tmem + lo + C::T_UO + 128u * s + 32u + half * 16u, ll);
             tmem_wait_st();
             tc_fence_before_sync();
             __syncwarp();
@@ -250,7 +249,7 @@ scan_kernel(const ScanArgs p, StatusWord* status) {
             tc_fence_after_sync();
             store_o(p.chunks - 1);
 #pragma unroll 1
-            for (int cb = 0; cb < DK / 32; ++cb) {
+            for (int cb = half * KB; cb < (half + 1) * KB; ++cb) {
                 uint32_t v[32];
                 tmem_ld_32x32(tmem + lo + C::T_S + cb * 32u, v);
 #pragma unroll
@@ -261,7 +260,7 @@ scan_kernel(const ScanArgs p, StatusWord* status) {
     }
     tc_fence_before_sync();
     __syncthreads();
-    if (warp == 4) { tc_fence_after_sync(); tmem_dealloc(tmem, 512); }
+    if (warp == 8) { tc_fence_after_sync(); tmem_dealloc(tmem, 512); }
 }
 
 template <int KB, bool HASW>
