@@ -832,6 +832,10 @@ def run_case(a):
     import synth
     torch.cuda.set_device(0)
     dev = torch.device("cuda", 0)
+    if a.case == "hybrid":
+        import bench_hybrid
+        bench_hybrid.case(torch, dev)
+        return
     if a.case in ("layer1", "layer8"):
         M = 1 if a.case == "layer1" else 8
         plz_native.lib().plz_set_smallm_overlap(1)

@@ -96,8 +96,8 @@ def models(torch, size, dev, pk):
             tq = timed(torch, lambda _: g.replay(), steps)
         except P.PlzError:          # its small-M launch has no form for this batch and width
             P.lib().plz_set_smallm_overlap(0)
-            tq = float("nan")
-        out["decode"][f"B{B}_T{T}"] = {"gopunex_ms": tg, "gopunex_tok_s": B / tg * 1e3, "palettized_qwen_ms": tq, "palettized_qwen_tok_s": B / tq * 1e3,
+            tq = None
+        out["decode"][f"B{B}_T{T}"] = {"gopunex_ms": tg, "gopunex_tok_s": B / tg * 1e3, "palettized_qwen_ms": tq, "palettized_qwen_tok_s": B / tq * 1e3 if tq else None,
                                        "gopunex_weight_and_state_bytes": gop.weight_bytes() + cg.nbytes() + sum(st["S"].numel() * 4 for st in cg.layers if "S" in st)}
         del cg, cq, g
     return out
@@ -218,6 +218,18 @@ def kernels(torch, size, dev, pk):
         add("recurrent<decay>", f"decode B{B}", t, sb, like="attn_decode")
         del sts
     return rows
+
+
+def case(torch, dev):
+    """One launch of every kernel of the design on a small case (width 1024, 2048 tokens, then three single tokens): for ncu."""
+    from hybrid_model import Gopunex
+    m = Gopunex.random(gopunex_config(*SIZES["small"][:5], 3), dev, seed=1)
+    c = m.new_cache(1, 2048 + 8)
+    m.prefill(torch.randint(0, VOCAB, (1, 2048), device=dev), c)
+    m.use_graph = False
+    for _ in range(3):
+        m.decode_step(torch.zeros(1, dtype=torch.int64, device=dev), c)
+    torch.cuda.synchronize()
 
 
 def run(args, pk, sampler_cls):
