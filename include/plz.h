@@ -404,11 +404,18 @@ int32_t plz_bwd_dw_hard_lora(const plz_weight_t* w, const void* x, int64_t ldx, 
  * residual stream are fp32 in both. Rows are b * n + t: B sequences advance in lockstep by n tokens; pos is ONE int32 in device
  * memory, the position of the first of the n tokens, so that a captured step can be replayed at later positions.
  *
- * plz_seq_linear: y = act(x W^T + bias), W [N, K] row-major, act 0 none / 1 square of relu; y_f32: write fp32 from bf16 operands.
+ * plz_seq_linear: y = act(x W^T + bias), W [N, K] row-major, act 0 none / 1 square of relu / 2 gated: rows 2 i and 2 i + 1 of W are a
+ *   gate / up pair and y [M, N / 2] = gelu_tanh(gate) * up; y_f32: write fp32 from bf16 operands.
  *   Any shape; 16-byte aligned rows take the streaming (M <= 8) and tcgen05 (bf16) kernels.
- * plz_seq_embed: x fp32 [rows, W] = table[ids] * scale, xb (may be NULL) the same in dtype; an id outside [0, vocab) gives zeros and
- *   sets *bad (may be NULL).
- * plz_seq_residual_norm: x += mult * y / sqrt(mean(y^2) + eps) * (w + w_offset); xb (may be NULL) = x in dtype. w fp32 [W].
+ * plz_head_linear: y[m, h, :] = x[m, h, :] W_h^T for every head, W [H, N, K] row-major; x and y rows ldx / ldy apart, heads xh / yh apart;
+ *   gate (may be NULL) [M, H * N]: y *= sigmoid(gate).
+ * plz_seq_embed: x fp32 [rows, W] = table[ids] * scale, with norm_w (fp32 [W], may be NULL) then divided by its root mean square and times
+ *   norm_w + norm_offset; x2 (fp32, may be NULL) and xb (dtype, may be NULL) the same; an id outside [0, vocab) gives zeros and sets
+ *   *bad (may be NULL).
+ * plz_seq_stream: what happens to the residual stream x (fp32 [rows, W]) between two sublayers, any part may be absent:
+ *   x += mult * y / sqrt(mean(y^2) + eps) * (w + w_offset)   (y, the sublayer's output; w fp32 [W])
+ *   x += add_rows + add_vec                                  (fp32 [rows, W], fp32 [W])
+ *   out = x, with w_next x / sqrt(mean(x^2) + eps) * (w_next + w_offset)   (dtype; the operand of the next sublayer)
  * plz_seq_rows_norm: out[i] = x[idx[i]] / rms * (w + w_offset) in dtype (idx NULL: row i).
  * plz_seq_norm_gate: out = o / rms(o over each group of L values) * w[c] * sigmoid(gate), o fp32 [rows, groups * L], w fp32 [L].
  * plz_delta_prep: causal convolution + silu on the q, k, v slices of a projection, unit norm of q and k per head (q times q_scale),
@@ -419,14 +426,31 @@ int32_t plz_bwd_dw_hard_lora(const plz_weight_t* w, const void* x, int64_t ldx, 
  *   write of keys and values into the cache at *pos + t.
  * plz_attn_bias: causal attention of the n new tokens against the cache (which already holds them), score * scale + bias by distance
  *   (bias points at distance 0 of head 0; entry n_bias - 1 holds for everything farther; rows ldb apart, readable from 256 entries
- *   before distance 0 to 256 entries past n_bias - 1), optional sink in the denominator. host_pos = *pos when the caller knows it, or
+ *   before distance 0 to 256 entries past n_bias - 1), optional sink in the denominator (score sinks[h], or 0 when sinks is NULL).
+ *   The last dk2 of the dk query / key columns may come from a second key tensor that all heads share; the output may be multiplied by
+ *   sigmoid(gate). host_pos = *pos when the caller knows it, or
  *   -1 (n == 1 only). ws: plz_attn_bias_ws_bytes bytes for n == 1, else unused. */
 int32_t plz_seq_linear(int32_t dtype, const void* x, int64_t ldx, int32_t M, int32_t K, const void* w, int64_t ldw, int32_t N, const void* bias,
                        int32_t act, void* y, int64_t ldy, int32_t y_f32, void* stream);
 int32_t plz_seq_embed(int32_t dtype, const void* table, int64_t ldt, const int64_t* ids, int64_t rows, int32_t W, int64_t vocab, float scale,
-                      float* x, void* xb, int32_t* bad, void* stream);
-int32_t plz_seq_residual_norm(int32_t dtype, const void* y, int64_t ldy, const float* w, float w_offset, float mult, float eps, int64_t rows,
-                              int32_t W, float* x, void* xb, void* stream);
+                      const float* norm_w, float norm_offset, float eps, float* x, float* x2, void* xb, int32_t* bad, void* stream);
+typedef struct plz_head_linear {
+    const void* x; int64_t ldx, xh;
+    const void* w;
+    void* y; int64_t ldy, yh;
+    const void* gate; int64_t ldg;
+    int32_t M, H, N, K;
+} plz_head_linear_t;
+int32_t plz_head_linear(int32_t dtype, const plz_head_linear_t* args, void* stream);
+typedef struct plz_stream {
+    const void* y; int64_t ldy; const float* w;
+    float w_offset, mult, eps;
+    int64_t rows; int32_t W;
+    float* x;
+    const float* add_rows; const float* add_vec; const float* w_next;
+    void* out;
+} plz_stream_t;
+int32_t plz_seq_stream(int32_t dtype, const plz_stream_t* args, void* stream);
 int32_t plz_seq_rows_norm(int32_t dtype, const float* x, const int64_t* idx, const float* w, float w_offset, float eps, int64_t rows, int32_t W,
                           void* out, void* stream);
 int32_t plz_seq_norm_gate(int32_t dtype, const float* o, const void* gate, int64_t ldg, const float* w, float eps, int64_t rows, int32_t groups,
@@ -481,9 +505,49 @@ typedef struct plz_attn_bias {
     const int32_t* pos; int32_t host_pos, cap;
     int32_t B, n, H, G, dk, dv, sink;
     float scale;
+    const float* sinks;                                        /* [H] or NULL */
+    int64_t k_tok, v_tok;                                      /* elements between positions of k, v; 0: G * (dk - dk2), G * dv */
+    const void* k2; int64_t k2_batch; int32_t dk2;             /* [B, cap, dk2] */
+    const void* gate; int64_t ldg;                             /* [B * n, H * dv] or NULL */
 } plz_attn_bias_t;
 int64_t plz_attn_bias_ws_bytes(int32_t B, int32_t H, int32_t G, int32_t dv, int32_t cap);
 int32_t plz_attn_bias(int32_t dtype, const plz_attn_bias_t* args, void* ws, int64_t ws_bytes, void* stream);
+/* Attention over cached latents. A token leaves in the cache its latent c [R] and one key part kr [dr] that carries the position and is
+ * shared by all heads; keys and values of a head are products of c.
+ * plz_latent_prep: from one projection row: cq = rms_norm(q slice) * wq, c = rms_norm(c slice) * wc into the cache at *pos + t, kr = its
+ *   slice rotated, into the cache.
+ * plz_rotate: out[row, h, :] = x[row, h, :] with pairs (2 i, 2 i + 1), i < pairs, turned by (*pos + t) * freq[i] and scaled by m (freq in
+ *   double precision, the angle reduced before it is rounded); the other columns are copied. In place if out = x.
+ * plz_latent_attn: scores of queries that already are products with the key matrix (q [rows, H, R + dr]) against c and kr, softmax with
+ *   optional sinks [H], and the weighted sum of the latents, o [rows, H * R]. ws: plz_latent_attn_ws_bytes bytes. */
+typedef struct plz_latent_prep {
+    const void* proj; int64_t ldp; int32_t off_q, off_c, off_r;
+    const float* wq; const float* wc;
+    void* cq;                                                  /* [rows, q_rank] */
+    void* c; void* kr; int64_t c_batch, r_batch;               /* caches [B, cap, R], [B, cap, dr] */
+    const int32_t* pos; const double* freq; int32_t pairs; float m;
+    int32_t B, n, q_rank, R, dr, cap;
+    float eps;
+} plz_latent_prep_t;
+int32_t plz_latent_prep(int32_t dtype, const plz_latent_prep_t* args, void* stream);
+typedef struct plz_rotate {
+    const void* x; int64_t ldx, xh;                            /* rows and heads apart */
+    void* out; int64_t ldo, oh;
+    const int32_t* pos; const double* freq; int32_t pairs; float m;
+    int32_t B, n, H, dr;
+} plz_rotate_t;
+int32_t plz_rotate(int32_t dtype, const plz_rotate_t* args, void* stream);
+typedef struct plz_latent_attn {
+    const void* q; int64_t ldq;
+    const void* c; const void* kr; int64_t c_batch, r_batch;
+    void* o; int64_t ldo;
+    const float* sinks;
+    const int32_t* pos; int32_t host_pos, cap;
+    int32_t B, n, H, R, dr;
+    float scale;
+} plz_latent_attn_t;
+int64_t plz_latent_attn_ws_bytes(int32_t dtype, int32_t B, int32_t n, int32_t H, int32_t R, int32_t dr, int32_t cap);
+int32_t plz_latent_attn(int32_t dtype, const plz_latent_attn_t* args, void* ws, int64_t ws_bytes, void* stream);
 /* *pos += n, at the end of a step */
 int32_t plz_advance(int32_t* pos, int32_t n, void* stream);
 /* Next token of every row of fp32 logits [rows, V]: temperature 0: the largest (first of equals); else a draw from

@@ -10,9 +10,10 @@ import sys
 HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
 SOURCES = ["api.cu", "lut_gemm.cu", "lut_gemm_pair.cu", "tn_gemm.cu", "elementwise.cu", "gemv.cu", "smallm_mma.cu", "train_ops.cu", "soft_tensors.cu", "attention.cu", "attention_decode.cu", "layer_ops.cu",
-           "seq_linear.cu", "seq_ops.cu", "seq_recurrent.cu", "seq_chunk.cu", "seq_scan.cu", "attention_bias.cu", "attention_bias_tc.cu"]
-PRECISE = {"seq_linear.cu", "seq_ops.cu", "seq_recurrent.cu", "seq_chunk.cu", "seq_scan.cu", "attention_bias.cu"}   # compiled without --use_fast_math
-HEADERS = ["plz_sm100.cuh", "plz_host.h", "plz_launch.h", "soft_math.cuh", "seq_math.cuh", "seq_chunk.cuh", "attention_tiles.cuh", os.path.join("..", "..", "include", "plz.h")]
+           "seq_linear.cu", "seq_ops.cu", "seq_recurrent.cu", "seq_chunk.cu", "seq_scan.cu", "attention_bias.cu", "attention_bias_tc.cu",
+           "latent_ops.cu", "latent_attention.cu", "latent_attention_tc.cu"]
+PRECISE = {"seq_linear.cu", "seq_ops.cu", "seq_recurrent.cu", "seq_chunk.cu", "seq_scan.cu", "attention_bias.cu", "latent_ops.cu", "latent_attention.cu"}   # compiled without --use_fast_math
+HEADERS = ["plz_sm100.cuh", "plz_host.h", "plz_launch.h", "soft_math.cuh", "seq_math.cuh", "seq_chunk.cuh", "latent_attention.cuh", "attention_tiles.cuh", os.path.join("..", "..", "include", "plz.h")]
 LIB = os.path.join(HERE, "libplz.so")
 NVCC = os.environ.get("NVCC", "/usr/local/cuda/bin/nvcc")
 FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",

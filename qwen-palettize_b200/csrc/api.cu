@@ -83,16 +83,17 @@ int make_tmap_bf16(CUtensorMap* map, const void* base, uint64_t rows, uint64_t c
 }
 
 int make_tmap_bf16_heads(CUtensorMap* map, const void* base, uint64_t dim, uint64_t heads, uint64_t tokens, uint64_t batch, uint64_t tok_pitch,
-                         uint64_t batch_pitch, uint32_t box_tokens) {
+                         uint64_t batch_pitch, uint32_t box_tokens, uint64_t head_pitch) {
+    if (head_pitch == 0) head_pitch = dim;
     EncodeTiledFn enc = get_encode_fn();
     static thread_local int bound_dev = -1;
     int dev = -1;
     if (cudaGetDevice(&dev) == cudaSuccess && dev != bound_dev) { cudaSetDevice(dev); bound_dev = dev; }   // see make_tmap_bf16
     if (!enc) { set_last_error("cuTensorMapEncodeTiled is not available from the driver"); return PLZ_ERR_CUDA; }
     if (!base) { set_last_error("null tensor pointer"); return PLZ_ERR_NULL; }
-    if (((uintptr_t)base & 15) || dim % 8 || tok_pitch % 8 || batch_pitch % 8) { set_last_error("bf16 head tensor: base and pitches must be multiples of 16 bytes"); return PLZ_ERR_BAD_ALIGN; }
+    if (((uintptr_t)base & 15) || dim % 8 || head_pitch % 8 || tok_pitch % 8 || batch_pitch % 8) { set_last_error("bf16 head tensor: base and pitches must be multiples of 16 bytes"); return PLZ_ERR_BAD_ALIGN; }
     cuuint64_t dims[4] = {dim, heads, tokens, batch};
-    cuuint64_t strides[3] = {dim * 2, tok_pitch * 2, batch_pitch * 2};
+    cuuint64_t strides[3] = {head_pitch * 2, tok_pitch * 2, batch_pitch * 2};
     cuuint32_t box[4] = {64, 1, box_tokens, 1};
     cuuint32_t estr[4] = {1, 1, 1, 1};
     CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
@@ -966,26 +967,36 @@ int32_t plz_seq_linear(int32_t dtype, const void* x, int64_t ldx, int32_t M, int
                        int32_t act, void* y, int64_t ldy, int32_t y_f32, void* stream) {
     int rc = check_dtype(dtype);
     if (rc) return rc;
-    if (M < 0 || ldx < K || ldw < K || ldy < N) { set_last_error("seq_linear: bad shape M=%d N=%d K=%d", M, N, K); return PLZ_ERR_BAD_SHAPE; }
+    if (M < 0 || ldx < K || ldw < K || ldy < (act == 2 ? N / 2 : N)) { set_last_error("seq_linear: bad shape M=%d N=%d K=%d", M, N, K); return PLZ_ERR_BAD_SHAPE; }
     return launch_seq_linear(dtype, x, ldx, M, K, w, ldw, N, bias, act, y, ldy, y_f32, (cudaStream_t)stream);
 }
 
 int32_t plz_seq_embed(int32_t dtype, const void* table, int64_t ldt, const int64_t* ids, int64_t rows, int32_t W, int64_t vocab, float scale,
-                      float* x, void* xb, int32_t* bad, void* stream) {
+                      const float* norm_w, float norm_offset, float eps, float* x, float* x2, void* xb, int32_t* bad, void* stream) {
     int rc = check_dtype(dtype);
     if (rc || (rc = check_rows(rows))) return rc;
     if (W <= 0 || vocab <= 0 || ldt < W) { set_last_error("seq_embed: bad shape"); return PLZ_ERR_BAD_SHAPE; }
     if (rows && (!table || !ids || !x)) { set_last_error("null pointer"); return PLZ_ERR_NULL; }
-    return launch_seq_embed(dtype, table, ldt, (const long long*)ids, rows, W, vocab, scale, x, xb, bad, (cudaStream_t)stream);
+    return launch_seq_embed(dtype, table, ldt, (const long long*)ids, rows, W, vocab, scale, norm_w, norm_offset, eps, x, x2, xb, bad, (cudaStream_t)stream);
 }
 
-int32_t plz_seq_residual_norm(int32_t dtype, const void* y, int64_t ldy, const float* w, float w_offset, float mult, float eps, int64_t rows,
-                              int32_t W, float* x, void* xb, void* stream) {
+int32_t plz_head_linear(int32_t dtype, const plz_head_linear_t* a, void* stream) {
     int rc = check_dtype(dtype);
-    if (rc || (rc = check_rows(rows))) return rc;
-    if (W <= 0 || ldy < W) { set_last_error("seq_residual_norm: bad shape"); return PLZ_ERR_BAD_SHAPE; }
-    if (rows && (!y || !w || !x)) { set_last_error("null pointer"); return PLZ_ERR_NULL; }
-    return launch_seq_residual_norm(dtype, y, ldy, w, w_offset, mult, eps, rows, W, x, xb, (cudaStream_t)stream);
+    if (rc) return rc;
+    if (!a || (a->M > 0 && (!a->x || !a->w || !a->y))) { set_last_error("null pointer"); return PLZ_ERR_NULL; }
+    if (a->M < 0 || a->H <= 0 || a->H > 65535 || a->N <= 0 || a->K <= 0 || a->ldx < 0 || a->xh < a->K || a->yh < a->N || a->ldy < 0 ||
+        (a->gate && a->ldg < (int64_t)a->H * a->N)) {
+        set_last_error("head_linear: bad shape M=%d H=%d N=%d K=%d", a->M, a->H, a->N, a->K); return PLZ_ERR_BAD_SHAPE;
+    }
+    return launch_head_linear(dtype, *a, (cudaStream_t)stream);
+}
+
+int32_t plz_seq_stream(int32_t dtype, const plz_stream_t* a, void* stream) {
+    int rc = check_dtype(dtype);
+    if (rc) return rc;
+    if (!a || (a->rows && !a->x) || (a->y && !a->w) || (a->w_next && !a->out)) { set_last_error("null pointer"); return PLZ_ERR_NULL; }
+    if (a->W <= 0 || (a->y && a->ldy < a->W) || (rc = check_rows(a->rows))) { set_last_error("seq_stream: bad shape"); return PLZ_ERR_BAD_SHAPE; }
+    return launch_seq_stream(dtype, *a, (cudaStream_t)stream);
 }
 
 int32_t plz_seq_rows_norm(int32_t dtype, const float* x, const int64_t* idx, const float* w, float w_offset, float eps, int64_t rows, int32_t W,
@@ -1071,13 +1082,61 @@ int32_t plz_attn_bias(int32_t dtype, const plz_attn_bias_t* a, void* ws, int64_t
     }
     if (a->B == 0 || a->n == 0) return PLZ_OK;
     cudaStream_t s = (cudaStream_t)stream;
+    if (a->k2 ? (a->dk2 <= 0 || a->dk2 > a->dk) : a->dk2 != 0) { set_last_error("attn_bias: second key part of %d columns", a->dk2); return PLZ_ERR_BAD_SHAPE; }
+    plz_attn_bias_t f = *a;
+    const int dk1 = a->dk - a->dk2;
+    if (!f.k_tok) f.k_tok = (int64_t)a->G * dk1;
+    if (!f.v_tok) f.v_tok = (int64_t)a->G * a->dv;
     const int per16 = dtype == 0 ? 8 : 4;
-    const bool vec = a->dk % 8 == 0 && a->dv % 8 == 0 && a->ldq % per16 == 0 && a->k_batch % per16 == 0 && a->v_batch % per16 == 0 &&
-                     !((uintptr_t)a->q & 15) && !((uintptr_t)a->k & 15) && !((uintptr_t)a->v & 15);
-    if (a->n == 1 && vec && a->dk <= 256 && a->dv <= 256) return launch_attn_bias_decode(dtype, *a, a->cap, ws, ws ? ws_bytes : 0, s);
-    if (dtype == 0 && vec && a->n > 1 && a->dk <= 128 && a->dv <= 128 && a->scale > 0.f && (!a->bias || a->bias_top) && a->ldo % 8 == 0 && !((uintptr_t)a->o & 15))
-        return launch_attn_bias_tc(*a, s);
-    return launch_attn_bias_simt(dtype, *a, s);
+    const bool vec = dk1 % 8 == 0 && a->dk2 % 8 == 0 && a->dv % 8 == 0 && a->ldq % per16 == 0 && a->k_batch % per16 == 0 && a->v_batch % per16 == 0 && a->k2_batch % per16 == 0 &&
+                     f.k_tok % per16 == 0 && f.v_tok % per16 == 0 && !((uintptr_t)a->q & 15) && !((uintptr_t)a->k & 15) && !((uintptr_t)a->v & 15) && !((uintptr_t)a->k2 & 15);
+    const bool plain = !a->k2 && !a->sinks && !a->gate && f.k_tok == (int64_t)a->G * a->dk && f.v_tok == (int64_t)a->G * a->dv;
+    if (a->n == 1 && vec && plain && a->dk <= 256 && a->dv <= 256) return launch_attn_bias_decode(dtype, f, a->cap, ws, ws ? ws_bytes : 0, s);
+    if (dtype == 0 && vec && plain && a->n > 1 && dk1 > 0 && (dk1 + 63) / 64 + (a->dk2 + 63) / 64 <= 2 && a->dv <= 128 && a->scale > 0.f && (!a->bias || a->bias_top) &&
+        a->ldo % 8 == 0 && !((uintptr_t)a->o & 15) && (!a->gate || (a->ldg % 8 == 0 && !((uintptr_t)a->gate & 15))))
+        return launch_attn_bias_tc(f, s);
+    return launch_attn_bias_simt(dtype, f, s);
+}
+
+static int check_rotation(const int32_t* pos, const double* freq, int32_t pairs, int32_t dr) {
+    if (!pos || (pairs && !freq)) { set_last_error("null pointer"); return PLZ_ERR_NULL; }
+    if (pairs < 0 || 2 * pairs > dr) { set_last_error("rotation of %d pairs in %d columns", pairs, dr); return PLZ_ERR_BAD_SHAPE; }
+    return PLZ_OK;
+}
+
+int32_t plz_latent_prep(int32_t dtype, const plz_latent_prep_t* a, void* stream) {
+    int rc = check_dtype(dtype);
+    if (rc) return rc;
+    if (!a || !a->proj || !a->wq || !a->wc || !a->cq || !a->c || (a->dr && !a->kr)) { set_last_error("null pointer"); return PLZ_ERR_NULL; }
+    if (a->B < 0 || a->n < 0 || a->q_rank <= 0 || a->R <= 0 || a->dr < 0 || (rc = check_rows((int64_t)a->B * a->n))) { set_last_error("latent_prep: bad shape"); return PLZ_ERR_BAD_SHAPE; }
+    if ((rc = check_rotation(a->pos, a->freq, a->pairs, a->dr))) return rc;
+    return launch_latent_prep(dtype, *a, (cudaStream_t)stream);
+}
+
+int32_t plz_rotate(int32_t dtype, const plz_rotate_t* a, void* stream) {
+    int rc = check_dtype(dtype);
+    if (rc) return rc;
+    if (!a || !a->x || !a->out) { set_last_error("null pointer"); return PLZ_ERR_NULL; }
+    if (a->B < 0 || a->n < 0 || a->H <= 0 || a->dr <= 0 || (rc = check_rows((int64_t)a->B * a->n))) { set_last_error("rotate: bad shape"); return PLZ_ERR_BAD_SHAPE; }
+    if ((rc = check_rotation(a->pos, a->freq, a->pairs, a->dr))) return rc;
+    return launch_rotate(dtype, *a, (cudaStream_t)stream);
+}
+
+int64_t plz_latent_attn_ws_bytes(int32_t dtype, int32_t B, int32_t n, int32_t H, int32_t R, int32_t dr, int32_t cap) {
+    if (B <= 0 || n <= 0 || H <= 0 || R <= 0 || cap <= 0) return 0;
+    return latent_attn_ws_bytes(dtype, B, n, H, R, dr, cap);
+}
+
+int32_t plz_latent_attn(int32_t dtype, const plz_latent_attn_t* a, void* ws, int64_t ws_bytes, void* stream) {
+    int rc = check_dtype(dtype);
+    if (rc) return rc;
+    if (!a || !a->q || !a->c || (a->dr && !a->kr) || !a->o || !a->pos) { set_last_error("null pointer"); return PLZ_ERR_NULL; }
+    if (a->B < 0 || a->n < 0 || a->H <= 0 || a->R <= 0 || a->dr < 0 || a->B > 65535 || a->ldq < (int64_t)a->H * (a->R + a->dr) || a->ldo < (int64_t)a->H * a->R ||
+        (a->n > 1 && a->host_pos < 0) || a->host_pos + (int64_t)a->n > a->cap || (int64_t)a->n * a->H > 0x7FFFFFFF) {
+        set_last_error("latent_attn: bad shape H=%d R=%d dr=%d n=%d pos=%d cap=%d", a->H, a->R, a->dr, a->n, a->host_pos, a->cap); return PLZ_ERR_BAD_SHAPE;
+    }
+    if (a->B == 0 || a->n == 0) return PLZ_OK;
+    return launch_latent_attn(dtype, *a, ws, ws ? ws_bytes : 0, (cudaStream_t)stream);
 }
 
 int32_t plz_advance(int32_t* pos, int32_t n, void* stream) {

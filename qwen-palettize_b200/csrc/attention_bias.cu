@@ -1,6 +1,7 @@
 // Causal attention with a per-head bias by distance and a sink, against the key / value cache, on the CUDA cores: fp32 products
 // and softmax for both types and any head sizes. It is the 32-bit mode, and serves bf16 head sizes outside the tensor-core kernel's
-// range.  score(i, j) = q_i . k_j * scale + bias[h][i - j];  with the sink, the denominator starts at exp(0).
+// range.  score(i, j) = q_i . k_j * scale + bias[h][i - j];  with a sink, the denominator starts at exp(its score).  The last key
+// columns may come from a second tensor shared by all heads; the output may be multiplied by sigmoid(gate).
 //
 // Block = 32 queries of one head, 128 threads: thread = (query, one of four key slices). Keys and values pass through shared memory
 // 32 at a time.
@@ -19,6 +20,10 @@ struct BiasParams {
     const int* pos;
     int n, H, G, dk, dv, sink;
     float scale;
+    const float* sinks;
+    long long k_tok, v_tok;
+    const void* k2; long long k2_batch; int dk2;               // [B, T, dk2]
+    const void* gate; long long ldg;
 };
 
 template <typename T, int DVT>   // DVT: value columns per thread (dv <= 4 * DVT)
@@ -43,7 +48,8 @@ attn_bias_kernel(const BiasParams p) {
     }
     const int i = pos + q0 + qi;                                   // absolute position of this thread's query
     const int last = pos + min(p.n, q0 + kQ) - 1;                  // largest key any query of the block sees
-    float m = p.sink ? 0.f : -INFINITY, l = p.sink ? 1.f : 0.f;
+    const int dk1 = p.dk - p.dk2;
+    float m = p.sink ? (p.sinks ? p.sinks[h] : 0.f) : -INFINITY, l = p.sink ? 1.f : 0.f;
     float acc[DVT];
 #pragma unroll
     for (int d = 0; d < DVT; ++d) acc[d] = 0.f;
@@ -52,11 +58,15 @@ attn_bias_kernel(const BiasParams p) {
         __syncthreads();
         for (int e = tid; e < kK * p.dk; e += 128) {
             const int r = e / p.dk, c = e - r * p.dk;
-            sK[r * pk + c] = j0 + r <= last ? to_f(((const T*)p.k)[b * p.k_batch + ((long long)(j0 + r) * p.G + hk) * p.dk + c]) : 0.f;
+            float v = 0.f;
+            if (j0 + r <= last)
+                v = to_f(c < dk1 ? ((const T*)p.k)[b * p.k_batch + (j0 + r) * p.k_tok + hk * dk1 + c]
+                                 : ((const T*)p.k2)[b * p.k2_batch + (long long)(j0 + r) * p.dk2 + c - dk1]);
+            sK[r * pk + c] = v;
         }
         for (int e = tid; e < kK * p.dv; e += 128) {
             const int r = e / p.dv, c = e - r * p.dv;
-            sV[e] = j0 + r <= last ? to_f(((const T*)p.v)[b * p.v_batch + ((long long)(j0 + r) * p.G + hk) * p.dv + c]) : 0.f;
+            sV[e] = j0 + r <= last ? to_f(((const T*)p.v)[b * p.v_batch + (j0 + r) * p.v_tok + hk * p.dv + c]) : 0.f;
         }
         __syncthreads();
         float s[8];
@@ -104,10 +114,11 @@ attn_bias_kernel(const BiasParams p) {
     if (q0 + qi < p.n) {
         const float inv = l > 0.f ? 1.0f / l : 0.f;
         T* dst = (T*)p.o + (b * p.n + q0 + qi) * p.ldo + (long long)h * p.dv;
+        const T* gate = p.gate ? (const T*)p.gate + (b * p.n + q0 + qi) * p.ldg + (long long)h * p.dv : nullptr;
 #pragma unroll
         for (int d = 0; d < DVT; ++d) {
             const int c = sl + 4 * d;
-            if (c < p.dv) dst[c] = from_f<T>(acc[d] * inv);
+            if (c < p.dv) dst[c] = from_f<T>(acc[d] * inv * (gate ? sigmoid_f(to_f(gate[c])) : 1.f));
         }
     }
 }
@@ -137,7 +148,8 @@ int launch_attn_bias_simt(int dtype, const AttnBiasArgs& a, cudaStream_t stream)
     BiasParams p = {};
     p.q = a.q; p.ldq = a.ldq; p.k = a.k; p.v = a.v; p.k_batch = a.k_batch; p.v_batch = a.v_batch; p.o = a.o; p.ldo = a.ldo;
     p.bias = a.bias; p.ldb = a.ldb; p.n_bias = a.n_bias; p.pos = a.pos;
-    p.n = a.n; p.H = a.H; p.G = a.G; p.dk = a.dk; p.dv = a.dv; p.sink = a.sink; p.scale = a.scale;
+    p.n = a.n; p.H = a.H; p.G = a.G; p.dk = a.dk; p.dv = a.dv; p.sink = a.sink || a.sinks; p.scale = a.scale;
+    p.sinks = a.sinks; p.k_tok = a.k_tok; p.v_tok = a.v_tok; p.k2 = a.k2; p.k2_batch = a.k2_batch; p.dk2 = a.dk2; p.gate = a.gate; p.ldg = a.ldg;
     return dtype == 1 ? launch_any<float>(p, a.B, stream) : launch_any<__nv_bfloat16>(p, a.B, stream);
 }
 

@@ -78,6 +78,11 @@ struct Cfg {
     static constexpr uint32_t SMEM_BYTES = BAR_OFF + 1024 /*align*/ + 256 /*barriers*/;
 };
 
+// tanh form of gelu, z * sigmoid(2 sqrt(2 / pi) (z + 0.044715 z^3)), in the one place where its speed matters
+__device__ __forceinline__ float gelu_tanh_fast(float z) {
+    return __fdividef(z, 1.0f + exp2f(fminf(-2.302208198f * fmaf(0.044715f * z * z, z, z), 80.0f)));
+}
+
 template <int MT, int BMODE, bool NARROW, int FUSE>
 __global__ void __launch_bounds__(kThreads, 1)
 lut_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB,
@@ -447,6 +452,40 @@ lut_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__
                     if (m < p.M) rs = __ldg(p.row_scale + m);
                 }
                 const float scale = p.alpha * rs;
+                if (FUSE == 4) {
+                    // columns 2 i, 2 i + 1 are a gate / up pair: the warp's 128 accumulator columns make one box of 64 outputs
+                    if (lane == 0) tma_store_wait_read();
+                    __syncwarp();
+#pragma unroll 1
+                    for (int c = 0; c < 4; ++c) {
+                        uint32_t v[32];
+                        tmem_ld_32x32(tmem_base + ((uint32_t)(lane_group * 32) << 16) + mt * 256u + col_half * 128 + c * 32, v);
+                        if (mt == nmt - 1 && c == 3) {
+                            tc_fence_before_sync();
+                            __syncwarp();
+                            if (lane == 0) mbar_arrive(tmem_empty);
+                        }
+#pragma unroll
+                        for (int g = 0; g < 2; ++g) {
+                            uint32_t o[4];
+#pragma unroll
+                            for (int i = 0; i < 4; ++i) {
+                                const float z0 = __uint_as_float(v[g * 16 + 4 * i]), z1 = __uint_as_float(v[g * 16 + 4 * i + 2]);
+                                o[i] = pack_bf16x2(gelu_tanh_fast(z0) * __uint_as_float(v[g * 16 + 4 * i + 1]),
+                                                   gelu_tanh_fast(z1) * __uint_as_float(v[g * 16 + 4 * i + 3]));
+                            }
+                            *reinterpret_cast<uint4*>(stage + swz128(lane, c * 2 + g)) = make_uint4(o[0], o[1], o[2], o[3]);
+                        }
+                    }
+                    fence_proxy_async_smem();
+                    __syncwarp();
+                    const int jo = (j0 + col_half * 128) >> 1;
+                    if (lane == 0 && jo < p.J && m0 + mt * 128 + lane_group * 32 < p.M) {
+                        tma_store_2d(&tmD, stage_u32, jo, m0 + mt * 128 + lane_group * 32);
+                        tma_store_commit();
+                    }
+                    continue;
+                }
 #pragma unroll 1
                 for (int b = 0; b < 2; ++b) {
                     const int col = col_half * 128 + b * 64;
@@ -564,7 +603,7 @@ static int launch_t(const LutGemmArgs& a, cudaStream_t stream) {
             if ((rc = make_tmap_bf16(&tmB2, a.B2, a.J, a.r2, a.ldb2, 64, 256))) return rc;
         }
     }
-    const int out_cols = (FUSE == 1) ? a.J / 2 : a.J;  // the SwiGLU form writes one column per gate/up pair
+    const int out_cols = (FUSE == 1 || FUSE == 4) ? a.J / 2 : a.J;  // the gated forms write one column per gate/up pair
     if ((rc = make_tmap_bf16(&tmD, a.out, a.M, out_cols, a.ld_out, 64, 32))) return rc;
     LutGemmParams p;
     p.M = a.M; p.J = out_cols; p.R = a.R; p.n_extra = a.r2 > 0 ? 1 : 0;
@@ -641,6 +680,7 @@ int launch_lut_gemm(const LutGemmArgs& a, cudaStream_t stream) {
                 if (narrow) return launch_t<1, B_TMA_K, true, 3>(a, stream);
                 return big ? launch_t<2, B_TMA_K, false, 3>(a, stream) : launch_t<1, B_TMA_K, false, 3>(a, stream);
             }
+            if (a.fuse == 4) return big ? launch_t<2, B_TMA_K, false, 4>(a, stream) : launch_t<1, B_TMA_K, false, 4>(a, stream);
             if (narrow) return launch_t<1, B_TMA_K, true>(a, stream);
             return big ? launch_t<2, B_TMA_K, false>(a, stream) : launch_t<1, B_TMA_K, false>(a, stream);
         case B_TMA_MN:

@@ -26,9 +26,9 @@ int make_tmap_bf16(CUtensorMap* map, const void* base, uint64_t rows, uint64_t c
                    uint32_t box_cols, uint32_t box_rows);
 
 // bf16 [batch, tokens, heads, dim] with the given pitches (elements): boxes of 64 dim columns x 1 head x box_tokens, 128-byte swizzle,
-// out-of-range elements read as zero and are not written. dim may be any multiple of 8.
+// out-of-range elements read as zero and are not written. dim may be any multiple of 8. head_pitch 0: heads are dim apart.
 int make_tmap_bf16_heads(CUtensorMap* map, const void* base, uint64_t dim, uint64_t heads, uint64_t tokens, uint64_t batch, uint64_t tok_pitch,
-                         uint64_t batch_pitch, uint32_t box_tokens);
+                         uint64_t batch_pitch, uint32_t box_tokens, uint64_t head_pitch = 0);
 
 #define PLZ_CUDA_CHECK(expr)                                                            \
     do {                                                                                \

@@ -20,6 +20,7 @@ struct LutGemmArgs {
     int r2; const void* A2; long long lda2; const void* B2; long long ldb2;
     void* out; long long ld_out; float alpha;
     // fused MLP front end (forward decode mode only): fuse 1 = gate/up pair + SwiGLU (J = 2 N), 2 = one matrix;
+    // fuse 4 (dense B): columns 2 i, 2 i + 1 are a gate / up pair, out[:, i] = gelu_tanh(gate) * up;
     // col_scale bf16 [K] and row_scale fp32 [M] are the RMSNorm factors (either may be null)
     int fuse; const void* packed2; const void* palette2; const void* col_scale; const float* row_scale;
     void* gate_out; void* up_out; long long ld_gu;  // fuse == 1: optional bf16 copies of the two pre-activations
@@ -167,10 +168,12 @@ int launch_add(const void* a, long long lda, const void* b, long long ldb, const
 // dtype: 0 = bf16, 1 = fp32 (activations and weights; accumulation and the marked fp32 tensors are fp32 in both)
 int launch_seq_linear(int dtype, const void* x, long long ldx, int M, int K, const void* w, long long ldw, int N, const void* bias, int act,
                       void* y, long long ldy, int y_f32, cudaStream_t stream);
+using HeadLinearArgs = plz_head_linear_t;
+int launch_head_linear(int dtype, const HeadLinearArgs& a, cudaStream_t stream);
 int launch_seq_embed(int dtype, const void* table, long long ldt, const long long* ids, long long rows, int W, long long vocab, float scale,
-                     float* x, void* xb, int* bad, cudaStream_t stream);
-int launch_seq_residual_norm(int dtype, const void* y, long long ldy, const float* w, float w_offset, float mult, float eps, long long rows, int W,
-                             float* x, void* xb, cudaStream_t stream);
+                     const float* norm_w, float norm_offset, float eps, float* x, float* x2, void* xb, int* bad, cudaStream_t stream);
+using StreamArgs = plz_stream_t;
+int launch_seq_stream(int dtype, const StreamArgs& a, cudaStream_t stream);
 int launch_seq_rows_norm(int dtype, const float* x, const long long* idx, const float* w, float w_offset, float eps, long long rows, int W, void* out,
                          cudaStream_t stream);
 int launch_seq_norm_gate(int dtype, const float* o, const void* gate, long long ldg, const float* w, float eps, long long rows, int groups, int L,
@@ -192,6 +195,14 @@ long long attn_bias_decode_ws_bytes(int B, int H, int G, int dv, int cap);
 int launch_attn_bias_decode(int dtype, const AttnBiasArgs& a, int cap, void* ws, long long ws_bytes, cudaStream_t stream);
 int launch_attn_bias_tc(const AttnBiasArgs& a, cudaStream_t stream);   // attention_bias_tc.cu
 int launch_attn_bias_simt(int dtype, const AttnBiasArgs& a, cudaStream_t stream);
+// latent_ops.cu / latent_attention.cu / latent_attention_tc.cu: attention over cached latents
+using LatentPrepArgs = plz_latent_prep_t;
+int launch_latent_prep(int dtype, const LatentPrepArgs& a, cudaStream_t stream);
+using RotateArgs = plz_rotate_t;
+int launch_rotate(int dtype, const RotateArgs& a, cudaStream_t stream);
+using LatentAttnArgs = plz_latent_attn_t;
+long long latent_attn_ws_bytes(int dtype, int B, int n, int H, int R, int dr, int cap);
+int launch_latent_attn(int dtype, const LatentAttnArgs& a, void* ws, long long ws_bytes, cudaStream_t stream);
 int launch_advance(int* pos, int n, cudaStream_t stream);
 int launch_sample(const float* logits, long long ld, int rows, int V, float temperature, int top_k, uint32_t seed, const int* pos, long long* out,
                   cudaStream_t stream);

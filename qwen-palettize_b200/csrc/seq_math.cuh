@@ -28,7 +28,10 @@ __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf
 __device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
-enum SeqAct { ACT_NONE = 0, ACT_RELU2 = 1 };
+__device__ __forceinline__ float gelu_tanh_f(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * z * z, z, z))); }
+
+// ACT_GLU_GELU: rows 2 i and 2 i + 1 of the weight are a gate / up pair, output column i is gelu_tanh(gate) * up
+enum SeqAct { ACT_NONE = 0, ACT_RELU2 = 1, ACT_GLU_GELU = 2 };
 __device__ __forceinline__ float activate(float v, int act) {
     if (act == ACT_RELU2) { const float r = fmaxf(v, 0.f); return r * r; }
     return v;

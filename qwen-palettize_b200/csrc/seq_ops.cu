@@ -1,5 +1,5 @@
-// Row-wise steps of the hybrid decoders around their Linears, recurrences and attention: embedding with a scale, the norm on a
-// sublayer's output fused with the fp32 residual update, the norm + gate that closes a recurrent mixer, the short causal
+// Row-wise steps of the hybrid decoders around their Linears, recurrences and attention: embedding with a scale or a norm, the norm on a
+// sublayer's output fused with the fp32 residual update and the norm ahead of the next sublayer, the norm + gate that closes a recurrent mixer, the short causal
 // convolution with its activation, unit norm and decay, the query / key norm that feeds the cache, and token sampling.
 //
 // Rows are b * n + t: B sequences advance in lockstep by n tokens each; *pos (device memory, so that a captured step can be
@@ -9,88 +9,137 @@
 namespace plz {
 namespace {
 
-// x[r, :] = table[ids[r], :] * scale (fp32), xb the same in T (bf16 models: the operand of the first Linear)
+// x[r, :] = table[ids[r], :] * scale (fp32), then (NORM) over its root mean square times w + w_offset; x2 the same, xb the same in T
+// (bf16 models: the operand of the first Linear)
+struct EmbedParams {
+    const void* table; long long ldt; const long long* ids; int W; long long vocab; float scale;
+    const float* w; float w_offset, eps;
+    float* x; float* x2; void* xb; int* bad;
+};
 template <typename T>
 __global__ void __launch_bounds__(256)
-embed_scale_kernel(const T* __restrict__ table, long long ldt, const long long* __restrict__ ids, int W, long long vocab, float scale,
-                   float* __restrict__ x, T* __restrict__ xb, int* __restrict__ bad) {
+embed_scale_kernel(const EmbedParams p) {
+    __shared__ float part[8];
     const long long r = blockIdx.x;
     pdl_launch_dependents();
     pdl_wait();
-    const long long id = ids[r];
-    const bool ok = id >= 0 && id < vocab;
-    if (!ok && bad && threadIdx.x == 0) *bad = 1;
-    for (int c = threadIdx.x; c < W; c += 256) {
-        const float v = ok ? to_f(table[id * ldt + c]) * scale : 0.f;
-        x[r * W + c] = v;
-        if (xb) xb[r * W + c] = from_f<T>(v);
+    const long long id = p.ids[r];
+    const bool ok = id >= 0 && id < p.vocab;
+    if (!ok && p.bad && threadIdx.x == 0) *p.bad = 1;
+    const T* row = (const T*)p.table + (ok ? id : 0) * p.ldt;
+    float rs = 1.f;
+    if (p.w) {
+        float s = 0.f;
+        for (int c = threadIdx.x; c < p.W; c += 256) { const float v = ok ? to_f(row[c]) * p.scale : 0.f; s = fmaf(v, v, s); }
+        rs = 1.0f / sqrtf(block_sum<8>(s, part) / (float)p.W + p.eps);
+    }
+    for (int c = threadIdx.x; c < p.W; c += 256) {
+        float v = ok ? to_f(row[c]) * p.scale : 0.f;
+        if (p.w) v = v * rs * (p.w[c] + p.w_offset);
+        p.x[r * p.W + c] = v;
+        if (p.x2) p.x2[r * p.W + c] = v;
+        if (p.xb) ((T*)p.xb)[r * p.W + c] = from_f<T>(v);
     }
 }
 
-// x += mult * y / rms(y) * (w + w_offset); xb = T(x)
+// x += mult * y / rms(y) * (w + w_offset);  x += add_rows + add_vec;  out = T(x), or T(x / rms(x) * (w_next + w_offset))
+struct StreamParams {
+    const void* y; long long ldy; const float* w; float w_offset, mult, eps; int W;
+    float* x; const float* add_rows; const float* add_vec; const float* w_next; void* out;
+};
 template <typename T>
 __global__ void __launch_bounds__(256)
-residual_norm_kernel(const T* __restrict__ y, long long ldy, const float* __restrict__ w, float w_offset, float mult, float eps, int W,
-                     float* __restrict__ x, T* __restrict__ xb) {
+stream_kernel(const StreamParams p) {
     __shared__ float part[8];
     const long long r = blockIdx.x;
     pdl_launch_dependents();
     pdl_wait();
-    const T* yr = y + r * ldy;
-    float s = 0.f;
-    for (int c = threadIdx.x; c < W; c += 256) { const float v = to_f(yr[c]); s = fmaf(v, v, s); }
-    s = block_sum<8>(s, part);
-    const float rs = 1.0f / sqrtf(s / (float)W + eps);
-    for (int c = threadIdx.x; c < W; c += 256) {
-        const float v = x[r * W + c] + mult * (to_f(yr[c]) * rs * (w[c] + w_offset));
-        x[r * W + c] = v;
-        if (xb) xb[r * W + c] = from_f<T>(v);
+    const T* yr = (const T*)p.y + r * p.ldy;
+    float* xr = p.x + r * p.W;
+    const float* er = p.add_rows ? p.add_rows + r * p.W : nullptr;
+    T* out = (T*)p.out + (p.out ? r * p.W : 0);
+    float rs = 0.f;
+    if (p.y) {
+        float s = 0.f;
+        for (int c = threadIdx.x; c < p.W; c += 256) { const float v = to_f(yr[c]); s = fmaf(v, v, s); }
+        rs = 1.0f / sqrtf(block_sum<8>(s, part) / (float)p.W + p.eps);
+    }
+    float sx = 0.f;
+    for (int c = threadIdx.x; c < p.W; c += 256) {
+        float v = xr[c];
+        if (p.y) v += p.mult * (to_f(yr[c]) * rs * (p.w[c] + p.w_offset));
+        if (er) v += er[c];
+        if (p.add_vec) v += p.add_vec[c];
+        xr[c] = v;
+        sx = fmaf(v, v, sx);
+        if (p.out && !p.w_next) out[c] = from_f<T>(v);
+    }
+    if (p.out && p.w_next) {
+        const float rx = 1.0f / sqrtf(block_sum<8>(sx, part) / (float)p.W + p.eps);
+        for (int c = threadIdx.x; c < p.W; c += 256) out[c] = from_f<T>(xr[c] * rx * (p.w_next[c] + p.w_offset));   // this thread's own x
     }
 }
-// the same for W % 4 == 0 and 16-byte aligned rows, four columns per access, y kept in registers (W <= 4096)
-template <typename T> struct Quad { T v[4]; };
-template <typename T>
+// the same for W % 4 == 0 and 16-byte aligned rows, four columns per access, y and x kept in registers (W <= 1024 * NQ)
+__device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
+    const uint2 r = *reinterpret_cast<const uint2*>(p);
+    return make_float4(__uint_as_float(r.x << 16), __uint_as_float(r.x & 0xFFFF0000u), __uint_as_float(r.y << 16), __uint_as_float(r.y & 0xFFFF0000u));
+}
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w)); }
+__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ float dot4(float4 a) { return a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w; }
+template <typename T, int NQ>
 __global__ void __launch_bounds__(256)
-residual_norm4_kernel(const T* __restrict__ y, long long ldy, const float* __restrict__ w, float w_offset, float mult, float eps, int W,
-                      float* __restrict__ x, T* __restrict__ xb) {
+stream4_kernel(const StreamParams p) {
     __shared__ float part[8];
     const long long r = blockIdx.x;
-    const int n4 = W >> 2;
+    const int n4 = p.W >> 2;
     pdl_launch_dependents();
     pdl_wait();
-    const T* yr = y + r * ldy;
-    float f[4][4];
+    const T* yr = (const T*)p.y + r * p.ldy;
+    float* xr = p.x + r * p.W;
+    const float* er = p.add_rows ? p.add_rows + r * p.W : nullptr;
+    T* out = (T*)p.out + (p.out ? r * p.W : 0);
+    float4 x[NQ], y[NQ];
     float s = 0.f;
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
+    for (int i = 0; i < NQ; ++i) {
         const int c = threadIdx.x + i * 256;
         if (c < n4) {
-            if (sizeof(T) == 2) {
-                const uint2 q = *reinterpret_cast<const uint2*>(yr + c * 4);
-                f[i][0] = __uint_as_float(q.x << 16); f[i][1] = __uint_as_float(q.x & 0xFFFF0000u);
-                f[i][2] = __uint_as_float(q.y << 16); f[i][3] = __uint_as_float(q.y & 0xFFFF0000u);
-            } else {
-                const float4 q = *reinterpret_cast<const float4*>(yr + c * 4);
-                f[i][0] = q.x; f[i][1] = q.y; f[i][2] = q.z; f[i][3] = q.w;
-            }
-#pragma unroll
-            for (int e = 0; e < 4; ++e) s = fmaf(f[i][e], f[i][e], s);
+            x[i] = load4(xr + c * 4);
+            if (p.y) { y[i] = load4(yr + c * 4); s += dot4(y[i]); }
         }
     }
-    s = block_sum<8>(s, part);
-    const float rs = 1.0f / sqrtf(s / (float)W + eps);
+    float rs = 0.f;
+    if (p.y) rs = p.mult / sqrtf(block_sum<8>(s, part) / (float)p.W + p.eps);
+    float sx = 0.f;
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
+    for (int i = 0; i < NQ; ++i) {
         const int c = threadIdx.x + i * 256;
         if (c < n4) {
-            float4 a = *reinterpret_cast<const float4*>(x + r * W + c * 4);
-            const float4 g = __ldg(reinterpret_cast<const float4*>(w + c * 4));
-            a.x += mult * (f[i][0] * rs * (g.x + w_offset)); a.y += mult * (f[i][1] * rs * (g.y + w_offset));
-            a.z += mult * (f[i][2] * rs * (g.z + w_offset)); a.w += mult * (f[i][3] * rs * (g.w + w_offset));
-            *reinterpret_cast<float4*>(x + r * W + c * 4) = a;
-            if (xb) {
-                if (sizeof(T) == 2) *reinterpret_cast<uint2*>(xb + r * W + c * 4) = make_uint2(pack_bf16x2(a.x, a.y), pack_bf16x2(a.z, a.w));
-                else *reinterpret_cast<float4*>(xb + r * W + c * 4) = a;
+            float4 a = x[i];
+            if (p.y) {
+                const float4 g = __ldg(reinterpret_cast<const float4*>(p.w + c * 4));
+                a.x += y[i].x * rs * (g.x + p.w_offset); a.y += y[i].y * rs * (g.y + p.w_offset);
+                a.z += y[i].z * rs * (g.z + p.w_offset); a.w += y[i].w * rs * (g.w + p.w_offset);
+            }
+            if (er) { const float4 e = load4(er + c * 4); a.x += e.x; a.y += e.y; a.z += e.z; a.w += e.w; }
+            if (p.add_vec) { const float4 e = __ldg(reinterpret_cast<const float4*>(p.add_vec + c * 4)); a.x += e.x; a.y += e.y; a.z += e.z; a.w += e.w; }
+            store4(xr + c * 4, a);
+            if (p.out && !p.w_next) store4(out + c * 4, a);
+            sx += dot4(a);
+            x[i] = a;
+        }
+    }
+    if (p.out && p.w_next) {
+        const float rx = 1.0f / sqrtf(block_sum<8>(sx, part) / (float)p.W + p.eps);
+#pragma unroll
+        for (int i = 0; i < NQ; ++i) {
+            const int c = threadIdx.x + i * 256;
+            if (c < n4) {
+                const float4 g = __ldg(reinterpret_cast<const float4*>(p.w_next + c * 4));
+                store4(out + c * 4, make_float4(x[i].x * rx * (g.x + p.w_offset), x[i].y * rx * (g.y + p.w_offset), x[i].z * rx * (g.z + p.w_offset),
+                                                x[i].w * rx * (g.w + p.w_offset)));
             }
         }
     }
@@ -206,11 +255,6 @@ delta_prep_kernel(const DeltaPrep p) {
 // The same for portions: a warp takes one item over kPrepRows consecutive tokens, four channels per lane (head sizes up to 128, a
 // multiple of 4), the convolution's inputs sliding through registers. Up to four taps (missing ones count as zero weights).
 constexpr int kPrepRows = 16;
-__device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
-    const uint2 r = *reinterpret_cast<const uint2*>(p);
-    return make_float4(__uint_as_float(r.x << 16), __uint_as_float(r.x & 0xFFFF0000u), __uint_as_float(r.y << 16), __uint_as_float(r.y & 0xFFFF0000u));
-}
-__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
 template <typename T>
 __global__ void __launch_bounds__(256)
 delta_prep_rows_kernel(const DeltaPrep p) {
@@ -422,25 +466,29 @@ typedef __nv_bfloat16 bf;
 }  // namespace
 
 int launch_seq_embed(int dtype, const void* table, long long ldt, const long long* ids, long long rows, int W, long long vocab, float scale,
-                     float* x, void* xb, int* bad, cudaStream_t stream) {
+                     const float* norm_w, float norm_offset, float eps, float* x, float* x2, void* xb, int* bad, cudaStream_t stream) {
     if (rows <= 0) return PLZ_OK;
-    if (dtype == 1) PLZ_LAUNCH_CHAIN(embed_scale_kernel<float>, dim3((unsigned)rows), dim3(256), 0, stream, (const float*)table, ldt, ids, W, vocab, scale, x, (float*)xb, bad);
-    else PLZ_LAUNCH_CHAIN(embed_scale_kernel<bf>, dim3((unsigned)rows), dim3(256), 0, stream, (const bf*)table, ldt, ids, W, vocab, scale, x, (bf*)xb, bad);
+    const EmbedParams p = {table, ldt, ids, W, vocab, scale, norm_w, norm_offset, eps, x, x2, xb, bad};
+    if (dtype == 1) PLZ_LAUNCH_CHAIN(embed_scale_kernel<float>, dim3((unsigned)rows), dim3(256), 0, stream, p);
+    else PLZ_LAUNCH_CHAIN(embed_scale_kernel<bf>, dim3((unsigned)rows), dim3(256), 0, stream, p);
     return PLZ_OK;
 }
 
 template <typename T>
-static int residual_norm_t(const T* y, long long ldy, const float* w, float off, float mult, float eps, long long rows, int W, float* x, T* xb, cudaStream_t s) {
-    const bool vec = W % 4 == 0 && W <= 4096 && ldy % 4 == 0 && !((uintptr_t)y & 15) && !((uintptr_t)x & 15) && !((uintptr_t)w & 15) && !((uintptr_t)xb & 15);
-    if (vec) PLZ_LAUNCH_CHAIN(residual_norm4_kernel<T>, dim3((unsigned)rows), dim3(256), 0, s, y, ldy, w, off, mult, eps, W, x, xb);
-    else PLZ_LAUNCH_CHAIN(residual_norm_kernel<T>, dim3((unsigned)rows), dim3(256), 0, s, y, ldy, w, off, mult, eps, W, x, xb);
+static int stream_t_(const StreamArgs& a, cudaStream_t s) {
+    const StreamParams p = {a.y, a.ldy, a.w, a.w_offset, a.mult, a.eps, a.W, a.x, a.add_rows, a.add_vec, a.w_next, a.out};
+    const uintptr_t ptrs = (uintptr_t)a.y | (uintptr_t)a.w | (uintptr_t)a.x | (uintptr_t)a.add_rows | (uintptr_t)a.add_vec | (uintptr_t)a.w_next | (uintptr_t)a.out;
+    const bool vec = a.W % 4 == 0 && a.ldy % 4 == 0 && !(ptrs & 15);
+    const dim3 grid((unsigned)a.rows), block(256);
+    if (vec && a.W <= 2048) PLZ_LAUNCH_CHAIN((stream4_kernel<T, 2>), grid, block, 0, s, p);
+    else if (vec && a.W <= 4096) PLZ_LAUNCH_CHAIN((stream4_kernel<T, 4>), grid, block, 0, s, p);
+    else if (vec && a.W <= 8192) PLZ_LAUNCH_CHAIN((stream4_kernel<T, 8>), grid, block, 0, s, p);
+    else PLZ_LAUNCH_CHAIN(stream_kernel<T>, grid, block, 0, s, p);
     return PLZ_OK;
 }
-int launch_seq_residual_norm(int dtype, const void* y, long long ldy, const float* w, float w_offset, float mult, float eps, long long rows, int W,
-                             float* x, void* xb, cudaStream_t stream) {
-    if (rows <= 0) return PLZ_OK;
-    if (dtype == 1) return residual_norm_t<float>((const float*)y, ldy, w, w_offset, mult, eps, rows, W, x, (float*)xb, stream);
-    return residual_norm_t<bf>((const bf*)y, ldy, w, w_offset, mult, eps, rows, W, x, (bf*)xb, stream);
+int launch_seq_stream(int dtype, const StreamArgs& a, cudaStream_t stream) {
+    if (a.rows <= 0) return PLZ_OK;
+    return dtype == 1 ? stream_t_<float>(a, stream) : stream_t_<bf>(a, stream);
 }
 
 int launch_seq_rows_norm(int dtype, const float* x, const long long* idx, const float* w, float w_offset, float eps, long long rows, int W, void* out,

@@ -5,7 +5,10 @@ sequence-length agnostic, so one code path serves whole prompts, portions of pro
     MIXERS['lightning']       decayed linear attention, RMS norm over all heads, sigmoid gate
     MIXERS['channel_delta']   gated delta rule with one decay per head and key channel, short convolutions on q, k, v
     MIXERS['attention']       softmax attention with a learned bias by distance, a sink, whole-projection q / k norm and value mixing
-    MLPS['dense']             W_down relu(W_up x)^2
+    MIXERS['latent_attention']    attention over a cached low-rank latent per token, rotary positions on a part of every head, learned sinks
+    MIXERS['latent_attention_2']  the same without positions and sinks, with an output gate
+    MLPS['relu2']             W_down relu(W_up x)^2
+    MLPS['gated_gelu']        W_down (gelu_tanh(W_gate x) * W_up x)
 """
 from __future__ import annotations
 
@@ -59,20 +62,27 @@ class Loader:
         return self.raw(name, shape).to(self.device, torch.float32).contiguous()
 
     def stack(self, names, shapes, biases: bool = False):
-        """The named matrices one under the other, each starting at a multiple of eight rows (zero rows between), so that one Linear
-        serves all of them and every slice of its output starts on 16 bytes. Returns (weight, bias or None, first row of each)."""
-        K = shapes[0][1]
-        offs, at = [], 0
-        for _, (N, _) in zip(names, shapes):
-            offs.append(at)
-            at += (N + 7) // 8 * 8
-        w = torch.zeros(at, K, dtype=self.dtype, device=self.device)
-        b = torch.zeros(at, dtype=self.dtype, device=self.device) if biases else None
+        """The named matrices one under the other (stack_rows). Returns (weight, bias or None, first row of each)."""
+        w, offs = stack_rows([self.mat(name, shape) for name, shape in zip(names, shapes)])
+        if not biases:
+            return w, None, offs
+        b = torch.zeros(w.shape[0], dtype=self.dtype, device=self.device)
         for name, shape, o in zip(names, shapes, offs):
-            w[o:o + shape[0]] = self.mat(name, shape)
-            if biases:
-                b[o:o + shape[0]] = self.mat(name + ".b", (shape[0],))
+            b[o:o + shape[0]] = self.mat(name + ".b", (shape[0],))
         return w, b, offs
+
+
+def stack_rows(mats):
+    """Matrices one under the other, each starting at a multiple of eight rows (zero rows between), so that one Linear serves all of them
+    and every slice of its output starts on 16 bytes. Returns (weight, first row of each)."""
+    offs, at = [], 0
+    for m in mats:
+        offs.append(at)
+        at += (m.shape[0] + 7) // 8 * 8
+    w = torch.zeros(at, mats[0].shape[1], dtype=mats[0].dtype, device=mats[0].device)
+    for m, o in zip(mats, offs):
+        w[o:o + m.shape[0]] = m
+    return w, offs
 
 
 CHUNK_FROM = 64     # portions of at least this many tokens take the chunked recurrence (bf16 models)
@@ -212,6 +222,125 @@ class BiasAttention:
         return S.linear(o, self.w_out)
 
 
+def rotary_frequencies(rot: dict):
+    """(frequency of every pair, factor on cos and sin) of a rotation entry: base^(-2 i / dims), and with 'scaling' (YaRN) a blend of
+    that and the same over 'factor', by how often a pair turns over the 'original' length: all of it kept above 'fast' turns, all divided
+    below 'slow'."""
+    dims, base, sc = rot["dims"], rot["base"], rot.get("scaling")
+    if dims % 2:
+        raise ValueError(f"rotation of {dims} dimensions")
+    freq = [math.pow(base, -2.0 * i / dims) for i in range(dims // 2)]
+    if not sc:
+        return freq, 1.0
+
+    def dim_of(turns):
+        return dims * math.log(sc["original"] / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+    lo, hi = max(math.floor(dim_of(sc["fast"])), 0), min(math.ceil(dim_of(sc["slow"])), dims - 1)
+    for i, f in enumerate(freq):
+        slow = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
+        freq[i] = f * (slow / sc["factor"] + 1.0 - slow)
+    return freq, 0.1 * math.log(sc["factor"]) + 1.0
+
+
+class LatentAttention:
+    """Attention whose keys and values are products of one normed latent per token, which is all the cache holds (beside one rotated key
+    part that the heads share). Queries pass through a latent of their own.
+
+    Two forms give the same result. *Absorbed*: the key matrix is applied to the queries and the value matrix to the output, and all heads
+    attend to the cached rows themselves: the work of a token grows with the latent's size, nothing is formed per cached token. It serves
+    single tokens and short portions. *Expanded*: keys and values of all cached tokens are formed once per portion and ordinary attention
+    runs on them: fewer products per pair of tokens, for long portions."""
+    ROTATED, SINK, GATE = True, True, False
+
+    def __init__(self, mc: dict, L: Loader, width: int):
+        self.H, self.dn, self.dv = mc["heads"], mc["dim"], mc["vdim"]
+        self.dr = mc["rot_dim"] if self.ROTATED else 0
+        self.rq, self.R, self.scale = mc["q_rank"], mc["kv_rank"], mc["scale"]
+        H, dn, dr, dv, R = self.H, self.dn, self.dr, self.dv, self.R
+        # the latent and the key part are separate slices of the projection, so that each starts on 16 bytes
+        dkv = L.mat("dkv", (R + dr, width))
+        parts = {"dq": L.mat("dq", (self.rq, width)), "c": dkv[:R], "r": dkv[R:]}
+        if self.GATE:
+            parts["g"] = L.mat("g", (H * dv, width))
+        self.w_in, at = stack_rows(list(parts.values()))
+        self.off = dict(zip(parts, at))
+        self.wq, self.wc = L.f32("dq.norm", (self.rq,)), L.f32("dkv.norm", (R,))
+        self.w_uq = L.mat("uq", (H * (dn + dr), self.rq))
+        uk, uv = L.mat("uk", (H * dn, R)), L.mat("uv", (H * dv, R))
+        self.w_kv, (_, self.off_v) = stack_rows([uk, uv])                        # expanded: keys and values of a latent
+        self.w_qk = uk.view(H, dn, R).transpose(1, 2).contiguous()               # absorbed: per head, queries -> latent space
+        self.w_ov = uv.view(H, dv, R)                                            #           per head, latent space -> values
+        self.w_out = L.mat("o", (width, H * dv))
+        self.sinks = L.f32("sink", (H,)) if self.SINK else None
+        self.rot = None
+        if dr:
+            freq, m = rotary_frequencies(mc["rot"])
+            if 2 * len(freq) > dr:
+                raise ValueError(f"rotation of {2 * len(freq)} dimensions in a part of {dr}")
+            self.rot = S.Rotation(torch.tensor(freq, dtype=torch.float64, device=L.device), m)
+
+    @classmethod
+    def shapes(cls, mc: dict, width: int) -> dict:
+        H, dn, dv, R, rq = mc["heads"], mc["dim"], mc["vdim"], mc["kv_rank"], mc["q_rank"]
+        dr = mc["rot_dim"] if cls.ROTATED else 0
+        out = {"dq": (rq, width), "dq.norm": (rq,), "uq": (H * (dn + dr), rq), "dkv": (R + dr, width), "dkv.norm": (R,), "uk": (H * dn, R),
+               "uv": (H * dv, R), "o": (width, H * dv)}
+        if cls.SINK:
+            out["sink"] = (H,)
+        if cls.GATE:
+            out["g"] = (H * dv, width)
+        return out
+
+    def state_spec(self):
+        spec = {"c": StateSpec(("T_max", self.R))}
+        if self.dr:
+            spec["kr"] = StateSpec(("T_max", self.dr))
+        return spec
+
+    def decode_weights(self):
+        """Matrices that a one-token step reads."""
+        return [self.w_in, self.w_uq, self.w_qk, self.w_ov, self.w_out]
+
+    def _absorb(self, ctx: StepContext) -> bool:
+        """Fewer multiplications per head (those of the absorbed attention count twice: its tiles are narrower)."""
+        if ctx.n == 1:
+            return True
+        n, pos = ctx.n, ctx.host_pos
+        pairs, per = n * (pos + 0.5 * n), self.R * (self.dn + self.dv)
+        return n * per + 2 * pairs * (2 * self.R + self.dr) < (pos + n) * per + pairs * (self.dn + self.dr + self.dv)
+
+    def forward(self, x: torch.Tensor, st: dict, ctx: StepContext) -> torch.Tensor:
+        B, n, H, dn, dr, dv, R, off = ctx.B, ctx.n, self.H, self.dn, self.dr, self.dv, self.R, self.off
+        p = S.linear(x, self.w_in)
+        kr = st.get("kr")
+        cq = S.latent_prep(p, (off["dq"], off["c"], off["r"]), self.wq, self.wc, st["c"], kr, self.rot, ctx.pos, B, n, ctx.eps)
+        gate = p[:, off["g"]:off["g"] + H * dv] if self.GATE else None
+        q = S.linear(cq, self.w_uq)
+        q_rot = q.view(B * n, H, dn + dr)[:, :, dn:]
+        if self._absorb(ctx):
+            qa = torch.empty(B * n, H, R + dr, dtype=q.dtype, device=q.device)
+            S.head_linear(q, dn + dr, self.w_qk, qa[:, :, :R])
+            if dr:
+                S.rotate(q_rot, qa[:, :, R:], self.rot, ctx.pos, B, n)
+            o = S.latent_attention(qa, st["c"], kr, self.sinks, ctx.pos, ctx.host_pos, B, n, self.scale)
+            o = S.head_linear(o.view(B * n, H * R), R, self.w_ov, gate=gate).view(B * n, H * dv)
+        else:
+            if dr:
+                S.rotate(q_rot, q_rot, self.rot, ctx.pos, B, n)
+            T = ctx.host_pos + n
+            kv = torch.empty(B, T, self.w_kv.shape[0], dtype=q.dtype, device=q.device)
+            for b in range(B):
+                S.linear(st["c"][b, :T], self.w_kv, out=kv[b])
+            o = S.attention_bias(q, kv, kv[:, :, self.off_v:], None, ctx.pos, ctx.host_pos, B, n, H, H, dn + dr, dv, self.scale, self.SINK, self.sinks, kr,
+                                 gate)
+        return S.linear(o, self.w_out)
+
+
+class GatedLatentAttention(LatentAttention):
+    """Without positions (no rotated part) and sinks; the concatenated heads are multiplied by a sigmoid of a projection of the input."""
+    ROTATED, SINK, GATE = False, False, True
+
+
 class DenseMlp:
     def __init__(self, fc: dict, L: Loader, width: int):
         self.up, self.down = L.mat("up", (fc["ff"], width)), L.mat("down", (width, fc["ff"]))
@@ -224,5 +353,20 @@ class DenseMlp:
         return S.linear(S.linear(x, self.up, act=S.ACT_RELU2), self.down)
 
 
-MIXERS = {"lightning": Lightning, "channel_delta": ChannelDelta, "attention": BiasAttention}
-MLPS = {"dense": DenseMlp}
+class GatedMlp:
+    def __init__(self, fc: dict, L: Loader, width: int):
+        pair = (L.mat("gate", (fc["ff"], width)), L.mat("up", (fc["ff"], width)))
+        self.gate_up = torch.stack(pair, 1).view(2 * fc["ff"], width)        # rows alternate, the Linear's epilogue joins each pair
+        self.down = L.mat("down", (width, fc["ff"]))
+
+    @staticmethod
+    def shapes(fc: dict, width: int) -> dict:
+        return {"gate": (fc["ff"], width), "up": (fc["ff"], width), "down": (width, fc["ff"])}
+
+    def forward(self, x: torch.Tensor) -> torch.Tensor:
+        return S.linear(S.linear(x, self.gate_up, act=S.ACT_GLU_GELU), self.down)
+
+
+MIXERS = {"lightning": Lightning, "channel_delta": ChannelDelta, "attention": BiasAttention, "latent_attention": LatentAttention,
+          "latent_attention_2": GatedLatentAttention}
+MLPS = {"relu2": DenseMlp, "gated_gelu": GatedMlp}

@@ -19,9 +19,9 @@ if _HERE not in sys.path:
 
 import safetensors_io  # noqa: E402
 from decode_model import PalettizedQwen  # noqa: E402
-from hybrid_model import Gopunex  # noqa: E402
+import hybrid_model  # noqa: E402
 
-ARCHITECTURES = {"Gopunex": Gopunex, "PalettizedQwen": PalettizedQwen}
+ARCHITECTURES = {**hybrid_model.ARCHITECTURES, "PalettizedQwen": PalettizedQwen}
 DTYPES = {"bfloat16": torch.bfloat16, "float32": torch.float32}
 
 

@@ -71,7 +71,38 @@ class AttnBias(C.Structure):
     _fields_ = [("q", C.c_void_p), ("ldq", C.c_int64), ("k", C.c_void_p), ("v", C.c_void_p), ("k_batch", C.c_int64), ("v_batch", C.c_int64),
                 ("o", C.c_void_p), ("ldo", C.c_int64), ("bias", C.c_void_p), ("ldb", C.c_int64), ("n_bias", C.c_int32), ("bias_top", C.c_void_p),
                 ("pos", C.c_void_p), ("host_pos", C.c_int32), ("cap", C.c_int32), ("B", C.c_int32), ("n", C.c_int32), ("H", C.c_int32),
-                ("G", C.c_int32), ("dk", C.c_int32), ("dv", C.c_int32), ("sink", C.c_int32), ("scale", C.c_float)]
+                ("G", C.c_int32), ("dk", C.c_int32), ("dv", C.c_int32), ("sink", C.c_int32), ("scale", C.c_float),
+                ("sinks", C.c_void_p), ("k_tok", C.c_int64), ("v_tok", C.c_int64), ("k2", C.c_void_p), ("k2_batch", C.c_int64), ("dk2", C.c_int32),
+                ("gate", C.c_void_p), ("ldg", C.c_int64)]
+
+
+class HeadLinear(C.Structure):
+    _fields_ = [("x", C.c_void_p), ("ldx", C.c_int64), ("xh", C.c_int64), ("w", C.c_void_p), ("y", C.c_void_p), ("ldy", C.c_int64), ("yh", C.c_int64),
+                ("gate", C.c_void_p), ("ldg", C.c_int64), ("M", C.c_int32), ("H", C.c_int32), ("N", C.c_int32), ("K", C.c_int32)]
+
+
+class Stream(C.Structure):
+    _fields_ = [("y", C.c_void_p), ("ldy", C.c_int64), ("w", C.c_void_p), ("w_offset", C.c_float), ("mult", C.c_float), ("eps", C.c_float),
+                ("rows", C.c_int64), ("W", C.c_int32), ("x", C.c_void_p), ("add_rows", C.c_void_p), ("add_vec", C.c_void_p), ("w_next", C.c_void_p),
+                ("out", C.c_void_p)]
+
+
+class LatentPrep(C.Structure):
+    _fields_ = [("proj", C.c_void_p), ("ldp", C.c_int64), ("off_q", C.c_int32), ("off_c", C.c_int32), ("off_r", C.c_int32), ("wq", C.c_void_p),
+                ("wc", C.c_void_p), ("cq", C.c_void_p), ("c", C.c_void_p), ("kr", C.c_void_p), ("c_batch", C.c_int64), ("r_batch", C.c_int64),
+                ("pos", C.c_void_p), ("freq", C.c_void_p), ("pairs", C.c_int32), ("m", C.c_float), ("B", C.c_int32), ("n", C.c_int32),
+                ("q_rank", C.c_int32), ("R", C.c_int32), ("dr", C.c_int32), ("cap", C.c_int32), ("eps", C.c_float)]
+
+
+class Rotate(C.Structure):
+    _fields_ = [("x", C.c_void_p), ("ldx", C.c_int64), ("xh", C.c_int64), ("out", C.c_void_p), ("ldo", C.c_int64), ("oh", C.c_int64), ("pos", C.c_void_p),
+                ("freq", C.c_void_p), ("pairs", C.c_int32), ("m", C.c_float), ("B", C.c_int32), ("n", C.c_int32), ("H", C.c_int32), ("dr", C.c_int32)]
+
+
+class LatentAttn(C.Structure):
+    _fields_ = [("q", C.c_void_p), ("ldq", C.c_int64), ("c", C.c_void_p), ("kr", C.c_void_p), ("c_batch", C.c_int64), ("r_batch", C.c_int64),
+                ("o", C.c_void_p), ("ldo", C.c_int64), ("sinks", C.c_void_p), ("pos", C.c_void_p), ("host_pos", C.c_int32), ("cap", C.c_int32),
+                ("B", C.c_int32), ("n", C.c_int32), ("H", C.c_int32), ("R", C.c_int32), ("dr", C.c_int32), ("scale", C.c_float)]
 
 
 _I32, _I64, _P, _F = C.c_int32, C.c_int64, C.c_void_p, C.c_float
@@ -138,8 +169,13 @@ SIGNATURES = {
     "plz_add": [_P, _I64, _P, _I64, _P, _I64, _I32, _I32, _P, _I64, _P],
     "plz_bwd_dw_hard_lora": [_WP, _P, _I64, _P, _I64, _I32, _P, _P, _P, _I32, _P, _P, _P],
     "plz_seq_linear": [_I32, _P, _I64, _I32, _I32, _P, _I64, _I32, _P, _I32, _P, _I64, _I32, _P],
-    "plz_seq_embed": [_I32, _P, _I64, _P, _I64, _I32, _I64, _F, _P, _P, _P, _P],
-    "plz_seq_residual_norm": [_I32, _P, _I64, _P, _F, _F, _F, _I64, _I32, _P, _P, _P],
+    "plz_head_linear": [_I32, C.POINTER(HeadLinear), _P],
+    "plz_seq_embed": [_I32, _P, _I64, _P, _I64, _I32, _I64, _F, _P, _F, _F, _P, _P, _P, _P, _P],
+    "plz_seq_stream": [_I32, C.POINTER(Stream), _P],
+    "plz_latent_prep": [_I32, C.POINTER(LatentPrep), _P],
+    "plz_rotate": [_I32, C.POINTER(Rotate), _P],
+    "plz_latent_attn_ws_bytes": [_I32, _I32, _I32, _I32, _I32, _I32, _I32],
+    "plz_latent_attn": [_I32, C.POINTER(LatentAttn), _P, _I64, _P],
     "plz_seq_rows_norm": [_I32, _P, _P, _P, _F, _F, _I64, _I32, _P, _P],
     "plz_seq_norm_gate": [_I32, _P, _P, _I64, _P, _F, _I64, _I32, _I32, _P, _P],
     "plz_delta_prep": [_I32, C.POINTER(DeltaPrep), _P],
@@ -154,7 +190,7 @@ SIGNATURES = {
     "plz_distill_loss": [_P, _I64, _P, _I64, _I32, _I32, _F, _F, _F, _P, _P, _P, _I64, _I32, _P],
 }
 _RESTYPES = {"plz_last_error": C.c_char_p, "plz_launch_count": C.c_uint64, "plz_attn_decode_ws_bytes": C.c_int64,
-             "plz_attn_bias_ws_bytes": C.c_int64, "plz_chunk_ws_bytes": C.c_int64}
+             "plz_attn_bias_ws_bytes": C.c_int64, "plz_chunk_ws_bytes": C.c_int64, "plz_latent_attn_ws_bytes": C.c_int64}
 
 
 def lib():

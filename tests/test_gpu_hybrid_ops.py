@@ -41,7 +41,7 @@ def test_linear(dt, M, N, K):
 def test_embedding_and_norms(dt, W):
     import seq_ops as S
     table, ids = rnd(50, W, dt=dt), torch.tensor([[3, 49, 0], [7, 7, 11]]).cuda()
-    x, xb = S.embed(table, ids, 0.37)
+    x, xb, _ = S.embed(table, ids, 0.37)
     assert rel(x, table.double().cpu()[ids.cpu().reshape(-1)] * 0.37) < 1e-6 and (xb is x) == (dt == torch.float32)
     y, w = rnd(6, W, seed=3, dt=dt) * 0.01, rnd(W, seed=4)
     want = x.double().cpu() + 0.7 * O.rms(y.double().cpu(), 1e-3) * (1 + w.double().cpu())
