@@ -1092,7 +1092,7 @@ int32_t plz_attn_bias(int32_t dtype, const plz_attn_bias_t* a, void* ws, int64_t
                      f.k_tok % per16 == 0 && f.v_tok % per16 == 0 && !((uintptr_t)a->q & 15) && !((uintptr_t)a->k & 15) && !((uintptr_t)a->v & 15) && !((uintptr_t)a->k2 & 15);
     const bool plain = !a->k2 && !a->sinks && !a->gate && f.k_tok == (int64_t)a->G * a->dk && f.v_tok == (int64_t)a->G * a->dv;
     if (a->n == 1 && vec && plain && a->dk <= 256 && a->dv <= 256) return launch_attn_bias_decode(dtype, f, a->cap, ws, ws ? ws_bytes : 0, s);
-    if (dtype == 0 && vec && plain && a->n > 1 && dk1 > 0 && (dk1 + 63) / 64 + (a->dk2 + 63) / 64 <= 2 && a->dv <= 128 && a->scale > 0.f && (!a->bias || a->bias_top) &&
+    if (dtype == 0 && vec && a->n > 1 && dk1 > 0 && (dk1 + 63) / 64 + (a->dk2 + 63) / 64 <= 3 && a->dv <= 128 && a->scale > 0.f && (!a->bias || a->bias_top) &&
         a->ldo % 8 == 0 && !((uintptr_t)a->o & 15) && (!a->gate || (a->ldg % 8 == 0 && !((uintptr_t)a->gate & 15))))
         return launch_attn_bias_tc(f, s);
     return launch_attn_bias_simt(dtype, f, s);

@@ -180,14 +180,18 @@ bool on_tensor_cores(int dtype, int R, int dr) { return dtype == 0 && latent_tc_
 // key splits of a launch over a cache of `cap` positions whose length may be known on the device only
 int plan_splits(int dtype, int B, int n, int H, int R, int dr, int cap) {
     const bool tc = on_tensor_cores(dtype, R, dr);
-    const int rows = n * H, step = tc ? kLatTile : kKeys;
-    const long long groups = (long long)B * (tc ? (rows + latent_tc_rows(rows) - 1) / latent_tc_rows(rows) : (rows + kRows - 1) / kRows);
-    const long long want = tc ? seq_sm_count() : 2ll * seq_sm_count();
-    long long s = tc ? want / groups : (want + groups - 1) / groups;
-    const int most = (cap + step - 1) / step;
-    if (s > most) s = most;
-    if (s > kLatMaxSplits) s = kLatMaxSplits;
-    return s < 1 ? 1 : (int)s;
+    const int rows = n * H, step = tc ? kLatTile : kKeys, per = tc ? latent_tc_rows(rows, R, dr) : kRows;
+    const long long groups = (long long)B * ((rows + per - 1) / per);
+    const int tiles = (cap + step - 1) / step, sms = seq_sm_count(), most = tiles < kLatMaxSplits ? tiles : kLatMaxSplits;
+    const long long slots = tc ? sms : 2ll * sms;        // CTAs at once
+    // waves of CTAs times the tiles of each, one more tile's time for start and end
+    int best = 1;
+    long long best_cost = -1;
+    for (int s = 1; s <= most; ++s) {
+        const long long cost = ((groups * s + slots - 1) / slots) * ((tiles + s - 1) / s + 1);
+        if (best_cost < 0 || cost < best_cost) { best = s; best_cost = cost; }
+    }
+    return best;
 }
 
 }  // namespace
@@ -206,7 +210,7 @@ int launch_latent_attn(int dtype, const LatentAttnArgs& a, void* ws, long long w
     l.ws_o = (float*)ws;
     l.ws_ml = l.ws_o + rows * l.splits * a.R;
     int rc;
-    const bool aligned = a.ldq % 8 == 0 && a.c_batch % 8 == 0 && a.r_batch % 8 == 0 && !((uintptr_t)a.q & 15) && !((uintptr_t)a.c & 15) && !((uintptr_t)a.kr & 15);
+    const bool aligned = a.scale > 0.f && a.ldq % 8 == 0 && a.c_batch % 8 == 0 && a.r_batch % 8 == 0 && !((uintptr_t)a.q & 15) && !((uintptr_t)a.c & 15) && !((uintptr_t)a.kr & 15);
     if (on_tensor_cores(dtype, a.R, a.dr) && aligned) {
         rc = launch_latent_tc(a, l, stream);
     } else {

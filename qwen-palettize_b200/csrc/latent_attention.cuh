@@ -18,7 +18,7 @@ struct LatentParams {
 };
 
 bool latent_tc_fits(int R, int dr);
-int latent_tc_rows(int rows);          // query rows of one CTA of the tensor-core form
+int latent_tc_rows(int rows, int R, int dr);          // query rows of one CTA of the tensor-core form
 int launch_latent_tc(const LatentAttnArgs& a, const LatentParams& l, cudaStream_t stream);
 
 }  // namespace plz
