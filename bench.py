@@ -834,7 +834,7 @@ def run_case(a):
     dev = torch.device("cuda", 0)
     if a.case == "hybrid":
         import bench_hybrid
-        bench_hybrid.case(torch, dev)
+        bench_hybrid.case(torch, dev, a.design)
         return
     if a.case in ("layer1", "layer8"):
         M = 1 if a.case == "layer1" else 8
@@ -1176,7 +1176,8 @@ def main():
     ap.add_argument("--pair-gemm", type=int, default=1, help="0: keep the large products on the one-CTA-per-tile kernels (comparison)")
     ap.add_argument("--workload", default="linear", choices=["linear", "distill", "hybrid"],
                     help="linear (default): the benchmark step of one Linear; distill: the super-block distillation step (its own JSON line); "
-                         "hybrid: prefill and decode of the Gopunex decoder beside PalettizedQwen at equal size, and a per-kernel table (JSON lines)")
+                         "hybrid: prefill and decode of a hybrid decoder (--design) beside PalettizedQwen at equal size, and a per-kernel table (JSON lines)")
+    ap.add_argument("--design", default="gopunex", choices=["gopunex", "latodra"], help="--workload hybrid, --case hybrid: which decoder")
     ap.add_argument("--sizes", default="small,medium,large", help="--workload hybrid: which of the sizes small, medium, large")
     ap.add_argument("--case", default=None, help="run ONE kernel of the hot path a few times on a small case and exit (for ncu captures)")
     ap.add_argument("--kernels", action="store_true", help="per-kernel table: one JSON line per measurement")
