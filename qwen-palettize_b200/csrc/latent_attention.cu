@@ -116,7 +116,8 @@ latent_rows_kernel(const RowsParams p) {
     }
 }
 
-// One block per query row: weights exp2(m_s - M) of the splits once, then column sums with independent loads.
+// One block per query row and 256 latent columns: weights exp2(m_s - M) of the splits once, then column sums with independent loads
+// (a split without keys has weight 0 and is not read).
 template <typename T>
 __global__ void __launch_bounds__(128)
 latent_combine_kernel(const LatentParams p, T* __restrict__ o, long long ldo) {
@@ -125,18 +126,18 @@ latent_combine_kernel(const LatentParams p, T* __restrict__ o, long long ldo) {
     const long long row = blockIdx.x;                       // b * n * H + t * H + h
     const int h = (int)(row % p.H), t = threadIdx.x, lane = t & 31, w = t >> 5;
     pdl_launch_dependents();
-    pdl_wait();
     const float sink = p.sinks ? p.sinks[h] * kLatLog2e : kLatNegBig;
-    const float m = t < p.splits ? p.ws_ml[(row * p.splits + t) * 2] : kLatNegBig, l = t < p.splits ? p.ws_ml[(row * p.splits + t) * 2 + 1] : 0.f;
-    float M = fmaxf(m, sink);
+    pdl_wait();
+    const float2 ml = t < p.splits ? *reinterpret_cast<const float2*>(p.ws_ml + (row * p.splits + t) * 2) : make_float2(kLatNegBig, 0.f);
+    float M = fmaxf(ml.x, sink);
 #pragma unroll
     for (int i = 16; i > 0; i >>= 1) M = fmaxf(M, __shfl_xor_sync(0xFFFFFFFFu, M, i));
     if (lane == 0) red[w] = M;
     __syncthreads();
     M = fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3]));
-    const float c = exp2f(m - M);
+    const float c = ml.y > 0.f ? exp2f(ml.x - M) : 0.f;
     wgt[t] = c;
-    float ls = c * l;
+    float ls = c * ml.y;
 #pragma unroll
     for (int i = 16; i > 0; i >>= 1) ls += __shfl_xor_sync(0xFFFFFFFFu, ls, i);
     if (lane == 0) red[4 + w] = ls;
@@ -145,11 +146,14 @@ latent_combine_kernel(const LatentParams p, T* __restrict__ o, long long ldo) {
     const float inv = L > 0.f ? 1.0f / L : 0.f;
     T* dst = o + (row / p.H) * ldo + (long long)h * p.R;
     const float* src = p.ws_o + row * p.splits * p.R;
-    for (int d = t; d < p.R; d += 128) {
+    const int end = min(p.R, (int)(blockIdx.y + 1) * 256);
+    for (int d = (int)blockIdx.y * 256 + t; d < end; d += 128) {
         float acc = 0.f;
 #pragma unroll 8
-        for (int s = 0; s < p.splits; ++s)
-            if (wgt[s] > 0.f) acc = fmaf(wgt[s], src[(long long)s * p.R + d], acc);
+        for (int s = 0; s < p.splits; ++s) {
+            const float f = wgt[s], v = f > 0.f ? __ldcs(src + (long long)s * p.R + d) : 0.f;
+            acc = fmaf(f, v, acc);
+        }
         dst[d] = from_f<T>(acc * inv);
     }
 }
@@ -207,8 +211,8 @@ int launch_latent_attn(int dtype, const LatentAttnArgs& a, void* ws, long long w
     l.n = a.n; l.H = a.H; l.R = a.R; l.dr = a.dr; l.scale = a.scale; l.sinks = a.sinks;
     l.splits = plan_splits(dtype, a.B, a.n, a.H, a.R, a.dr, a.cap);
     const long long rows = (long long)a.B * a.n * a.H;
-    l.ws_o = (float*)ws;
-    l.ws_ml = l.ws_o + rows * l.splits * a.R;
+    l.ws_ml = (float*)ws;
+    l.ws_o = l.ws_ml + rows * l.splits * 2;
     int rc;
     const bool aligned = a.scale > 0.f && a.ldq % 8 == 0 && a.c_batch % 8 == 0 && a.r_batch % 8 == 0 && !((uintptr_t)a.q & 15) && !((uintptr_t)a.c & 15) && !((uintptr_t)a.kr & 15);
     if (on_tensor_cores(dtype, a.R, a.dr) && aligned) {
@@ -219,8 +223,8 @@ int launch_latent_attn(int dtype, const LatentAttnArgs& a, void* ws, long long w
         rc = dtype == 1 ? launch_rows<float>(p, a.B, stream) : launch_rows<__nv_bfloat16>(p, a.B, stream);
     }
     if (rc) return rc;
-    if (dtype == 1) PLZ_LAUNCH_CHAIN(latent_combine_kernel<float>, dim3((unsigned)rows), dim3(128), 0, stream, l, (float*)a.o, a.ldo);
-    else PLZ_LAUNCH_CHAIN(latent_combine_kernel<__nv_bfloat16>, dim3((unsigned)rows), dim3(128), 0, stream, l, (__nv_bfloat16*)a.o, a.ldo);
+    if (dtype == 1) PLZ_LAUNCH_CHAIN(latent_combine_kernel<float>, dim3((unsigned)rows, (a.R + 255) / 256), dim3(128), 0, stream, l, (float*)a.o, a.ldo);
+    else PLZ_LAUNCH_CHAIN(latent_combine_kernel<__nv_bfloat16>, dim3((unsigned)rows, (a.R + 255) / 256), dim3(128), 0, stream, l, (__nv_bfloat16*)a.o, a.ldo);
     return PLZ_OK;
 }
 

@@ -7,10 +7,10 @@
 //   O^T [latent column = lane][query row] += C^T P^T          the SAME shared-memory tile read MN-major, P^T written by the softmax threads
 // A cached byte enters shared memory once and serves as key and as value.
 //
-// One CTA takes N query rows of a sequence and one split of its keys, 128 keys at a time. Warps 0-3 are the softmax threads (thread = key),
-// warp 4 issues the MMAs, warp 5 the copies. A tile arrives as units of 128 latent columns (32 KB) in a ring plus the shared key part; a unit
+// One CTA takes N query rows of a sequence and one split of its keys, 128 keys at a time. Warps 0-7 are the softmax threads (thread = key and
+// half of the query rows), warp 8 issues the MMAs, warp 9 the copies. A tile arrives as units of 128 latent columns (32 KB) in a ring plus the shared key part; a unit
 // is handed back as soon as the value product of its columns has run, so that the next tile streams in under the rest of the current one.
-// The maximum of a query row runs over the lanes: 31 shuffles per 32 rows inside a warp, the four warps meet in shared memory. The reference
+// The maximum of a query row runs over the lanes: recursive halving inside a warp, its four warps meet in shared memory. The reference
 // of the exponentials moves only when the maximum has grown by more than 8 (in log2 units), so O^T is rarely rescaled. Rows of the last
 // tile beyond the sequence are cleared in shared memory (a weight of zero times whatever lies there would not be safe).
 // Partial sums of the key splits go to the workspace that latent_combine_kernel merges.
@@ -20,7 +20,7 @@
 namespace plz {
 namespace {
 
-constexpr int kLatThreads = 192;
+constexpr int kLatThreads = 320;
 constexpr uint32_t kUnit = 2 * kBlk;            // 128 keys x 128 latent columns
 constexpr uint32_t kPBytes = 128 * 128;         // P^T: 128 keys x 64 query rows
 constexpr int kMaxUnits = 8;
@@ -38,6 +38,7 @@ struct LatTcParams {
     StatusWord* status;
 };
 
+__device__ __forceinline__ float join(float a, float b, bool max) { return max ? fmaxf(a, b) : a + b; }
 template <int W, bool MAX>
 __device__ __forceinline__ float over_lanes(float (&v)[W], int lane) {     // lane (mod W) gets the result of column lane (mod W)
 #pragma unroll
@@ -46,80 +47,88 @@ __device__ __forceinline__ float over_lanes(float (&v)[W], int lane) {     // la
 #pragma unroll
         for (int i = 0; i < half; ++i) {
             const float send = up ? v[i] : v[i + half], keep = up ? v[i + half] : v[i];
-            const float got = __shfl_xor_sync(0xFFFFFFFFu, send, half);
-            v[i] = MAX ? fmaxf(keep, got) : keep + got;
+            v[i] = join(keep, __shfl_xor_sync(0xFFFFFFFFu, send, half), MAX);
         }
     }
     float r = v[0];
-    if (W == 16) {
-        const float got = __shfl_xor_sync(0xFFFFFFFFu, r, 16);
-        r = MAX ? fmaxf(r, got) : r + got;
+#pragma unroll
+    for (int o = W; o < 32; o <<= 1) r = join(r, __shfl_xor_sync(0xFFFFFFFFu, r, o), MAX);
+    return r;
+}
+// result of every one of NC columns (8, 16, 24, 32) over the 32 lanes: lane i gets column i, for 24 columns lanes 16 .. 31 get 16 + i % 8
+template <int NC, bool MAX>
+__device__ __forceinline__ float columns_over_lanes(const float (&s)[NC], int lane) {
+    constexpr int W = NC == 24 ? 16 : NC;
+    float t[W];
+#pragma unroll
+    for (int i = 0; i < W; ++i) t[i] = s[i];
+    float r = over_lanes<W, MAX>(t, lane);
+    if (NC == 24) {
+        float u[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) u[i] = s[NC - 8 + i];
+        const float q = over_lanes<8, MAX>(u, lane);
+        if (lane >= 16) r = q;
     }
     return r;
 }
+// the column of a half that a lane holds after that
+template <int NC>
+__device__ __forceinline__ int column_of(int lane) { return NC == 24 ? (lane < 16 ? lane : 16 + (lane & 7)) : (lane & (NC - 1)); }
 
-// N / 16 groups of 16 columns from TMEM
-template <int N>
-__device__ __forceinline__ void load_cols(uint32_t t, float (&s)[N]) {
-#pragma unroll
-    for (int g = 0; g < N / 32; ++g) {
+__device__ __forceinline__ void tmem_st_32x8(uint32_t taddr, const uint32_t (&r)[8]) {
+    asm volatile("tcgen05.st.sync.aligned.32x32b.x8.b32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8};"
+                 ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]) : "memory");
+}
+template <int NC>
+__device__ __forceinline__ void load_cols(uint32_t t, float (&s)[NC]) {
+    if (NC == 32) {
         uint32_t v[32];
-        tmem_ld_32x32(t + g * 32, v);
+        tmem_ld_32x32(t, v);
 #pragma unroll
-        for (int i = 0; i < 32; ++i) s[g * 32 + i] = __uint_as_float(v[i]);
+        for (int i = 0; i < 32; ++i) s[i % NC] = __uint_as_float(v[i]);
     }
-    if (N % 32) {
+    if (NC & 16) {
         uint32_t v[16];
-        tmem_ld_32x16(t + N / 32 * 32, v);
+        tmem_ld_32x16(t, v);
 #pragma unroll
-        for (int i = 0; i < 16; ++i) s[N / 32 * 32 + i] = __uint_as_float(v[i]);
+        for (int i = 0; i < 16; ++i) s[i % NC] = __uint_as_float(v[i]);
+    }
+    if (NC & 8) {
+        uint32_t v[8];
+        tmem_ld_32x8(t + (NC - 8), v);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) s[NC - 8 + i] = __uint_as_float(v[i]);
     }
 }
-template <int N>
-__device__ __forceinline__ void store_cols(uint32_t t, const float (&s)[N]) {
-#pragma unroll
-    for (int g = 0; g < N / 32; ++g) {
+template <int NC>
+__device__ __forceinline__ void store_cols(uint32_t t, const float (&s)[NC]) {
+    if (NC == 32) {
         uint32_t v[32];
 #pragma unroll
-        for (int i = 0; i < 32; ++i) v[i] = __float_as_uint(s[g * 32 + i]);
-        tmem_st_32x32(t + g * 32, v);
+        for (int i = 0; i < 32; ++i) v[i] = __float_as_uint(s[i % NC]);
+        tmem_st_32x32(t, v);
     }
-    if (N % 32) {
+    if (NC & 16) {
         uint32_t v[16];
 #pragma unroll
-        for (int i = 0; i < 16; ++i) v[i] = __float_as_uint(s[N / 32 * 32 + i]);
-        tmem_st_32x16(t + N / 32 * 32, v);
-        tmem_wait_st();
+        for (int i = 0; i < 16; ++i) v[i] = __float_as_uint(s[i % NC]);
+        tmem_st_32x16(t, v);
     }
-}
-// result of every column over the 32 lanes: lane i gets columns i (r[0]) and, for N > 32, 32 + i (mod 16 for a group of 16; r[1])
-template <int N, bool MAX>
-__device__ __forceinline__ void columns_over_lanes(const float (&s)[N], int lane, float (&r)[2]) {
-    if (N >= 32) {
-        float t[32];
+    if (NC & 8) {
+        uint32_t v[8];
 #pragma unroll
-        for (int i = 0; i < 32; ++i) t[i] = s[i];
-        r[0] = over_lanes<32, MAX>(t, lane);
+        for (int i = 0; i < 8; ++i) v[i] = __float_as_uint(s[NC - 8 + i]);
+        tmem_st_32x8(t + (NC - 8), v);
     }
-    if (N == 64) {
-        float t[32];
-#pragma unroll
-        for (int i = 0; i < 32; ++i) t[i] = s[N - 32 + i];
-        r[1] = over_lanes<32, MAX>(t, lane);
-    }
-    if (N % 32) {
-        float t[16];
-#pragma unroll
-        for (int i = 0; i < 16; ++i) t[i] = s[N - 16 + i];
-        r[N / 32] = over_lanes<16, MAX>(t, lane);
-    }
+    tmem_wait_st();
 }
 
 template <int N>
 __global__ void __launch_bounds__(kLatThreads, 1)
 latent_tc_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant__ CUtensorMap tmR, const __grid_constant__ CUtensorMap tmQ,
                  const __grid_constant__ CUtensorMap tmQr, const LatTcParams p) {
-    constexpr int G = (N + 31) / 32;            // column groups of a lane
+    constexpr int NC = N / 2;                   // query rows of a softmax thread
     extern __shared__ uint8_t smem_raw[];
     const uint32_t raw = smem_u32(smem_raw);
     const uint32_t base = (raw + 1023u) & ~1023u;
@@ -130,11 +139,12 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant_
     auto r_full = [&](int s) { return bar + 128u + 8u * s; };
     auto r_empty = [&](int s) { return bar + 144u + 8u * s; };
     auto s_full = [&](int s) { return bar + 160u + 8u * s; };
-    const uint32_t q_full = bar + 176, p_full = bar + 184, o_done = bar + 192, mx_full = bar + 200;
-    volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(smem + p.off_x + 208);
+    const uint32_t q_full = bar + 176, p_full = bar + 184, o_done = bar + 192;
+    auto mx_full = [&](int half) { return bar + 200u + 8u * half; };
+    volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(smem + p.off_x + 216);
     volatile uint32_t* abort_flag = tmem_slot + 1;
-    float* wmax = reinterpret_cast<float*>(smem + p.off_x + 256);         // [2][4][64]
-    float* own = wmax + 2 * 4 * 64;                                       // per warp: [64] reference, [64] correction
+    float* wmax = reinterpret_cast<float*>(smem + p.off_x + 256);         // [2][8 warps][32]
+    float* own = wmax + 2 * 8 * 32;                                       // per warp: [32] reference, [32] correction
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int split = blockIdx.x, r0 = (int)blockIdx.y * N, b = blockIdx.z;
@@ -142,12 +152,12 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant_
     if (threadIdx.x == 0) {
         for (int s = 0; s < kMaxUnits; ++s) { mbar_init(u_full(s), 1); mbar_init(u_empty(s), 1); }
         for (int s = 0; s < 2; ++s) { mbar_init(r_full(s), 1); mbar_init(r_empty(s), 1); mbar_init(s_full(s), 1); }
-        mbar_init(q_full, 1); mbar_init(p_full, 4); mbar_init(o_done, 1); mbar_init(mx_full, 4);
+        mbar_init(q_full, 1); mbar_init(p_full, 8); mbar_init(o_done, 1); mbar_init(mx_full(0), 4); mbar_init(mx_full(1), 4);
         *abort_flag = 0;
         mbar_fence_init();
     }
-    if (warp == 4) { tmem_alloc(smem_u32((const void*)tmem_slot), p.tmem_cols); tmem_relinquish(); }
-    if (warp == 5 && lane == 0) { tma_prefetch_desc(&tmC); tma_prefetch_desc(&tmQ); if (p.r_blocks) { tma_prefetch_desc(&tmR); tma_prefetch_desc(&tmQr); } }
+    if (warp == 8) { tmem_alloc(smem_u32((const void*)tmem_slot), p.tmem_cols); tmem_relinquish(); }
+    if (warp == 9 && lane == 0) { tma_prefetch_desc(&tmC); tma_prefetch_desc(&tmQ); if (p.r_blocks) { tma_prefetch_desc(&tmR); tma_prefetch_desc(&tmQr); } }
     tc_fence_before_sync();
     __syncthreads();
     tc_fence_after_sync();
@@ -164,7 +174,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant_
     const int k0 = split * chunk, k1 = min(total, k0 + chunk);
     const int tiles = k1 > k0 ? (k1 - k0 + kT - 1) / kT : 0;
 
-    if (warp == 5) {
+    if (warp == 9) {
         if (lane == 0 && tiles > 0) {
             bool ok = true;
             mbar_arrive_expect_tx(q_full, (uint32_t)(p.c_blocks + p.r_blocks) * N * 128u);
@@ -199,7 +209,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant_
             for (int i = nr > p.r_ring ? nr - p.r_ring : 0; i < nr; ++i)
                 while (!mbar_try_wait(r_full(i % p.r_ring), (i / p.r_ring) & 1) && globaltimer_ns() - t0 < 100000000ull) {}
         }
-    } else if (warp == 4) {
+    } else if (warp == 8) {
         if (lane == 0 && tiles > 0) {
             const uint32_t id_s = make_idesc(128, N, 0, 0), id_o = make_idesc(128, N, 1, 1);
             const uint64_t dq = make_sdesc(base + p.off_q, 16u, 1024u), dp = make_sdesc(base + p.off_p, kBlk, 1024u);
@@ -252,67 +262,55 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant_
             }
         }
     } else {
-        const int t = threadIdx.x;                                        // key of the tile = TMEM lane
-        const uint32_t lane_off = (uint32_t)(warp * 32) << 16;
+        const int quarter = warp & 3, half = warp >> 2, t = quarter * 32 + lane;     // t: key of the tile = TMEM lane
+        const int c0 = half * NC, mine = column_of<NC>(lane);                        // first query row of this thread; the one it owns after a reduction
+        const uint32_t lane_off = ((uint32_t)(quarter * 32) << 16) + (uint32_t)c0;
         const float c = p.l.scale * kLatLog2e;
         const int lim0 = pos + r0 / H;                                    // last key that every row of this CTA sees
-        float* my_m = own + warp * 128;
-        float* my_a = my_m + 64;
-        float l[N], m_run[2] = {kLatNegBig, kLatNegBig};
+        float* my_m = own + warp * 64;
+        float* my_a = my_m + 32;
+        float l[NC], m_run = kLatNegBig;
 #pragma unroll
-        for (int i = 0; i < N; ++i) l[i] = 0.f;
+        for (int i = 0; i < NC; ++i) l[i] = 0.f;
         // a warp goes on or gives up as one
         auto wait = [&](uint32_t mbar, uint32_t parity, uint32_t role) {
             return __all_sync(0xFFFFFFFFu, mbar_wait(mbar, parity, abort_flag, p.status, ST_TIMEOUT_ACCUM, role)) != 0;
         };
+        // the four warps of a half exchange a value per query row; a buffer is written again two exchanges later
+        auto publish = [&](int j, float v) {
+            wmax[(j & 1) * 256 + warp * 32 + lane] = v;
+            __syncwarp();
+            if (lane == 0) mbar_arrive(mx_full(half));
+        };
+        auto shared_by = [&](int j, int w) { return wmax[(j & 1) * 256 + (half * 4 + w) * 32 + lane]; };
         bool ok = true;
         for (int j = 0; j < tiles && ok; ++j) {
             const int tok = k0 + j * kT + t;
             ok = wait(s_full(j & 1), (j >> 1) & 1, 86);
             if (!ok) break;
             tc_fence_after_sync();
-            float s[N];
-            load_cols<N>(tS(j & 1) + lane_off, s);
+            float s[NC];
+            load_cols<NC>(tS(j & 1) + lane_off, s);
             if (k0 + j * kT + kT - 1 > min(lim0, k1 - 1)) {               // some key of the tile is hidden from some row
 #pragma unroll
-                for (int i = 0; i < N; ++i)
-                    if (tok >= k1 || tok > pos + (r0 + i) / H) s[i] = -INFINITY;
+                for (int i = 0; i < NC; ++i)
+                    if (tok >= k1 || tok > pos + (r0 + c0 + i) / H) s[i] = -INFINITY;
             }
-#pragma unroll
-            for (int i = 0; i < N; ++i) s[i] *= c;
-            float mx[2];
-            columns_over_lanes<N, true>(s, lane, mx);
-            float* w = wmax + (j & 1) * 256 + warp * 64;
-            w[lane] = mx[0];
-            if (G == 2) w[32 + lane] = mx[1];
-            __syncwarp();
-            if (lane == 0) mbar_arrive(mx_full);
-            ok = wait(mx_full, j & 1, 87);
+            publish(j, columns_over_lanes<NC, true>(s, lane) * c);
+            ok = wait(mx_full(half), j & 1, 87);
             if (!ok) break;
-            bool moved = false;
-#pragma unroll
-            for (int g = 0; g < G; ++g) {
-                const float* a = wmax + (j & 1) * 256 + g * 32 + lane;
-                const float m = fmaxf(fmaxf(a[0], a[64]), fmaxf(a[128], a[192]));
-                const bool up = m > m_run[g] + kLazy;
-                my_a[g * 32 + lane] = up ? exp2f(m_run[g] - m) : 1.0f;
-                if (up) m_run[g] = m;
-                my_m[g * 32 + lane] = m_run[g];
-                moved |= up;
-            }
-            moved = __any_sync(0xFFFFFFFFu, moved);                       // the same in all four warps; orders the writes above
+            const float m = fmaxf(fmaxf(shared_by(j, 0), shared_by(j, 1)), fmaxf(shared_by(j, 2), shared_by(j, 3)));
+            const bool up = m > m_run + kLazy;
+            my_a[mine] = up ? exp2f(m_run - m) : 1.0f;
+            if (up) m_run = m;
+            my_m[mine] = m_run;
+            const bool moved = __any_sync(0xFFFFFFFFu, up);               // the same in all four warps
             __syncwarp();
 #pragma unroll
-            for (int i = 0; i < N; i += 4) {
-                const float4 m = *reinterpret_cast<const float4*>(my_m + i);
-                s[i] = exp2f(s[i] - m.x); s[i + 1] = exp2f(s[i + 1] - m.y); s[i + 2] = exp2f(s[i + 2] - m.z); s[i + 3] = exp2f(s[i + 3] - m.w);
-            }
-            if (moved) {
-#pragma unroll
-                for (int i = 0; i < N; ++i) l[i] = fmaf(l[i], my_a[i], s[i]);
-            } else {
-#pragma unroll
-                for (int i = 0; i < N; ++i) l[i] += s[i];
+            for (int i = 0; i < NC; i += 4) {
+                const float4 r = *reinterpret_cast<const float4*>(my_m + i);
+                s[i] = exp2f(fmaf(s[i], c, -r.x)); s[i + 1] = exp2f(fmaf(s[i + 1], c, -r.y));
+                s[i + 2] = exp2f(fmaf(s[i + 2], c, -r.z)); s[i + 3] = exp2f(fmaf(s[i + 3], c, -r.w));
             }
             if (j > 0) {                                                  // P^T and O^T are free once the products of the tile before have run
                 ok = wait(o_done, (j - 1) & 1, 88);
@@ -320,69 +318,66 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant_
                 tc_fence_after_sync();
                 if (moved) {
 #pragma unroll 1
-                    for (int m = 0; m < p.units; ++m) {
-                        float o[N];
-                        load_cols<N>(tO(m) + lane_off, o);
+                    for (int u = 0; u < p.units; ++u) {
+                        float o[NC];
+                        load_cols<NC>(tO(u) + lane_off, o);
 #pragma unroll
-                        for (int i = 0; i < N; ++i) o[i] *= my_a[i];
-                        store_cols<N>(tO(m) + lane_off, o);
+                        for (int i = 0; i < NC; ++i) o[i] *= my_a[i];
+                        store_cols<NC>(tO(u) + lane_off, o);
                     }
                 }
             }
 #pragma unroll
-            for (int q = 0; q < N / 8; ++q)
-                *reinterpret_cast<uint4*>(smem + p.off_p + swz128(t, q)) =
+            for (int q = 0; q < NC / 8; ++q)
+                *reinterpret_cast<uint4*>(smem + p.off_p + swz128(t, (c0 >> 3) + q)) =
                     make_uint4(pack_bf16x2(s[q * 8], s[q * 8 + 1]), pack_bf16x2(s[q * 8 + 2], s[q * 8 + 3]), pack_bf16x2(s[q * 8 + 4], s[q * 8 + 5]),
                                pack_bf16x2(s[q * 8 + 6], s[q * 8 + 7]));
-            if (tok >= total) {                                           // past the sequence: whatever the cache holds there must not count
-                for (int m = 0; m < p.units; ++m) {
-                    uint8_t* u = smem + ((j * p.units + m) % p.ring) * kUnit + t * 128;
+            if (tok >= total && half == 0) {                              // past the sequence: whatever the cache holds there must not count
+                for (int u = 0; u < p.units; ++u) {
+                    uint8_t* z = smem + ((j * p.units + u) % p.ring) * kUnit + t * 128;
 #pragma unroll
-                    for (int i = 0; i < 16; ++i) *reinterpret_cast<uint4*>(u + (i >> 3) * kBlk + (i & 7) * 16) = make_uint4(0u, 0u, 0u, 0u);
+                    for (int i = 0; i < 16; ++i) *reinterpret_cast<uint4*>(z + (i >> 3) * kBlk + (i & 7) * 16) = make_uint4(0u, 0u, 0u, 0u);
                 }
             }
             tc_fence_before_sync();
             fence_proxy_async_smem();
             __syncwarp();
             if (lane == 0) mbar_arrive(p_full);
+            if (moved) {
+#pragma unroll
+                for (int i = 0; i < NC; ++i) l[i] *= my_a[i];
+            }
+#pragma unroll
+            for (int i = 0; i < NC; ++i) l[i] += s[i];
+            __syncwarp();                                                 // my_m, my_a are written again in the next tile
         }
-        if (ok && tiles > 0) ok = wait(o_done, (tiles - 1) & 1, 89);
         if (ok) {
-            const long long row0 = (long long)b * rows + r0;
+            publish(tiles, columns_over_lanes<NC, false>(l, lane));
+            const long long row0 = (long long)b * rows + r0 + c0;
             const int S = p.l.splits;
-            if (tiles > 0) {
+            ok = wait(mx_full(half), tiles & 1, 90);
+            if (ok && quarter == 0 && lane < NC && r0 + c0 + mine < rows) {
+                float* ml = p.l.ws_ml + ((row0 + mine) * S + split) * 2;
+                ml[0] = m_run;
+                ml[1] = shared_by(tiles, 0) + shared_by(tiles, 1) + shared_by(tiles, 2) + shared_by(tiles, 3);
+            }
+            if (ok && tiles > 0) ok = wait(o_done, (tiles - 1) & 1, 89);
+            if (ok && tiles > 0) {
                 tc_fence_after_sync();
+                const int valid = min(NC, rows - r0 - c0);
+                const long long step = (long long)S * R;
 #pragma unroll 1
-                for (int m = 0; m < p.units; ++m) {
-                    float o[N];
-                    load_cols<N>(tO(m) + lane_off, o);
-                    const int d = m * 128 + t;
+                for (int u = 0; u < p.units; ++u) {
+                    float o[NC];
+                    load_cols<NC>(tO(u) + lane_off, o);
+                    const int d = u * 128 + t;
                     if (d < R) {
                         float* dst = p.l.ws_o + (row0 * S + split) * R + d;
 #pragma unroll
-                        for (int i = 0; i < N; ++i)
-                            if (r0 + i < rows) dst[(long long)i * S * R] = o[i];
-                    }
-                }
-            }
-            float ls[2];
-            columns_over_lanes<N, false>(l, lane, ls);
-            // the exchange buffer of the other parity than the last tile's
-            float* w = wmax + (tiles & 1) * 256 + warp * 64;
-            w[lane] = ls[0];
-            if (G == 2) w[32 + lane] = ls[1];
-            __syncwarp();
-            if (lane == 0) mbar_arrive(mx_full);
-            ok = wait(mx_full, tiles & 1, 90);
-            if (ok && warp == 0) {
-#pragma unroll
-                for (int g = 0; g < G; ++g) {
-                    const int i = g * 32 + lane;
-                    const float* a = wmax + (tiles & 1) * 256 + i;
-                    if (i < N && r0 + i < rows) {
-                        float* ml = p.l.ws_ml + ((row0 + i) * S + split) * 2;
-                        ml[0] = m_run[g];
-                        ml[1] = a[0] + a[64] + a[128] + a[192];
+                        for (int i = 0; i < NC; ++i) {
+                            if (i < valid) *dst = o[i];
+                            dst += step;
+                        }
                     }
                 }
             }
@@ -390,7 +385,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant_
     }
     tc_fence_before_sync();
     __syncthreads();
-    if (warp == 4) { tc_fence_after_sync(); tmem_dealloc(tmem, p.tmem_cols); }
+    if (warp == 8) { tc_fence_after_sync(); tmem_dealloc(tmem, p.tmem_cols); }
 }
 
 // shared-memory plan of a CTA with N query rows; false if it does not fit

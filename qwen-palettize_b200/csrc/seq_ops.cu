@@ -100,28 +100,26 @@ stream4_kernel(const StreamParams p) {
     float* xr = p.x + r * p.W;
     const float* er = p.add_rows ? p.add_rows + r * p.W : nullptr;
     T* out = (T*)p.out + (p.out ? r * p.W : 0);
-    float4 x[NQ], y[NQ];
-    float s = 0.f;
+    float4 x[NQ];                  // the sublayer's output, then the stream
+    float s = 0.f, rs = 0.f;
+    if (p.y) {
 #pragma unroll
-    for (int i = 0; i < NQ; ++i) {
-        const int c = threadIdx.x + i * 256;
-        if (c < n4) {
-            x[i] = load4(xr + c * 4);
-            if (p.y) { y[i] = load4(yr + c * 4); s += dot4(y[i]); }
+        for (int i = 0; i < NQ; ++i) {
+            const int c = threadIdx.x + i * 256;
+            if (c < n4) { x[i] = load4(yr + c * 4); s += dot4(x[i]); }
         }
+        rs = p.mult / sqrtf(block_sum<8>(s, part) / (float)p.W + p.eps);
     }
-    float rs = 0.f;
-    if (p.y) rs = p.mult / sqrtf(block_sum<8>(s, part) / (float)p.W + p.eps);
     float sx = 0.f;
 #pragma unroll
     for (int i = 0; i < NQ; ++i) {
         const int c = threadIdx.x + i * 256;
         if (c < n4) {
-            float4 a = x[i];
+            float4 a = load4(xr + c * 4);
             if (p.y) {
                 const float4 g = __ldg(reinterpret_cast<const float4*>(p.w + c * 4));
-                a.x += y[i].x * rs * (g.x + p.w_offset); a.y += y[i].y * rs * (g.y + p.w_offset);
-                a.z += y[i].z * rs * (g.z + p.w_offset); a.w += y[i].w * rs * (g.w + p.w_offset);
+                a.x += x[i].x * rs * (g.x + p.w_offset); a.y += x[i].y * rs * (g.y + p.w_offset);
+                a.z += x[i].z * rs * (g.z + p.w_offset); a.w += x[i].w * rs * (g.w + p.w_offset);
             }
             if (er) { const float4 e = load4(er + c * 4); a.x += e.x; a.y += e.y; a.z += e.z; a.w += e.w; }
             if (p.add_vec) { const float4 e = __ldg(reinterpret_cast<const float4*>(p.add_vec + c * 4)); a.x += e.x; a.y += e.y; a.z += e.z; a.w += e.w; }

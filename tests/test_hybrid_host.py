@@ -169,6 +169,7 @@ def test_oracle_against_closed_forms():
     """The plain implementation on inputs whose answers are known."""
     import gopunex_oracle as O
     d = torch.float64
+    torch.manual_seed(0)
     # decay 0: only the current token is left
     q, k, v = (torch.randn(5, 3, dtype=d) for _ in range(3))
     o = O.decayed_linear_attention(q, k, v, 0.0)
