@@ -116,13 +116,14 @@ latent_rows_kernel(const RowsParams p) {
     }
 }
 
-// One block per query row and 256 latent columns: weights exp2(m_s - M) of the splits once, then column sums with independent loads
-// (a split without keys has weight 0 and is not read).
-template <typename T>
+// One block per query row and 32 * V latent columns, V per lane; the four warps share the splits. Weights exp2(m_s - M) of the splits
+// once. A split without keys has weight 0 and was not written: the first one, which always has some, is read in its place.
+template <typename T, int V>
 __global__ void __launch_bounds__(128)
 latent_combine_kernel(const LatentParams p, T* __restrict__ o, long long ldo) {
     __shared__ float wgt[kLatMaxSplits];
     __shared__ float red[8];
+    __shared__ float sum[4][32 * V];
     const long long row = blockIdx.x;                       // b * n * H + t * H + h
     const int h = (int)(row % p.H), t = threadIdx.x, lane = t & 31, w = t >> 5;
     pdl_launch_dependents();
@@ -144,18 +145,39 @@ latent_combine_kernel(const LatentParams p, T* __restrict__ o, long long ldo) {
     __syncthreads();
     const float L = red[4] + red[5] + red[6] + red[7] + (p.sinks ? exp2f(sink - M) : 0.f);
     const float inv = L > 0.f ? 1.0f / L : 0.f;
-    T* dst = o + (row / p.H) * ldo + (long long)h * p.R;
-    const float* src = p.ws_o + row * p.splits * p.R;
-    const int end = min(p.R, (int)(blockIdx.y + 1) * 256);
-    for (int d = (int)blockIdx.y * 256 + t; d < end; d += 128) {
-        float acc = 0.f;
+    const int d = ((int)blockIdx.y * 32 + lane) * V;
+    float acc[V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) acc[e] = 0.f;
+    if (d < p.R) {
+        const float* src = p.ws_o + row * p.splits * p.R + d;
 #pragma unroll 8
-        for (int s = 0; s < p.splits; ++s) {
-            const float f = wgt[s], v = f > 0.f ? __ldcs(src + (long long)s * p.R + d) : 0.f;
-            acc = fmaf(f, v, acc);
+        for (int s = w; s < p.splits; s += 4) {
+            const float f = wgt[s];
+            const float* q = src + (f > 0.f ? (long long)s * p.R : 0ll);
+            if (V == 4) {
+                const float4 v = __ldcs(reinterpret_cast<const float4*>(q));
+                acc[0] = fmaf(f, v.x, acc[0]); acc[1 % V] = fmaf(f, v.y, acc[1 % V]); acc[2 % V] = fmaf(f, v.z, acc[2 % V]); acc[3 % V] = fmaf(f, v.w, acc[3 % V]);
+            } else {
+                acc[0] = fmaf(f, __ldcs(q), acc[0]);
+            }
         }
-        dst[d] = from_f<T>(acc * inv);
     }
+#pragma unroll
+    for (int e = 0; e < V; ++e) sum[w][lane * V + e] = acc[e];
+    __syncthreads();
+    const int col = (int)blockIdx.y * 32 * V + t;
+    if (t < 32 * V && col < p.R)
+        o[(row / p.H) * ldo + (long long)h * p.R + col] = from_f<T>((sum[0][t] + sum[1][t] + sum[2][t] + sum[3][t]) * inv);
+}
+
+template <typename T>
+int launch_combine(const LatentParams& l, long long rows, void* o, long long ldo, cudaStream_t stream) {
+    const int V = l.R % 4 == 0 ? 4 : 1;
+    const dim3 grid((unsigned)rows, (l.R + 32 * V - 1) / (32 * V));
+    if (V == 4) PLZ_LAUNCH_CHAIN((latent_combine_kernel<T, 4>), grid, dim3(128), 0, stream, l, (T*)o, ldo);
+    else PLZ_LAUNCH_CHAIN((latent_combine_kernel<T, 1>), grid, dim3(128), 0, stream, l, (T*)o, ldo);
+    return PLZ_OK;
 }
 
 template <typename T, int RT>
@@ -201,7 +223,8 @@ int plan_splits(int dtype, int B, int n, int H, int R, int dr, int cap) {
 }  // namespace
 
 long long latent_attn_ws_bytes(int dtype, int B, int n, int H, int R, int dr, int cap) {
-    return (long long)B * n * H * plan_splits(dtype, B, n, H, R, dr, cap) * (R + 2) * (long long)sizeof(float);
+    const long long slots = (long long)B * n * H * plan_splits(dtype, B, n, H, R, dr, cap);
+    return ((slots * 2 + 3) / 4 * 4 + slots * R) * (long long)sizeof(float);
 }
 
 int launch_latent_attn(int dtype, const LatentAttnArgs& a, void* ws, long long ws_bytes, cudaStream_t stream) {
@@ -212,7 +235,7 @@ int launch_latent_attn(int dtype, const LatentAttnArgs& a, void* ws, long long w
     l.splits = plan_splits(dtype, a.B, a.n, a.H, a.R, a.dr, a.cap);
     const long long rows = (long long)a.B * a.n * a.H;
     l.ws_ml = (float*)ws;
-    l.ws_o = l.ws_ml + rows * l.splits * 2;
+    l.ws_o = l.ws_ml + (rows * l.splits * 2 + 3) / 4 * 4;
     int rc;
     const bool aligned = a.scale > 0.f && a.ldq % 8 == 0 && a.c_batch % 8 == 0 && a.r_batch % 8 == 0 && !((uintptr_t)a.q & 15) && !((uintptr_t)a.c & 15) && !((uintptr_t)a.kr & 15);
     if (on_tensor_cores(dtype, a.R, a.dr) && aligned) {
@@ -223,9 +246,7 @@ int launch_latent_attn(int dtype, const LatentAttnArgs& a, void* ws, long long w
         rc = dtype == 1 ? launch_rows<float>(p, a.B, stream) : launch_rows<__nv_bfloat16>(p, a.B, stream);
     }
     if (rc) return rc;
-    if (dtype == 1) PLZ_LAUNCH_CHAIN(latent_combine_kernel<float>, dim3((unsigned)rows, (a.R + 255) / 256), dim3(128), 0, stream, l, (float*)a.o, a.ldo);
-    else PLZ_LAUNCH_CHAIN(latent_combine_kernel<__nv_bfloat16>, dim3((unsigned)rows, (a.R + 255) / 256), dim3(128), 0, stream, l, (__nv_bfloat16*)a.o, a.ldo);
-    return PLZ_OK;
+    return dtype == 1 ? launch_combine<float>(l, rows, a.o, a.ldo, stream) : launch_combine<__nv_bfloat16>(l, rows, a.o, a.ldo, stream);
 }
 
 }  // namespace plz

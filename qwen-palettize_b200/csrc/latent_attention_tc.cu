@@ -22,7 +22,8 @@ namespace {
 
 constexpr int kLatThreads = 320;
 constexpr uint32_t kUnit = 2 * kBlk;            // 128 keys x 128 latent columns
-constexpr uint32_t kPBytes = 128 * 128;         // P^T: 128 keys x 64 query rows
+// P^T: 128 keys, rows of 64 bytes (64-byte swizzle) for up to 32 query rows, else of 128
+__host__ __device__ constexpr uint32_t p_row(int N) { return N <= 32 ? 64u : 128u; }
 constexpr int kMaxUnits = 8;
 constexpr uint32_t kSmemBudget = 227 * 1024 - 1024 - 5120;   // alignment; barriers and softmax exchange (kExtra)
 constexpr uint32_t kExtra = 5120;
@@ -212,33 +213,44 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant_
     } else if (warp == 8) {
         if (lane == 0 && tiles > 0) {
             const uint32_t id_s = make_idesc(128, N, 0, 0), id_o = make_idesc(128, N, 1, 1);
-            const uint64_t dq = make_sdesc(base + p.off_q, 16u, 1024u), dp = make_sdesc(base + p.off_p, kBlk, 1024u);
+            // descriptors as words: only the low one (start address) moves
+            const uint64_t dq = make_sdesc(base + p.off_q, 16u, 1024u), dk = make_sdesc(base, 16u, 1024u), dv = make_sdesc(base, kBlk, 1024u);
+            const uint64_t dp = make_sdesc(base + p.off_p, kBlk, 8u * p_row(N)) ^ (N <= 32 ? (uint64_t)6 << 61 : 0ull);   // layout 2 -> 4: 64-byte swizzle
+            const uint32_t q_lo = (uint32_t)dq, q_hi = (uint32_t)(dq >> 32), k_lo = (uint32_t)dk, k_hi = (uint32_t)(dk >> 32);
+            const uint32_t v_lo = (uint32_t)dv, v_hi = (uint32_t)(dv >> 32), p_lo = (uint32_t)dp, p_hi = (uint32_t)(dp >> 32);
             const bool ahead = p.ring >= 2 * p.units && (p.r_blocks == 0 || p.r_ring == 2);
             bool ok = mbar_wait(q_full, 0, abort_flag, p.status, ST_TIMEOUT_FULL, 82);
             // one 64-column block of S^T
-            auto block = [&](int buf, uint32_t sA, int q_block, int cols, uint32_t& acc) {
-                const uint64_t da = make_sdesc(sA, 16u, 1024u);
-                const uint32_t bq = (uint32_t)dq + (uint32_t)(q_block * N * 8);
-                const int steps = (min(64, cols) + 15) >> 4;
-                for (int ks = 0; ks < steps; ++ks) {
-                    umma_bf16_words<1>(tS(buf), (uint32_t)da + ks * 2u, (uint32_t)(da >> 32), bq + ks * 2u, (uint32_t)(dq >> 32), id_s, acc);
-                    acc = 1u;
+            auto block = [&](uint32_t ts, uint32_t a, uint32_t bq, int cols, uint32_t acc) {
+                if (cols > 48) {
+#pragma unroll
+                    for (int ks = 0; ks < 4; ++ks) umma_bf16_words<1>(ts, a + ks * 2u, k_hi, bq + ks * 2u, q_hi, id_s, ks > 0 ? 1u : acc);
+                } else {
+                    for (int ks = 0; ks * 16 < cols; ++ks) umma_bf16_words<1>(ts, a + ks * 2u, k_hi, bq + ks * 2u, q_hi, id_s, ks > 0 ? 1u : acc);
                 }
             };
+            int s_unit = 0, s_ph = 0, v_unit = 0;          // ring positions of the scores (with its phase) and of the value products
             auto scores = [&](int j) {
-                uint32_t acc = 0u;
+                const uint32_t ts = tS(j & 1);
                 if (p.r_blocks) {
-                    const int s = j % p.r_ring;
-                    if (!mbar_wait(r_full(s), (j / p.r_ring) & 1, abort_flag, p.status, ST_TIMEOUT_FULL, 83)) return false;
+                    const int s = p.r_ring == 2 ? (j & 1) : 0;
+                    if (!mbar_wait_lean(r_full(s), (p.r_ring == 2 ? j >> 1 : j) & 1, abort_flag, p.status, ST_TIMEOUT_FULL, 83)) return false;
                     tc_fence_after_sync();
-                    for (int i = 0; i < p.r_blocks; ++i) block(j & 1, base + p.off_r + (s * p.r_blocks + i) * kBlk, p.c_blocks + i, p.l.dr - 64 * i, acc);
+                    for (int i = 0; i < p.r_blocks; ++i)
+                        block(ts, k_lo + (p.off_r >> 4) + (uint32_t)(s * p.r_blocks + i) * (kBlk >> 4), q_lo + (uint32_t)((p.c_blocks + i) * N * 8), p.l.dr - 64 * i, i > 0 ? 1u : 0u);
                     umma_commit(r_empty(s));
                 }
+                uint32_t bq = q_lo;
+                int left = R;
                 for (int m = 0; m < p.units; ++m) {
-                    const int idx = j * p.units + m, s = idx % p.ring;
-                    if (!mbar_wait(u_full(s), (idx / p.ring) & 1, abort_flag, p.status, ST_TIMEOUT_FULL, 84)) return false;
+                    if (!mbar_wait_lean(u_full(s_unit), s_ph, abort_flag, p.status, ST_TIMEOUT_FULL, 84)) return false;
                     tc_fence_after_sync();
-                    for (int i = 0; i < min(2, p.c_blocks - 2 * m); ++i) block(j & 1, base + s * kUnit + i * kBlk, 2 * m + i, R - 64 * (2 * m + i), acc);
+                    const uint32_t a = k_lo + (uint32_t)s_unit * (kUnit >> 4);
+                    block(ts, a, bq, left, (m > 0 || p.r_blocks) ? 1u : 0u);
+                    if (left > 64) block(ts, a + (kBlk >> 4), bq + (uint32_t)(N * 8), left - 64, 1u);
+                    bq += 2u * N * 8;
+                    left -= 128;
+                    if (++s_unit == p.ring) { s_unit = 0; s_ph ^= 1; }
                 }
                 umma_commit(s_full(j & 1));
                 return true;
@@ -246,16 +258,16 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant_
             if (ok) ok = scores(0);
             for (int j = 0; j < tiles && ok; ++j) {
                 if (ahead && j + 1 < tiles) { ok = scores(j + 1); if (!ok) break; }
-                ok = mbar_wait(p_full, j & 1, abort_flag, p.status, ST_TIMEOUT_FULL, 85);
+                ok = mbar_wait_lean(p_full, j & 1, abort_flag, p.status, ST_TIMEOUT_FULL, 85);
                 if (!ok) break;
                 tc_fence_after_sync();
+                const uint32_t acc = j > 0 ? 1u : 0u;
                 for (int m = 0; m < p.units; ++m) {
-                    const int s = (j * p.units + m) % p.ring;
-                    const uint64_t da = make_sdesc(base + s * kUnit, kBlk, 1024u);
+                    const uint32_t a = v_lo + (uint32_t)v_unit * (kUnit >> 4), to = tO(m);
 #pragma unroll
-                    for (int ks = 0; ks < 8; ++ks)
-                        umma_bf16_words<1>(tO(m), (uint32_t)da + ks * 128u, (uint32_t)(da >> 32), (uint32_t)dp + ks * 128u, (uint32_t)(dp >> 32), id_o, (j > 0 || ks > 0) ? 1u : 0u);
-                    umma_commit(u_empty(s));
+                    for (int ks = 0; ks < 8; ++ks) umma_bf16_words<1>(to, a + ks * 128u, v_hi, p_lo + ks * p_row(N), p_hi, id_o, ks > 0 ? 1u : acc);
+                    umma_commit(u_empty(v_unit));
+                    if (++v_unit == p.ring) v_unit = 0;
                 }
                 umma_commit(o_done);
                 if (!ahead && j + 1 < tiles) ok = scores(j + 1);
@@ -329,7 +341,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant_
             }
 #pragma unroll
             for (int q = 0; q < NC / 8; ++q)
-                *reinterpret_cast<uint4*>(smem + p.off_p + swz128(t, (c0 >> 3) + q)) =
+                *reinterpret_cast<uint4*>(smem + p.off_p + (N <= 32 ? t * 64u + ((((c0 >> 3) + q) ^ ((t >> 1) & 3)) << 4) : swz128(t, (c0 >> 3) + q))) =
                     make_uint4(pack_bf16x2(s[q * 8], s[q * 8 + 1]), pack_bf16x2(s[q * 8 + 2], s[q * 8 + 3]), pack_bf16x2(s[q * 8 + 4], s[q * 8 + 5]),
                                pack_bf16x2(s[q * 8 + 6], s[q * 8 + 7]));
             if (tok >= total && half == 0) {                              // past the sequence: whatever the cache holds there must not count
@@ -391,17 +403,18 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant_
 // shared-memory plan of a CTA with N query rows; false if it does not fit
 bool plan(int R, int dr, int N, LatTcParams* p) {
     p->c_blocks = (R + 63) / 64; p->r_blocks = (dr + 63) / 64; p->units = (R + 127) / 128;
-    const uint32_t fixed = kPBytes + (uint32_t)(p->c_blocks + p->r_blocks) * N * 128;
+    const uint32_t p_bytes = 128 * p_row(N), fixed = p_bytes + (uint32_t)(p->c_blocks + p->r_blocks) * N * 128;
     const uint32_t part = (uint32_t)p->r_blocks * kBlk;
     if (fixed + part + p->units * kUnit > kSmemBudget) return false;
-    p->r_ring = fixed + 2 * part + p->units * kUnit <= kSmemBudget ? 2 : 1;
+    // two whole tiles if they fit (then the scores run a tile ahead), else as many units as fit beside one key part
+    p->r_ring = fixed + 2 * part + 2 * p->units * kUnit <= kSmemBudget && 2 * p->units <= kMaxUnits ? 2 : 1;
     uint32_t ring = (kSmemBudget - fixed - p->r_ring * part) / kUnit;
     if (ring > 2u * p->units) ring = 2u * p->units;
     if (ring > (uint32_t)kMaxUnits) ring = kMaxUnits;
     p->ring = (int)ring;
     p->off_r = ring * kUnit;
     p->off_p = p->off_r + p->r_ring * part;
-    p->off_q = p->off_p + kPBytes;
+    p->off_q = p->off_p + p_bytes;
     p->off_x = p->off_q + (uint32_t)(p->c_blocks + p->r_blocks) * N * 128;
     p->tmem_cols = 32;
     while (p->tmem_cols < (uint32_t)(N * (2 + p->units))) p->tmem_cols *= 2;
