@@ -89,7 +89,7 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) { *reinterpre
 __device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
 __device__ __forceinline__ float dot4(float4 a) { return a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w; }
 template <typename T, int NQ>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, NQ <= 2 ? 8 : (NQ <= 4 ? 6 : 3))
 stream4_kernel(const StreamParams p) {
     __shared__ float part[8];
     const long long r = blockIdx.x;
@@ -479,6 +479,7 @@ static int stream_t_(const StreamArgs& a, cudaStream_t s) {
     const bool vec = a.W % 4 == 0 && a.ldy % 4 == 0 && !(ptrs & 15);
     const dim3 grid((unsigned)a.rows), block(256);
     if (vec && a.W <= 2048) PLZ_LAUNCH_CHAIN((stream4_kernel<T, 2>), grid, block, 0, s, p);
+    else if (vec && a.W <= 3072) PLZ_LAUNCH_CHAIN((stream4_kernel<T, 3>), grid, block, 0, s, p);
     else if (vec && a.W <= 4096) PLZ_LAUNCH_CHAIN((stream4_kernel<T, 4>), grid, block, 0, s, p);
     else if (vec && a.W <= 8192) PLZ_LAUNCH_CHAIN((stream4_kernel<T, 8>), grid, block, 0, s, p);
     else PLZ_LAUNCH_CHAIN(stream_kernel<T>, grid, block, 0, s, p);

@@ -303,7 +303,7 @@ class LatentAttention:
 
     def _absorb(self, ctx: StepContext) -> bool:
         """Fewer multiplications per head (those of the absorbed attention count twice: its tiles are narrower)."""
-        if ctx.n == 1:
+        if ctx.n == 1 or self.dn + self.dr > 512 or self.dv > 256:        # heads larger than the ordinary attention kernels take
             return True
         n, pos = ctx.n, ctx.host_pos
         pairs, per = n * (pos + 0.5 * n), self.R * (self.dn + self.dv)
