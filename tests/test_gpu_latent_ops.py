@@ -187,7 +187,7 @@ def test_latent_attention_long_and_split():
 
 
 @pytest.mark.parametrize("dt", DT)
-@pytest.mark.parametrize("Hh,dn,dr,dv", [(3, 24, 16, 40), (2, 128, 64, 128), (4, 64, 32, 48), (2, 40, 0, 16), (2, 64, 128, 72), (3, 10, 6, 7), (1, 200, 40, 144), (2, 8, 8, 8)])
+@pytest.mark.parametrize("Hh,dn,dr,dv", [(3, 24, 16, 40), (2, 128, 64, 128), (5, 56, 24, 72), (2, 40, 0, 16), (2, 64, 128, 72), (3, 10, 6, 7), (1, 200, 40, 144), (2, 8, 8, 8)])
 @pytest.mark.parametrize("B,n,pos", [(1, 2, 0), (2, 130, 0), (1, 64, 100), (2, 33, 127), (1, 300, 129)])
 def test_attention_with_a_shared_key_part(dt, Hh, dn, dr, dv, B, n, pos):
     """Own and shared key columns, learned sinks, gate, keys and values side by side in one buffer."""
